@@ -69,6 +69,15 @@ def _gimotar(c: dict):
 register_architecture("Gimotar", _gimotar)
 
 
+def _gimupel(c: dict):
+    from .gimupel import GimupelConfig
+    cfg = GimupelConfig.from_json(c)
+    return cfg, cfg.spec()
+
+
+register_architecture("Gimupel", _gimupel)
+
+
 def read_config_json(model_dir: str) -> dict:
     path = os.path.join(model_dir, "config.json")
     if not os.path.isfile(path):

@@ -41,10 +41,12 @@ class LayerSpec:
 @dataclass(frozen=True)
 class ScheduleEntry:
     """One execution of a layer. `cache` is the cache slot the mixer uses: entries with the same `cache` share keys and
-    values; `write_cache=False` means this execution only reads what the slot's owner wrote earlier in the same step."""
+    values; `write_cache=False` means this execution only reads what the slot's owner wrote earlier in the same step.
+    `add_embedding`: the residual stream as the embedding left it is added to the stream right before this execution."""
     layer: int
     cache: int
     write_cache: bool = True
+    add_embedding: bool = False
 
 
 @dataclass(frozen=True)

@@ -22,7 +22,7 @@ import numpy as np
 import torch
 
 from ..cache import CacheManager
-from ..parts import LayerCache
+from ..parts import LayerCache, PendingSum
 from .model import DecoderModel
 
 
@@ -238,6 +238,7 @@ class StepRunner:
                 lc.group, lc.page_size = g, cache.page_size
             lc.state = {name: t for (entry, name), t in cache.states.tensors.items() if entry == n}
             self.layer_caches.append(lc)
+        self.keep_embedding = any(e.add_embedding for e in model.spec.schedule)
         self.embed_state = {name: t for (entry, name), t in cache.states.tensors.items() if entry == -1}
 
     def forward(self, ids_out: torch.Tensor | None = None) -> torch.Tensor | None:
@@ -259,10 +260,14 @@ class StepRunner:
         ctx.shared.clear()
         x = self.ws.get("x", (meta.n_rows, spec.hidden_size), torch.float32)
         src = meta.src if self.prev_ids is not None else None
+        # the embedding output, kept where a later entry of the schedule adds it again (written by the gather itself
+        # where nothing else adds to it)
+        kept = self.ws.get("embed_out", tuple(x.shape), torch.float32) if self.keep_embedding else None
+        also = {"copy": kept} if kept is not None and not model.embed_extras else {}
         if model.embed_scale != 1.0:
-            self.ops.embed(model.embed, meta.tokens, x, src, self.prev_ids, model.embed_scale)
+            self.ops.embed(model.embed, meta.tokens, x, src, self.prev_ids, model.embed_scale, **also)
         else:
-            self.ops.embed(model.embed, meta.tokens, x, src, self.prev_ids)
+            self.ops.embed(model.embed, meta.tokens, x, src, self.prev_ids, **also)
         if "token_ids" in self.needs:
             ctx.token_ids = meta.tokens
             if src is not None:      # some rows take their token from the ids the previous step left on the device
@@ -270,8 +275,14 @@ class StepRunner:
                 self.ops.select_tokens(meta.tokens, src, self.prev_ids, ctx.token_ids)
         for part in model.embed_extras:
             part.forward(ctx, x, self.embed_state)
+        if kept is not None and not also:
+            self.ops.weighted_sum([x], [1.0], kept)
         delta = None
         for e, lc in zip(spec.schedule, self.layer_caches):
+            if e.add_embedding:
+                if hasattr(delta, "resolve"):
+                    delta = delta.resolve(ctx, x)
+                delta = PendingSum(delta, kept)
             x, delta = model.layers[e.layer].forward(ctx, x, delta, lc)
         logits = self.ws.get("logits", (meta.n_wanted, spec.vocab_size), torch.float32)
         if meta.n_wanted:

@@ -38,9 +38,10 @@ class Ops:
         raise NotImplementedError
 
     def embed(self, table: torch.Tensor, tokens: torch.Tensor, x: torch.Tensor, src: torch.Tensor | None = None,
-              prev_ids: torch.Tensor | None = None, scale: float = 1.0) -> None:
+              prev_ids: torch.Tensor | None = None, scale: float = 1.0, copy: torch.Tensor | None = None) -> None:
         """x[n, :] = float32(table[tokens[n], :]) * scale. tokens: int32 (N,). A token outside the table is an error.
-        With src (int32 (N,)) and prev_ids (int32): a row with src[n] >= 0 uses token prev_ids[src[n]] instead."""
+        With src (int32 (N,)) and prev_ids (int32): a row with src[n] >= 0 uses token prev_ids[src[n]] instead.
+        copy (N, D) float32: receives the same values as x."""
         raise NotImplementedError
 
     def add_rmsnorm(self, x: torch.Tensor, delta: torch.Tensor | None, weight: torch.Tensor, eps: float,
@@ -50,12 +51,20 @@ class Ops:
         groups > 1: the row is split into that many equal consecutive parts and the mean is taken over each part alone."""
         raise NotImplementedError
 
+    def add_layernorm(self, x: torch.Tensor, delta: torch.Tensor | None, extra: torch.Tensor | None, weight: torch.Tensor,
+                      eps: float, h: torch.Tensor, rows: torch.Tensor | None = None) -> None:
+        """rows None: x = (x + delta) + extra (each if given), in place; h[n] = T(weight * (x[n] - m) / sqrt(mean((x[n] -
+        m)^2) + eps)), m = mean(x[n]). rows (int32 (R,), -1 = none): h[r] is computed from x[rows[r]] + delta[rows[r]]; x is
+        not written and extra must be None. weight (D,) float32; delta, extra (N, D) float32."""
+        raise NotImplementedError
+
     def select_tokens(self, tokens: torch.Tensor, src: torch.Tensor, prev_ids: torch.Tensor, out: torch.Tensor) -> None:
         """out[n] = prev_ids[src[n]] if src[n] >= 0 else tokens[n] (all int32): the ids `embed` reads, as one tensor."""
         raise NotImplementedError
 
     def short_conv(self, h: torch.Tensor, w: torch.Tensor, state: torch.Tensor | None, meta: Any, out: torch.Tensor,
-                   residual: bool = True, activation: str | None = None, bias: torch.Tensor | None = None) -> None:
+                   residual: bool = True, activation: str | None = None, bias: torch.Tensor | None = None,
+                   offset: int | None = None) -> None:
         """Causal convolution over time within each portion of the step (meta.seg: first row, rows, first position,
         state slot). h, out: (N, C) T; w: (C, taps) T; state: (slots, taps - 1, C) float32, the last taps - 1 inputs of
         each request so far, oldest first. For the row at place i of its portion:
@@ -63,7 +72,8 @@ class Ops:
         state[slot, taps - 1 + k]. The sum is float32, j rising, rounded once. Afterwards state[slot] holds the portion's
         request's last taps - 1 inputs. Padding rows give zeros. activation "silu": out = z * sigmoid(z) of
         the float32 sum z (residual included), rounded once. bias (C,) float32: added to the sum after the taps, before
-        the residual and the activation."""
+        the residual and the activation. offset: h is (N, any width) float32 and the C inputs of a row are its columns
+        from `offset` on (no residual then); out stays (N, C) T."""
         raise NotImplementedError
 
     def gated_sum(self, a: torch.Tensor, gate_a: torch.Tensor | None, f: torch.Tensor | None, gate_f: torch.Tensor | None,
@@ -158,10 +168,24 @@ class Ops:
         raise NotImplementedError
 
     def head_norm_gate(self, o: torch.Tensor, heads: int, value_dim: int, weight: torch.Tensor | None, eps: float,
-                       gate: torch.Tensor | None, gate_offset: int, activation: str | None, out: torch.Tensor) -> None:
+                       gate: torch.Tensor | None, gate_offset: int, activation: str | None, out: torch.Tensor,
+                       gate_first: bool = False) -> None:
         """o: (N, H dv) float32. out[n, h, c] = T(o / sqrt(mean_c(o[n, h]^2) + eps) * weight[c] * act(gate[n, gate_offset +
         h dv + c])); weight (dv,) float32, shared by the heads, or (H dv,), one per head and channel (weight[h dv + c]),
-        or None (1); gate float32 (N, any width) or None (1); act "silu", "sigmoid"."""
+        or None (1); gate float32 (N, any width) or None (1); act "silu", "sigmoid". gate_first: the gate is applied before
+        the norm: u = o * act(gate), out = T(u / sqrt(mean_c(u[n, h]^2) + eps) * weight)."""
+        raise NotImplementedError
+
+    def ssd_scan(self, xbc: torch.Tensor, heads: int, groups: int, state_dim: int, value_dim: int, dt: torch.Tensor,
+                 dt_offset: int, dt_bias: torch.Tensor, a_log: torch.Tensor, skip: torch.Tensor, state: torch.Tensor,
+                 meta: Any, out: torch.Tensor) -> None:
+        """xbc: (N, H P + 2 G S) T, a row = [x heads | B groups | C groups]; dt: (N, any width) float32 whose columns
+        dt_offset .. dt_offset + H - 1 are the step sizes before bias and softplus; dt_bias, a_log, skip (H,) float32. Per
+        portion (meta.seg), token by token, per head h (group h // (H / G)), with the slot's state M (S x P): d = softplus(dt +
+        dt_bias[h]), M = exp(-exp(a_log[h]) * d) * M + (d * B) x^T, out[n, h] = M^T C + skip[h] * x. float32 throughout
+        (softplus(z) = max(z, 0) + log1p(exp(-|z|))); out (N, H P) float32; the state (`recurrent_state_shape(H, S, P)`) is
+        that after the portion's last token. Rows of padding are left as they are. A table may compute a long portion in
+        blocks of tokens, in another order of the same sums."""
         raise NotImplementedError
 
     def general_delta_scan(self, proj: torch.Tensor, heads: int, key_dim: int, value_dim: int, remove_offset: int,
@@ -259,11 +283,16 @@ class Ops:
         raise NotImplementedError
 
     def route_by_scores(self, logits: torch.Tensor, num_experts: int, top: int, groups: int, keep_groups: int,
-                        renormalize: bool, meta: Any, weights: torch.Tensor, align: int = 1) -> Any:
+                        renormalize: bool, meta: Any, weights: torch.Tensor, align: int = 1, scoring: str = "softmax",
+                        correction: torch.Tensor | None = None, group_top: int = 1, sum_eps: float = 0.0,
+                        scale: float = 1.0) -> Any:
         """logits: (N, >= E) float32, the first E columns are router logits. s = softmax over them; the experts form
         `groups` equal groups of neighbours, a group's score is its largest s, only experts of the keep_groups best groups
         (lower index first among equals) can be chosen; of those the `top` with the largest s (lower index first among
         equals), in falling order. weights[n, k] = s of the k-th choice (divided by their sum if renormalize); float32.
+        scoring "sigmoid": s = sigmoid(logit). correction (E,) float32: experts and groups are compared by s + correction,
+        the weights stay s. group_top 2: a group's score is the sum of its two largest (of its one, if it has one).
+        sum_eps: added to the sum that renormalize divides by; scale: multiplies the weights last.
         Returns the route of the (row, choice) pairs sorted by expert, as `route_by_table` does."""
         raise NotImplementedError
 

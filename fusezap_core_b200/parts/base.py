@@ -10,7 +10,8 @@ through the kernel table of the step (`ctx.ops`), taking scratch buffers from `c
                                                 (rows given: only those rows are normed and x is left as it is)
   PositionEncoding.prepare(max_len, device)      builds its tables
   PositionEncoding.rotate_and_store(ctx, qkv, q_out, cache, num_heads, num_kv_heads, head_dim)
-  Block.forward(ctx, x, delta, cache) -> (x, delta)   the arrangement of norms, mixer and feed-forward of one layer
+  Block.forward(ctx, x, delta, cache) -> (x, delta)   the arrangement of norms, mixer and feed-forward of one layer;
+                                                the delta handed in may be an object with `resolve(ctx, x) -> delta`
   LogitTransform.forward(ctx, logits) -> None    changes the float32 logits of the wanted rows in place
   EmbedExtra.forward(ctx, x, state) -> None      adds to the gathered embeddings x (N, D) float32 before the first layer
 
@@ -75,6 +76,23 @@ class LayerCache:
     page_size: int = 0
     write: bool = True                      # False: read what the slot's owner wrote earlier in this step
     state: dict[str, torch.Tensor] = field(default_factory=dict)   # name -> (num_slots, *shape) float32
+
+
+@dataclass
+class PendingSum:
+    """A pending residual term (or none) with one more stream to be added after it: what stands in place of the pending
+    term where a schedule entry adds the embedding output again. A norm that can add both in its own pass does; any other
+    consumer calls `resolve`, which adds the term and hands back the other stream as the one still pending."""
+    delta: torch.Tensor | None
+    extra: torch.Tensor
+
+    def fold_into_norm(self, ctx, x, weight, eps, h, rows) -> bool:
+        return False
+
+    def resolve(self, ctx, x) -> torch.Tensor:
+        if self.delta is not None:
+            ctx.ops.weighted_sum([x, self.delta], [1.0, 1.0], x)
+        return self.extra
 
 
 class Part:

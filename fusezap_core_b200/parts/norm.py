@@ -1,4 +1,4 @@
-"""RMSNorm with the residual add folded in.
+"""RMSNorm and LayerNorm with the residual add folded in.
 
 `x <- x + delta` (the pending term of the previous sublayer), then `h = w * (x / sqrt(mean(x^2) + eps))`
 (fusezap/serve/models/llama.py:500-503, 508-523: `mean = sum * (1/D)`, the fused kernel also writes the residual
@@ -6,12 +6,15 @@ stream). The residual stream x is float32 in both dtypes; the sum of squares, th
 computed in 32-bit and h is rounded once to the activation dtype. With `groups` > 1 the vector is normed in that many
 equal consecutive parts, each by its own mean square; the weight still spans the whole vector. With `offset` the
 multiplier is `offset + w` (a weight stored as its distance from one has offset 1), added in float32 once at load.
+
+LayerNorm: `h = w * (x - mean(x)) / sqrt(mean((x - mean(x))^2) + eps)`, no bias; the same residual add, and where the
+pending term is a `PendingSum` its other stream is added in the same pass.
 """
 from __future__ import annotations
 import torch
 
 from ..weights import ParamSpec
-from .base import Norm, register_norm
+from .base import Norm, PendingSum, register_norm
 
 
 @register_norm("rmsnorm")
@@ -59,3 +62,30 @@ class RMSNorm(Norm):
             ctx.ops.add_rmsnorm(x, delta, self.weight, self.eps, h, rows)
         else:
             ctx.ops.add_rmsnorm(x, delta, self.weight, self.eps, h, rows, groups=self.groups)
+
+
+@register_norm("layernorm")
+class LayerNorm(Norm):
+    def __init__(self, size: int, eps: float, name: str = "weight"):
+        """name: the weight's tensor name relative to the part ("" when the part's prefix is the whole name)."""
+        self.size, self.eps, self.name = size, float(eps), name
+        self.weight: torch.Tensor | None = None
+
+    def tensors(self) -> dict[str, ParamSpec]:
+        return {self.name: ParamSpec((self.size,), role="vector", init="ones")}
+
+    def bind(self, tensors, ops) -> None:
+        self.weight = tensors[self.name].float().contiguous()
+
+    def forward(self, ctx, x, delta, rows=None, n_rows=None):
+        n = x.shape[0] if rows is None else (n_rows if n_rows is not None else rows.shape[0])
+        h = ctx.ws.get("norm_h" if rows is None else "norm_h_rows", (n, self.size), ctx.ops.dtype)
+        extra = None
+        if isinstance(delta, PendingSum) and rows is None:
+            delta, extra = delta.delta, delta.extra
+        elif hasattr(delta, "resolve"):
+            if rows is not None:
+                raise NotImplementedError("a pending operation on the stream cannot be resolved for selected rows only")
+            delta = delta.resolve(ctx, x)
+        ctx.ops.add_layernorm(x, delta, extra, self.weight, self.eps, h, rows)
+        return h

@@ -11,7 +11,12 @@ and the weighted sum are 32-bit; the activation is computed from unrounded 32-bi
 
 Options: `router_bias`: the logits are `W_router h + b` (tensor `<router_bias>`); `shared_gate=False`: the shared expert
 is added as it is, without a gate. With one group and `renormalize`, the weights are the softmax over the chosen logits
-alone (softmax over all, divided by the chosen ones' sum, is the same number). The part takes a block's other term and
+alone (softmax over all, divided by the chosen ones' sum, is the same number). `scoring` "sigmoid": s = sigmoid(z);
+`correction`: experts and groups are chosen by `s + c` (tensor `<correction>`, one number per expert) while the weights
+use s; `group_score` "top2": a group's score is the sum of its two largest choice scores (of its only one, if it has
+one); `sum_eps` is added to the sum that `renormalize` divides by; `weight_scale` multiplies the weights last.
+`alpha`, `limit`, `up_shift`: an expert computes g = min(W_gate h, limit), u = clamp(W_up h, -limit, limit) and
+`W_down (g * sigmoid(alpha g) * (u + up_shift))`; the defaults are silu(g) * u. The part takes a block's other term and
 multiplier into its last kernel: `forward(ctx, h, add=a, scale=m)` returns `m * (a + ff(h))`.
 """
 from __future__ import annotations
@@ -24,7 +29,9 @@ from .base import FeedForward, register_feed_forward
 from .feed_forward import SwiGLU
 
 _NAMES = {"router": "router", "expert": "experts.{}", "gate": "gate_proj", "up": "up_proj", "down": "down_proj",
-          "shared": "shared_expert", "shared_gate": "shared_gate", "router_bias": "router.bias"}
+          "shared": "shared_expert", "shared_gate": "shared_gate", "router_bias": "router.bias", "correction": "correction"}
+SCORINGS = ("softmax", "sigmoid")
+GROUP_SCORES = {"max": 1, "top2": 2}       # how many of a group's largest choice scores are added up
 
 
 @register_feed_forward("routed_moe")
@@ -33,7 +40,9 @@ class RoutedMoE(FeedForward):
 
     def __init__(self, hidden_size: int, intermediate_size: int, num_experts: int, top: int, groups: int = 1,
                  keep_groups: int = 1, shared_size: int = 0, renormalize: bool = False, names: dict | None = None,
-                 router_bias: bool = False, shared_gate: bool = True):
+                 router_bias: bool = False, shared_gate: bool = True, scoring: str = "softmax", correction: bool = False,
+                 group_score: str = "max", sum_eps: float = 0.0, weight_scale: float = 1.0, alpha: float = 1.0,
+                 limit: float = math.inf, up_shift: float = 0.0):
         if not 0 < top <= num_experts:
             raise ValueError(f"top {top} must lie in 1..{num_experts}")
         if groups <= 0 or num_experts % groups or not 0 < keep_groups <= groups or top > keep_groups * (num_experts // groups):
@@ -41,6 +50,12 @@ class RoutedMoE(FeedForward):
         self.D, self.I, self.E, self.top = hidden_size, intermediate_size, num_experts, top
         self.groups, self.keep, self.renormalize = int(groups), int(keep_groups), bool(renormalize)
         self.names = {**_NAMES, **(names or {})}
+        if scoring not in SCORINGS or group_score not in GROUP_SCORES:
+            raise ValueError(f"scoring {scoring!r} / group_score {group_score!r} is not one of {SCORINGS} / {sorted(GROUP_SCORES)}")
+        self.scoring, self.has_correction, self.group_top = scoring, bool(correction), GROUP_SCORES[group_score]
+        self.sum_eps, self.weight_scale = float(sum_eps), float(weight_scale)
+        self.alpha, self.limit, self.up_shift = float(alpha), float(limit), float(up_shift)
+        self.correction = None
         self.router_bias, self.shared_gate = bool(router_bias), bool(shared_gate) and shared_size > 0
         self.b_router = None
         self.shared = None
@@ -64,6 +79,8 @@ class RoutedMoE(FeedForward):
         out[n["router"]] = ParamSpec((self.E, self.D))
         if self.router_bias:
             out[n["router_bias"]] = ParamSpec((self.E,), role="vector")
+        if self.has_correction:
+            out[n["correction"]] = ParamSpec((self.E,), role="vector")
         if self.shared is not None:
             out.update({f"{n['shared']}.{k}": v for k, v in self.shared.tensors().items() if v.group is None})
             if self.shared_gate:
@@ -85,6 +102,8 @@ class RoutedMoE(FeedForward):
         if self.router_bias:
             b = tensors[n["router_bias"]].float()
             self.b_router = torch.cat([b, b.new_zeros(router.shape[0] - self.E)]).contiguous()
+        if self.has_correction:
+            self.correction = tensors[n["correction"]].float().contiguous()
 
     def weight_tensors(self) -> list:
         return [self.w_router, self.w_gate_up, self.w_down]
@@ -94,10 +113,14 @@ class RoutedMoE(FeedForward):
         z = ws.get("router_logits", (n, self.w_router.shape[0]), torch.float32)
         ops.linear(h, self.w_router, self.b_router, z)
         weights = ws.get("router_weights", (n, self.top), torch.float32)
+        rule = {}
+        if (self.scoring, self.has_correction, self.group_top, self.sum_eps, self.weight_scale) != ("softmax", False, 1, 0.0, 1.0):
+            rule = {"scoring": self.scoring, "correction": self.correction, "group_top": self.group_top,
+                    "sum_eps": self.sum_eps, "scale": self.weight_scale}
         route = ops.route_by_scores(z, self.E, self.top, self.groups, self.keep, self.renormalize, ctx.meta, weights,
-                                    math.gcd(self.D, self.I))
+                                    math.gcd(self.D, self.I), **rule)
         y = ws.get("moe_act", (n * self.top, self.I), ops.dtype)             # rows in the sorted order of the pairs
-        ops.grouped_linear_glu(h, self.w_gate_up, route, y, 1.0, math.inf, 0.0)      # silu(gate) * up
+        ops.grouped_linear_glu(h, self.w_gate_up, route, y, self.alpha, self.limit, self.up_shift)
         terms = ws.get("moe_terms", (n * self.top, self.D), torch.float32)   # row n * top + k: the k-th expert of row n
         ops.grouped_linear_scatter(y, self.w_down, route, terms)
         shared = self.shared.forward(ctx, h, tag="shared_") if self.shared is not None else None

@@ -4,7 +4,8 @@
 multiplies the token's own input). A step may bring any portion of a sequence: the last `taps - 1` inputs of the
 sequence so far live in a state slot `(taps - 1, size)` (oldest first, zero when the request gets its slot), are read
 for the first rows of the portion and replaced by the portion's last inputs afterwards. The sum is in 32-bit, taps in
-rising j, and rounded once.
+rising j, and rounded once. The input may be a range of columns of a wider float32 product (`forward(..., offset=)`),
+which is then neither copied nor rounded before the convolution.
 """
 from __future__ import annotations
 import torch
@@ -43,9 +44,14 @@ class ShortConv(Part):
     def state_need(self) -> dict:
         return {"conv": (self.taps - 1, self.size)} if self.taps > 1 else {}
 
-    def forward(self, ctx, h: torch.Tensor, state: torch.Tensor | None, tag: str = "conv_out") -> torch.Tensor:
+    def forward(self, ctx, h: torch.Tensor, state: torch.Tensor | None, tag: str = "conv_out", offset: int | None = None) -> torch.Tensor:
         """h: (N, size) T; state: (slots, taps - 1, size) float32 (None when taps == 1). Returns (N, size) T and leaves
-        the state of every portion's request at the portion's end."""
+        the state of every portion's request at the portion's end. With `offset`: h is (N, any width) float32 and the
+        inputs are its columns from `offset` on."""
+        if offset is not None:
+            out = ctx.ws.get(tag, (h.shape[0], self.size), ctx.ops.dtype)
+            ctx.ops.short_conv(h, self.weight, state, ctx.meta, out, self.residual, self.activation, bias=self.bias, offset=offset)
+            return out
         out = ctx.ws.get(tag, tuple(h.shape), h.dtype)
         if self.bias is not None:
             ctx.ops.short_conv(h, self.weight, state, ctx.meta, out, self.residual, self.activation, bias=self.bias)

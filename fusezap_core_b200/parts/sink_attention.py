@@ -14,7 +14,8 @@ mixer gives back pages that lie wholly between the kept first tokens and the win
 
 Options, all off by default: `bias` names the products that have one (of "q", "k", "v", "out"; tensor `<name><bias_suffix>`);
 `qk_norm`: every q and k head is divided by its root mean square (`norm_eps` inside the root) and multiplied by a weight
-of key_dim values shared by the heads (`<q><norm_suffix>`, `<k><norm_suffix>`), before the rotation; `query_temperature`
+of key_dim values shared by the heads (`<q><norm_suffix>`, `<k><norm_suffix>`; `norm_weight=False`: there is no such
+weight), before the rotation; `query_temperature`
 (coef, every): q at position p is multiplied by `1 + coef * ln(floor((p + 1) / every) + 1)`; `softcap` c > 0: the scaled
 score s becomes `c * tanh(s / c)`; `head_gate`: head h's output is multiplied by `sigmoid(W_gate h)_h`, one number per
 head, before the output product; `own_kv=False`: the layer has no key and value projections and reads, with queries of
@@ -46,7 +47,7 @@ class SinkAttention(Mixer):
                  position: str | None = None, names: dict | None = None, bias: tuple = (), bias_suffix: str = ".bias",
                  qk_norm: bool = False, norm_eps: float = 1e-6, norm_suffix: str = "_norm", query_temperature: tuple | None = None,
                  softcap: float = 0.0, head_gate: bool = False, own_kv: bool = True, cache_window: int | None = None,
-                 span: int = 0, value_mix: str | None = None, value_mix_key: str = "first_values"):
+                 span: int = 0, value_mix: str | None = None, value_mix_key: str = "first_values", norm_weight: bool = True):
         if num_heads % num_kv_heads:
             raise ValueError(f"{num_heads} query heads are not a multiple of {num_kv_heads} kv heads")
         if pairing not in PAIRINGS:
@@ -63,6 +64,7 @@ class SinkAttention(Mixer):
             raise ValueError(f"query temperature {query_temperature!r}: the period must be positive")
         self.bias, self.bias_suffix = tuple(bias), bias_suffix
         self.qk_norm, self.norm_eps, self.norm_suffix = bool(qk_norm), float(norm_eps), norm_suffix
+        self.norm_weight = bool(norm_weight)
         self.q_temp = (float(query_temperature[0]), int(query_temperature[1])) if query_temperature is not None else None
         self.softcap, self.head_gate, self.own_kv = float(softcap), bool(head_gate), bool(own_kv)
         self.cache_window = self.window if cache_window is None else int(cache_window)
@@ -87,7 +89,7 @@ class SinkAttention(Mixer):
         for x in self.bias:
             if self.own_kv or x not in ("k", "v"):
                 out[n[x] + self.bias_suffix] = ParamSpec((rows[x],), role="vector")
-        if self.qk_norm:
+        if self.qk_norm and self.norm_weight:
             out[n["q"] + self.norm_suffix] = ParamSpec((self.dk,), role="vector", init="ones")
             if self.own_kv:
                 out[n["k"] + self.norm_suffix] = ParamSpec((self.dk,), role="vector", init="ones")
@@ -114,7 +116,10 @@ class SinkAttention(Mixer):
         self.wo = tensors[n["out"]]
         self.bo = tensors[n["out"] + self.bias_suffix].float().contiguous() if "out" in self.bias else None
         self.sink = tensors[n["sink"]].float().contiguous() if self.has_sink else None
-        if self.qk_norm:
+        if self.qk_norm and not self.norm_weight:      # (the kernel multiplies by ones: exact)
+            self.q_norm_w = torch.ones(self.dk, dtype=torch.float32, device=self.wqkv.device)
+            self.k_norm_w = self.q_norm_w if self.own_kv else None
+        elif self.qk_norm:
             self.q_norm_w = tensors[n["q"] + self.norm_suffix].float().contiguous()
             self.k_norm_w = tensors[n["k"] + self.norm_suffix].float().contiguous() if self.own_kv else None
         if self.value_mix == "blend":

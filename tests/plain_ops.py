@@ -689,3 +689,77 @@ class PlainOpsGated(PlainOpsDeep):
         if add is not None:
             acc = acc + add
         out.copy_(acc * scale)
+
+
+class PlainOpsSpace(PlainOpsGated):
+    """The operations of the state-space mixer, of the layer norm, of a schedule that adds the embedding output again, and
+    of the router with sigmoid scores and a correction."""
+
+    def embed(self, table, tokens, x, src=None, prev_ids=None, scale=1.0, copy=None) -> None:
+        super().embed(table, tokens, x, src, prev_ids, scale)
+        if copy is not None:
+            copy.copy_(x)
+
+    def add_layernorm(self, x, delta, extra, weight, eps, h, rows=None) -> None:
+        if rows is None:
+            for t in (delta, extra):
+                if t is not None:
+                    x.add_(t)
+            src = x
+        else:
+            assert extra is None
+            r = rows.long().clamp(min=0)
+            src = x[r] + (delta[r] if delta is not None else 0)
+        d = src - src.mean(-1, keepdim=True)
+        y = weight.float() * (d * torch.rsqrt((d * d).mean(-1, keepdim=True) + eps))
+        if rows is not None:
+            y = torch.where((rows < 0)[:, None], torch.zeros_like(y), y)
+        h.copy_(y.to(h.dtype))
+
+    def short_conv(self, h, w, state, meta, out, residual=True, activation=None, bias=None, offset=None) -> None:
+        if offset is not None:
+            assert h.dtype == torch.float32 and not residual
+            h = h[:, offset: offset + out.shape[1]]
+        super().short_conv(h, w, state, meta, out, residual, activation, bias)
+
+    def head_norm_gate(self, o, heads, value_dim, weight, eps, gate, gate_offset, activation, out, gate_first=False):
+        if not gate_first:
+            return super().head_norm_gate(o, heads, value_dim, weight, eps, gate, gate_offset, activation, out)
+        n = o.shape[0]
+        u = (o * self._act(gate[:, gate_offset: gate_offset + o.shape[1]], activation)).view(n, heads, value_dim)
+        y = (u * torch.rsqrt((u * u).mean(-1, keepdim=True) + eps)).reshape(n, -1)
+        w = weight.float() if weight is not None else torch.ones(1)
+        out.copy_((y * (w.repeat(heads) if w.shape[0] == value_dim and heads > 1 else w)).to(out.dtype))
+
+    def ssd_scan(self, xbc, heads, groups, state_dim, value_dim, dt, dt_offset, dt_bias, a_log, skip, state, meta, out) -> None:
+        H, G, N, P = heads, groups, state_dim, value_dim
+        out.zero_()
+        for sg in meta.segments:
+            r = slice(sg.row0, sg.row0 + sg.n)
+            v = xbc[r].double()
+            x = v[:, :H * P].reshape(-1, H, P)
+            B = v[:, H * P: H * P + G * N].reshape(-1, G, N).repeat_interleave(H // G, 1)
+            C = v[:, H * P + G * N:].reshape(-1, G, N).repeat_interleave(H // G, 1)
+            d = torch.nn.functional.softplus(dt[r, dt_offset: dt_offset + H].double() + dt_bias.double(), threshold=200.0)
+            a = torch.exp(-torch.exp(a_log.double()) * d)
+            M = state[sg.state_slot].double()
+            for t in range(sg.n):
+                M = a[t][:, None, None] * M + (d[t][:, None] * B[t])[:, :, None] * x[t][:, None, :]
+                out[sg.row0 + t] = (torch.einsum("hnp,hn->hp", M, C[t]) + skip.double()[:, None] * x[t]).reshape(-1).float()
+            state[sg.state_slot] = M.float()
+
+    def route_by_scores(self, logits, num_experts, top, groups, keep_groups, renormalize, meta, weights, align=1,
+                        scoring="softmax", correction=None, group_top=1, sum_eps=0.0, scale=1.0):
+        z = logits[:, :num_experts].float()
+        s = torch.softmax(z, -1) if scoring == "softmax" else torch.sigmoid(z)
+        c = s if correction is None else s + correction.float()
+        per = num_experts // groups
+        gs = torch.sort(c.view(-1, groups, per), dim=-1, descending=True).values[..., :group_top].sum(-1)
+        best = torch.sort(gs, dim=-1, descending=True, stable=True).indices[:, :keep_groups]
+        allowed = torch.zeros_like(gs, dtype=torch.bool).scatter_(1, best, True).repeat_interleave(per, 1)
+        order = torch.sort(torch.where(allowed, c, torch.full_like(c, -float("inf"))), dim=-1, descending=True, stable=True).indices[:, :top]
+        w = torch.gather(s, 1, order)
+        if renormalize:
+            w = w / (w.sum(-1, keepdim=True) + sum_eps)
+        weights.copy_(w * scale)
+        return order, meta.seq_row >= 0
