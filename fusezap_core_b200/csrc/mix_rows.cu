@@ -174,12 +174,20 @@ add_rmsnorm_groups_vec_kernel(float* __restrict__ x, const float* __restrict__ d
 }
 
 // ------------------------------------------------------------------------------------------------ short convolution
-// seg: (first row, rows, first position, state slot) per portion. state: (slots, taps - 1, C) float32, oldest first.
-template <typename T>
+// seg: (first row, rows, first position, state slot) per portion. state: (slots, taps - 1, C) float32, oldest first. The
+// inputs are C neighbouring columns of rows of ld values of TI (TI = T and ld = C, or a range of a wider float32 product).
+// `single`: every portion of the step is one token; the thread that owns a channel then also moves its state on.
+template <typename TI>
+__device__ __forceinline__ void conv_state_single(float* __restrict__ st, const TI* __restrict__ own, int C, int taps) {
+  for (int m = 0; m + 1 < taps - 1; ++m) st[(size_t)m * C] = st[(size_t)(m + 1) * C];
+  st[(size_t)(taps - 2) * C] = Cvt<TI>::to_f(*own);
+}
+
+template <typename TI, typename T>
 __global__ void __launch_bounds__(256)
-short_conv_kernel(const T* __restrict__ h, const T* __restrict__ w, const float* __restrict__ state,
+short_conv_kernel(const TI* __restrict__ h, int ld, const T* __restrict__ w, float* __restrict__ state,
                   const int* __restrict__ seg, const int* __restrict__ seq_row, T* __restrict__ out, int C, int taps,
-                  int residual, int act, const float* __restrict__ bias) {
+                  int residual, int act, const float* __restrict__ bias, int single) {
   fz_grid_launch_dependents();
   fz_grid_wait();
   const int n = blockIdx.x;
@@ -193,21 +201,22 @@ short_conv_kernel(const T* __restrict__ h, const T* __restrict__ w, const float*
   }
   const int row0 = seg[4 * s], slot = seg[4 * s + 3];
   const int i = n - row0;
-  const float* st = state != nullptr && slot >= 0 ? state + (size_t)slot * (taps - 1) * C : nullptr;
+  float* st = state != nullptr && slot >= 0 ? state + (size_t)slot * (taps - 1) * C : nullptr;
   {
     float acc = 0.f;
     for (int j = 0; j < taps; ++j) {
       const int k = i - (taps - 1) + j;
       float v = 0.f;
-      if (k >= 0) v = Cvt<T>::to_f(h[(size_t)(row0 + k) * C + c]);
+      if (k >= 0) v = Cvt<TI>::to_f(h[(size_t)(row0 + k) * ld + c]);
       else if (st != nullptr) v = st[(size_t)(taps - 1 + k) * C + c];
       acc = fmaf(Cvt<T>::to_f(w[(size_t)c * taps + j]), v, acc);
     }
     if (bias != nullptr) acc += bias[c];
-    if (residual) acc += Cvt<T>::to_f(h[(size_t)n * C + c]);
+    if (residual) acc += Cvt<TI>::to_f(h[(size_t)n * ld + c]);
     if (act) acc = acc * (1.0f / (1.0f + expf(-acc)));      // silu of the 32-bit sum
     orow[c] = Cvt<T>::from_f(acc);
   }
+  if (single && st != nullptr && taps > 1) conv_state_single(st + c, h + (size_t)n * ld + c, C, taps);
 }
 
 // The same with eight channels per thread (16-byte loads of the inputs, the state and the output) for C % 8 == 0.
@@ -235,11 +244,11 @@ __device__ __forceinline__ void st8(__nv_bfloat16* p, const float* v) {
 
 // TAPS > 0: the tap count is known at compile time and the thread's 8 x TAPS weights (contiguous in the (C, taps)
 // matrix) come in as TAPS 16-byte groups (bfloat16) instead of one by one; TAPS == 0: any tap count.
-template <typename T, int TAPS>
+template <typename TI, typename T, int TAPS>
 __global__ void __launch_bounds__(128)
-short_conv_vec_kernel(const T* __restrict__ h, const T* __restrict__ w, const float* __restrict__ state,
+short_conv_vec_kernel(const TI* __restrict__ h, int ld, const T* __restrict__ w, float* __restrict__ state,
                       const int* __restrict__ seg, const int* __restrict__ seq_row, T* __restrict__ out, int C, int taps,
-                      int residual, int act, const float* __restrict__ bias) {
+                      int residual, int act, const float* __restrict__ bias, int single) {
   fz_grid_launch_dependents();
   fz_grid_wait();
   const int n = blockIdx.x;
@@ -250,7 +259,7 @@ short_conv_vec_kernel(const T* __restrict__ h, const T* __restrict__ w, const fl
   if (s >= 0) {
     const int row0 = seg[4 * s], slot = seg[4 * s + 3];
     const int i = n - row0;
-    const float* st = state != nullptr && slot >= 0 ? state + (size_t)slot * (taps - 1) * C : nullptr;
+    float* st = state != nullptr && slot >= 0 ? state + (size_t)slot * (taps - 1) * C : nullptr;
     if constexpr (TAPS > 0) {
       float wv[8 * TAPS];                  // wv[e * TAPS + j]: tap j of channel c0 + e
 #pragma unroll
@@ -259,7 +268,7 @@ short_conv_vec_kernel(const T* __restrict__ h, const T* __restrict__ w, const fl
       for (int j = 0; j < TAPS; ++j) {
         const int k = i - (TAPS - 1) + j;
         float v[8];
-        if (k >= 0) ld8(h + (size_t)(row0 + k) * C + c0, v);
+        if (k >= 0) ld8(h + (size_t)(row0 + k) * ld + c0, v);
         else if (st != nullptr) ld8(st + (size_t)(TAPS - 1 + k) * C + c0, v);
         else continue;
 #pragma unroll
@@ -269,7 +278,7 @@ short_conv_vec_kernel(const T* __restrict__ h, const T* __restrict__ w, const fl
       for (int j = 0; j < taps; ++j) {
         const int k = i - (taps - 1) + j;
         float v[8];
-        if (k >= 0) ld8(h + (size_t)(row0 + k) * C + c0, v);
+        if (k >= 0) ld8(h + (size_t)(row0 + k) * ld + c0, v);
         else if (st != nullptr) ld8(st + (size_t)(taps - 1 + k) * C + c0, v);
         else continue;
 #pragma unroll
@@ -284,13 +293,22 @@ short_conv_vec_kernel(const T* __restrict__ h, const T* __restrict__ w, const fl
     }
     if (residual) {
       float v[8];
-      ld8(h + (size_t)n * C + c0, v);
+      ld8(h + (size_t)n * ld + c0, v);
 #pragma unroll
       for (int e = 0; e < 8; ++e) acc[e] += v[e];
     }
     if (act) {
 #pragma unroll
       for (int e = 0; e < 8; ++e) acc[e] = acc[e] * (1.0f / (1.0f + expf(-acc[e])));      // silu of the 32-bit sum
+    }
+    if (single && st != nullptr && taps > 1) {
+      float v[8];
+      for (int m = 0; m + 1 < taps - 1; ++m) {
+        ld8(st + (size_t)(m + 1) * C + c0, v);
+        st8(st + (size_t)m * C + c0, v);
+      }
+      ld8(h + (size_t)n * ld + c0, v);
+      st8(st + (size_t)(taps - 2) * C + c0, v);
     }
   }
   st8(out + (size_t)n * C + c0, acc);
@@ -300,9 +318,9 @@ short_conv_vec_kernel(const T* __restrict__ h, const T* __restrict__ w, const fl
 // (the portion's own rows, and what is left of the old state when the portion is shorter than taps - 1). A thread owns
 // one channel of one portion, reads all it needs and then writes. grid (portions, channel blocks).
 constexpr int MAX_TAPS = 32;
-template <typename T>
+template <typename TI>
 __global__ void __launch_bounds__(256)
-short_conv_state_kernel(const T* __restrict__ h, float* __restrict__ state, const int* __restrict__ seg, int C, int taps) {
+short_conv_state_kernel(const TI* __restrict__ h, int ld, float* __restrict__ state, const int* __restrict__ seg, int C, int taps) {
   fz_grid_launch_dependents();
   fz_grid_wait();
   const int s = blockIdx.x;
@@ -315,7 +333,7 @@ short_conv_state_kernel(const T* __restrict__ h, float* __restrict__ state, cons
   for (int m = 0; m < MAX_TAPS - 1; ++m) {
     if (m < taps - 1) {
       const int k = cnt - (taps - 1) + m;
-      keep[m] = k >= 0 ? Cvt<T>::to_f(h[(size_t)(row0 + k) * C + c]) : st[(size_t)(taps - 1 + k) * C + c];
+      keep[m] = k >= 0 ? Cvt<TI>::to_f(h[(size_t)(row0 + k) * ld + c]) : st[(size_t)(taps - 1 + k) * C + c];
     }
   }
 #pragma unroll
@@ -454,18 +472,32 @@ rotate_heads_kernel(const T* __restrict__ q, int W, int off, const float* __rest
     out[((size_t)n * H + hh) * Wo + out_off + d] = Cvt<T>::from_f(v);
   }
 }
-template <typename T>
-void launch_conv_vec(dim3 grid, cudaStream_t stream, const T* h, const T* w, const float* state, const int* seg,
-                     const int* seq_row, T* out, int C, int taps, int residual, int act, const float* bias) {
-  const bool w_ok = ((uintptr_t)w & 15) == 0;       // the grouped weight loads want 16-byte aligned rows of 8 x taps values
-#define FZ_CV(N) fz_launch(short_conv_vec_kernel<T, N>, grid, dim3(128), 0, stream, h, w, state, seg, seq_row, out, C, taps, residual, act, bias)
-  if (w_ok && taps == 2) FZ_CV(2);
-  else if (w_ok && taps == 3) FZ_CV(3);
-  else if (w_ok && taps == 4) FZ_CV(4);
-  else if (w_ok && taps == 5) FZ_CV(5);
-  else if (w_ok && taps == 8) FZ_CV(8);
-  else FZ_CV(0);
+template <typename TI, typename T>
+int launch_conv(const TI* h, int ld, const T* w, float* state, const int* seg, const int* seq_row, T* out, int N, int n_seg,
+                int C, int taps, int residual, int act, const float* bias, int single, cudaStream_t stream) {
+  const bool vec = C % 8 == 0 && ((size_t)ld * sizeof(TI)) % 16 == 0 &&
+                   (((uintptr_t)h | (uintptr_t)out | (uintptr_t)state | (uintptr_t)bias) & 15) == 0;
+  if (vec) {
+    const dim3 grid(N, (C / 8 + 127) / 128);
+    const bool w_ok = ((uintptr_t)w & 15) == 0;       // the grouped weight loads want 16-byte aligned rows of 8 x taps values
+#define FZ_CV(K) fz_launch(short_conv_vec_kernel<TI, T, K>, grid, dim3(128), 0, stream, h, ld, w, state, seg, seq_row, out, C, taps, residual, act, bias, single)
+    if (w_ok && taps == 2) FZ_CV(2);
+    else if (w_ok && taps == 3) FZ_CV(3);
+    else if (w_ok && taps == 4) FZ_CV(4);
+    else if (w_ok && taps == 5) FZ_CV(5);
+    else if (w_ok && taps == 8) FZ_CV(8);
+    else FZ_CV(0);
 #undef FZ_CV
+  } else {
+    fz_launch(short_conv_kernel<TI, T>, dim3(N, (C + 255) / 256), dim3(256), 0, stream, h, ld, w, state, seg, seq_row, out, C, taps,
+              residual, act, bias, single);
+  }
+  FZ_LAUNCH_CHECK();
+  if (taps > 1 && state != nullptr && n_seg > 0 && !single) {
+    fz_launch(short_conv_state_kernel<TI>, dim3(n_seg, (C + 255) / 256), dim3(256), 0, stream, h, ld, state, seg, C, taps);
+    FZ_LAUNCH_CHECK();
+  }
+  return FZ_OK;
 }
 }  // namespace
 
@@ -492,30 +524,19 @@ FZ_API int fz_add_rmsnorm_groups(float* x, const float* delta, const void* w, in
   return FZ_BAD_DTYPE;
 }
 
-FZ_API int fz_short_conv(const void* h, const void* w, float* state, const int* seg, const int* seq_row, void* out,
-                         int dtype, int N, int n_seg, int C, int taps, int residual, int act, const float* bias,
-                         cudaStream_t stream) {
+// in_dtype: the type of the inputs, rows of ld values of which C from column `off` on are read (dtype itself, or float32).
+// single: every portion of the step is one token (the state then moves on in the same launch).
+FZ_API int fz_short_conv(const void* h, int in_dtype, int ld, int off, const void* w, float* state, const int* seg,
+                         const int* seq_row, void* out, int dtype, int N, int n_seg, int C, int taps, int residual, int act,
+                         const float* bias, int single, cudaStream_t stream) {
   if (N <= 0) return FZ_OK;
-  if (taps < 1 || taps > MAX_TAPS) return FZ_BAD_SHAPE;
-  const bool vec = C % 8 == 0 && (((uintptr_t)h | (uintptr_t)out | (uintptr_t)state | (uintptr_t)bias) & 15) == 0;
-  const dim3 vgrid(N, (C / 8 + 127) / 128);
-  if (dtype == FZ_F32) {
-    if (vec) launch_conv_vec<float>(vgrid, stream, (const float*)h, (const float*)w, (const float*)state, seg, seq_row, (float*)out, C, taps, residual, act, bias);
-    else fz_launch(short_conv_kernel<float>, dim3(N, (C + 255) / 256), dim3(256), 0, stream, (const float*)h, (const float*)w, (const float*)state, seg, seq_row, (float*)out, C, taps, residual, act, bias);
-    FZ_LAUNCH_CHECK();
-    if (taps > 1 && state != nullptr && n_seg > 0)
-      fz_launch(short_conv_state_kernel<float>, dim3(n_seg, (C + 255) / 256), dim3(256), 0, stream, (const float*)h, state, seg, C, taps);
-  } else if (dtype == FZ_BF16) {
-    if (vec) launch_conv_vec<__nv_bfloat16>(vgrid, stream, (const __nv_bfloat16*)h, (const __nv_bfloat16*)w, (const float*)state, seg, seq_row, (__nv_bfloat16*)out, C, taps, residual, act, bias);
-    else fz_launch(short_conv_kernel<__nv_bfloat16>, dim3(N, (C + 255) / 256), dim3(256), 0, stream, (const __nv_bfloat16*)h, (const __nv_bfloat16*)w, (const float*)state, seg, seq_row, (__nv_bfloat16*)out, C, taps, residual, act, bias);
-    FZ_LAUNCH_CHECK();
-    if (taps > 1 && state != nullptr && n_seg > 0)
-      fz_launch(short_conv_state_kernel<__nv_bfloat16>, dim3(n_seg, (C + 255) / 256), dim3(256), 0, stream, (const __nv_bfloat16*)h, state, seg, C, taps);
-  } else {
-    return FZ_BAD_DTYPE;
-  }
-  FZ_LAUNCH_CHECK();
-  return FZ_OK;
+  if (taps < 1 || taps > MAX_TAPS || off < 0 || off + C > ld) return FZ_BAD_SHAPE;
+#define FZ_CONV(TI, T) return launch_conv<TI, T>((const TI*)h + off, ld, (const T*)w, state, seg, seq_row, (T*)out, N, n_seg, C, taps, residual, act, bias, single, stream)
+  if (in_dtype == FZ_F32 && dtype == FZ_F32) FZ_CONV(float, float);
+  if (in_dtype == FZ_BF16 && dtype == FZ_BF16) FZ_CONV(__nv_bfloat16, __nv_bfloat16);
+  if (in_dtype == FZ_F32 && dtype == FZ_BF16) FZ_CONV(float, __nv_bfloat16);
+#undef FZ_CONV
+  return FZ_BAD_DTYPE;
 }
 
 FZ_API int fz_gated_sum(const float* a, const float* ga, const float* f, const float* gf, float* out, int N, int D,

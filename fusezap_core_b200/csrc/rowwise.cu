@@ -11,23 +11,28 @@
 // ------------------------------------------------------------------------------------------------ embedding
 // src (may be null): src[n] >= 0 takes the row's token from prev_ids[src[n]] (the ids the previous step chose, still on
 // the device) instead of tokens[n]. scale: every value is multiplied by it in float32 (1 for the models that do not
-// scale their embeddings: the product is then exact).
+// scale their embeddings: the product is then exact). copy (may be null): receives the same values as x.
 template <typename T>
 __global__ void embed_kernel(const T* __restrict__ table, const int* __restrict__ tokens, const int* __restrict__ src,
-                             const int* __restrict__ prev_ids, float* __restrict__ x, int D, int V, float scale, int* err) {
+                             const int* __restrict__ prev_ids, float* __restrict__ x, float* __restrict__ copy, int D, int V,
+                             float scale, int* err) {
   fz_grid_launch_dependents();
   fz_grid_wait();
   const int n = blockIdx.x;
   int tok = tokens[n];
   if (src != nullptr && src[n] >= 0) tok = prev_ids[src[n]];
   float* xr = x + (size_t)n * D;
+  float* cr = copy != nullptr ? copy + (size_t)n * D : nullptr;
   if (tok < 0 || tok >= V) {
     if (threadIdx.x == 0) atomicOr(err, FZ_ERR_TOKEN_RANGE);
-    for (int d = threadIdx.x; d < D; d += blockDim.x) xr[d] = 0.f;
+    for (int d = threadIdx.x; d < D; d += blockDim.x) {
+      xr[d] = 0.f;
+      if (cr) cr[d] = 0.f;
+    }
     return;
   }
   const T* tr = table + (size_t)tok * D;
-  if (D % 8 == 0 && ((((uintptr_t)tr) | ((uintptr_t)xr)) & 15) == 0) {
+  if (D % 8 == 0 && ((((uintptr_t)tr) | ((uintptr_t)xr) | ((uintptr_t)cr)) & 15) == 0) {
     // 16 bytes of the table row per thread and turn (8 bf16 or 4 float32 values): one round of loads for a row of 4096
     constexpr int PER = 16 / (int)sizeof(T);
     for (int d = threadIdx.x * PER; d < D; d += blockDim.x * PER) {
@@ -37,20 +42,27 @@ __global__ void embed_kernel(const T* __restrict__ table, const int* __restrict_
 #pragma unroll
       for (int i = 0; i < PER; ++i) f[i] = __fmul_rn(Cvt<T>::to_f(v[i]), scale);
 #pragma unroll
-      for (int i = 0; i < PER; i += 4) *(float4*)(xr + d + i) = make_float4(f[i], f[i + 1], f[i + 2], f[i + 3]);
+      for (int i = 0; i < PER; i += 4) {
+        *(float4*)(xr + d + i) = make_float4(f[i], f[i + 1], f[i + 2], f[i + 3]);
+        if (cr) *(float4*)(cr + d + i) = make_float4(f[i], f[i + 1], f[i + 2], f[i + 3]);
+      }
     }
     return;
   }
-  for (int d = threadIdx.x; d < D; d += blockDim.x) xr[d] = __fmul_rn(Cvt<T>::to_f(tr[d]), scale);
+  for (int d = threadIdx.x; d < D; d += blockDim.x) {
+    const float v = __fmul_rn(Cvt<T>::to_f(tr[d]), scale);
+    xr[d] = v;
+    if (cr) cr[d] = v;
+  }
 }
 
 FZ_API int fz_embed(const void* table, int table_dtype, const int* tokens, const int* src, const int* prev_ids, float* x,
-                    int N, int D, int V, float scale, int* err, cudaStream_t stream) {
+                    float* copy, int N, int D, int V, float scale, int* err, cudaStream_t stream) {
   if (N <= 0) return FZ_OK;
   if (table_dtype == FZ_F32)
-    fz_launch(embed_kernel<float>, dim3(N), dim3(512), 0, stream, (const float*)table, tokens, src, prev_ids, x, D, V, scale, err);
+    fz_launch(embed_kernel<float>, dim3(N), dim3(512), 0, stream, (const float*)table, tokens, src, prev_ids, x, copy, D, V, scale, err);
   else if (table_dtype == FZ_BF16)
-    fz_launch(embed_kernel<__nv_bfloat16>, dim3(N), dim3(512), 0, stream, (const __nv_bfloat16*)table, tokens, src, prev_ids, x, D, V, scale, err);
+    fz_launch(embed_kernel<__nv_bfloat16>, dim3(N), dim3(512), 0, stream, (const __nv_bfloat16*)table, tokens, src, prev_ids, x, copy, D, V, scale, err);
   else
     return FZ_BAD_DTYPE;
   FZ_LAUNCH_CHECK();
@@ -220,6 +232,158 @@ FZ_API int fz_add_rmsnorm(float* x, const float* delta, const void* w, int w_dty
   if (w_dtype == FZ_BF16 && h_dtype == FZ_BF16) FZ_NORM(__nv_bfloat16, __nv_bfloat16);
   if (w_dtype == FZ_BF16 && h_dtype == FZ_F32) FZ_NORM(__nv_bfloat16, float);
 #undef FZ_NORM
+  return FZ_BAD_DTYPE;
+}
+
+// ------------------------------------------------------------------------------------------------ add + LayerNorm
+// rows == nullptr: x[n] = (x[n] + delta[n]) + extra[n] (each if given, in place), h[n] = w * (x[n] - m) / sqrt(mean((x[n] -
+// m)^2) + eps) with m the row's mean, one block per row n. rows != nullptr: block r reads row rows[r] (x + delta, x
+// untouched) and writes h[r]; rows[r] < 0 gives zeros. The squares are taken of the deviations, after the mean is known.
+template <typename TH>
+__global__ void __launch_bounds__(256)
+add_layernorm_kernel(float* __restrict__ x, const float* __restrict__ delta, const float* __restrict__ extra,
+                     const float* __restrict__ w, TH* __restrict__ h, const int* __restrict__ rows, int n_src, int D, float eps,
+                     int* err) {
+  fz_grid_launch_dependents();
+  fz_grid_wait();
+  __shared__ float scratch[32];
+  const int r = blockIdx.x;
+  int src = r;
+  TH* hr = h + (size_t)r * D;
+  if (rows != nullptr) {
+    src = rows[r];
+    if (src < 0 || src >= n_src) {
+      if (src >= n_src && threadIdx.x == 0) atomicOr(err, FZ_ERR_ROW_RANGE);
+      for (int d = threadIdx.x; d < D; d += blockDim.x) hr[d] = Cvt<TH>::from_f(0.f);
+      return;
+    }
+  }
+  float* xr = x + (size_t)src * D;
+  const float* dr = delta ? delta + (size_t)src * D : nullptr;
+  const float* er = extra ? extra + (size_t)src * D : nullptr;
+  const bool write_x = rows == nullptr && (dr != nullptr || er != nullptr);
+  auto value = [&](int d) {
+    float v = xr[d];
+    if (dr) v += dr[d];
+    if (er) v += er[d];
+    return v;
+  };
+  float sum = 0.f;
+  for (int d = threadIdx.x; d < D; d += blockDim.x) {
+    const float v = value(d);
+    if (write_x) xr[d] = v;
+    sum += v;
+  }
+  const float mean = block_sum(sum, scratch) * (1.0f / (float)D);
+  float ss = 0.f;
+  for (int d = threadIdx.x; d < D; d += blockDim.x) {      // (a thread reads back what it wrote itself)
+    const float v = (write_x ? xr[d] : value(d)) - mean;
+    ss = fmaf(v, v, ss);
+  }
+  const float scale = 1.0f / sqrtf(block_sum(ss, scratch) * (1.0f / (float)D) + eps);
+  for (int d = threadIdx.x; d < D; d += blockDim.x)
+    hr[d] = Cvt<TH>::from_f(w[d] * (((write_x ? xr[d] : value(d)) - mean) * scale));
+}
+
+// The same for D % 4 == 0 and D <= 4 * NT * VPT: a thread keeps its VPT float4 groups of the row in registers, so the row
+// is read once; the weights and the row's index, which no kernel of the step writes, are read ahead of the wait.
+template <typename TH, int NT, int VPT>
+__global__ void __launch_bounds__(NT)
+add_layernorm_vec_kernel(float* __restrict__ x, const float* __restrict__ delta, const float* __restrict__ extra,
+                         const float* __restrict__ w, TH* __restrict__ h, const int* __restrict__ rows, int n_src, int D,
+                         float eps, int* err) {
+  fz_grid_launch_dependents();
+  const int r = blockIdx.x;
+  const int D4 = D >> 2;
+  float4 g[VPT];
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = threadIdx.x + i * NT;
+    g[i] = c < D4 ? load4f(w + 4 * c) : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  int src = r;
+  if (rows != nullptr) src = rows[r];
+  fz_grid_wait();
+  __shared__ float scratch[32];
+  TH* hr = h + (size_t)r * D;
+  if (src < 0 || src >= n_src) {
+    if (src >= n_src && threadIdx.x == 0) atomicOr(err, FZ_ERR_ROW_RANGE);
+    for (int d = threadIdx.x; d < D; d += blockDim.x) hr[d] = Cvt<TH>::from_f(0.f);
+    return;
+  }
+  float4* xr = (float4*)(x + (size_t)src * D);
+  const float4* add[2] = {delta ? (const float4*)(delta + (size_t)src * D) : nullptr,
+                          extra ? (const float4*)(extra + (size_t)src * D) : nullptr};
+  float4 v[VPT];
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = threadIdx.x + i * NT;
+    v[i] = c < D4 ? xr[c] : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+#pragma unroll
+  for (int k = 0; k < 2; ++k) {
+    if (add[k] == nullptr) continue;
+    float4 dv[VPT];
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int c = threadIdx.x + i * NT;
+      dv[i] = c < D4 ? add[k][c] : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) { v[i].x += dv[i].x; v[i].y += dv[i].y; v[i].z += dv[i].z; v[i].w += dv[i].w; }
+  }
+  float sum = 0.f;
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) sum += (v[i].x + v[i].y) + (v[i].z + v[i].w);
+  if (rows == nullptr && (add[0] != nullptr || add[1] != nullptr)) {
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int c = threadIdx.x + i * NT;
+      if (c < D4) xr[c] = v[i];
+    }
+  }
+  const float mean = block_sum(sum, scratch) * (1.0f / (float)D);
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    if (threadIdx.x + i * NT < D4) {
+      v[i].x -= mean; v[i].y -= mean; v[i].z -= mean; v[i].w -= mean;
+      ss = fmaf(v[i].x, v[i].x, ss); ss = fmaf(v[i].y, v[i].y, ss); ss = fmaf(v[i].z, v[i].z, ss); ss = fmaf(v[i].w, v[i].w, ss);
+    }
+  }
+  const float scale = 1.0f / sqrtf(block_sum(ss, scratch) * (1.0f / (float)D) + eps);
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = threadIdx.x + i * NT;
+    if (c < D4)
+      store4f(hr + 4 * c, g[i].x * (v[i].x * scale), g[i].y * (v[i].y * scale), g[i].z * (v[i].z * scale), g[i].w * (v[i].w * scale));
+  }
+}
+
+template <typename TH>
+static int launch_layernorm(float* x, const float* delta, const float* extra, const float* w, void* h, const int* rows,
+                            int n_out, int n_src, int D, float eps, int* err, cudaStream_t stream) {
+  const bool vec = D % 4 == 0 && D <= 4 * 512 * 8 &&
+                   (((uintptr_t)x | (uintptr_t)delta | (uintptr_t)extra | (uintptr_t)w | (uintptr_t)h) & 15) == 0;
+#define FZ_LN(NT, V) fz_launch(add_layernorm_vec_kernel<TH, NT, V>, dim3(n_out), dim3(NT), 0, stream, x, delta, extra, w, (TH*)h, rows, n_src, D, eps, err)
+  if (!vec) fz_launch(add_layernorm_kernel<TH>, dim3(n_out), dim3(256), 0, stream, x, delta, extra, w, (TH*)h, rows, n_src, D, eps, err);
+  else if (D <= 4 * 128) FZ_LN(128, 1);
+  else if (D <= 4 * 256) FZ_LN(256, 1);
+  else if (D <= 4 * 512) FZ_LN(512, 1);
+  else if (D <= 8 * 512) FZ_LN(512, 2);
+  else if (D <= 16 * 512) FZ_LN(512, 4);
+  else FZ_LN(512, 8);
+#undef FZ_LN
+  FZ_LAUNCH_CHECK();
+  return FZ_OK;
+}
+
+FZ_API int fz_add_layernorm(float* x, const float* delta, const float* extra, const float* w, void* h, int h_dtype,
+                            const int* rows, int n_out, int n_src, int D, float eps, int* err, cudaStream_t stream) {
+  if (n_out <= 0) return FZ_OK;
+  if (D <= 0 || (rows != nullptr && extra != nullptr)) return FZ_BAD_SHAPE;
+  if (h_dtype == FZ_F32) return launch_layernorm<float>(x, delta, extra, w, h, rows, n_out, n_src, D, eps, err, stream);
+  if (h_dtype == FZ_BF16) return launch_layernorm<__nv_bfloat16>(x, delta, extra, w, h, rows, n_out, n_src, D, eps, err, stream);
   return FZ_BAD_DTYPE;
 }
 

@@ -6,6 +6,7 @@
 // portion's tokens in order from the state in the request's slot and leaves the state there. Nothing depends on which
 // other portions share the step.
 #include "common.cuh"
+#include "scan.cuh"
 #include <math.h>
 
 namespace {
@@ -483,88 +484,7 @@ sink_attention_merge_kernel(const AttnArgs a) {
   pair_finish<T, DPL>(a, n, head, m, l, acc);
 }
 
-// ------------------------------------------------------------------------------------------------ recurrent scans
-// The state of a head is a key_dim x value_dim matrix S. A thread owns DPT = 8 consecutive rows of DC = 4 neighbouring
-// columns, as sixteen packed pairs: the recurrence runs on packed float32 x 2 instructions (each half rounds as the scalar
-// instruction does), every key and query value read from shared memory serves four columns, and a head is spread over
-// value_dim / 4 x R threads (the kernels are bound by the instructions they issue per token, not by memory). The R lanes that share the columns (R a power of two, R * 8 >= key_dim; lane = r * (32 / R)
-// + group, so that neighbouring lanes read one address of shared memory) add their partial dot products with shuffles.
-// State layout in memory: (slots, heads, value_dim, R * 8), so a thread's 8 values of a column are contiguous and a
-// column's run is read in 32-byte pieces; rows beyond key_dim stay zero. A block covers (blockDim / R) * 4 columns of one
-// head of one portion and walks the portion's tokens in chunks, staged in shared memory by all threads.
-constexpr int DPT = 8;
-constexpr int DC = 4;                       // value columns per thread: two packed pairs
-constexpr int SCAN_MAX_THREADS = 512;
-// While a chunk of tokens is computed, the inputs of the next one travel from global into a raw staging area of shared
-// memory (`cp.async`, four bytes each); after the chunk they are turned into what the recurrence reads (rotated or unit
-// vectors, decays, gates) in a second area. tch: tokens per chunk (16, or 8 where shared memory would not hold 16).
-
-// Sum over the R lanes that hold the rows of one column group: they are 32 / R lanes apart.
-template <int R>
-__device__ __forceinline__ float lanes_sum(float v) {
-#pragma unroll
-  for (int o = 16; o >= 32 / R; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-  return v;
-}
-
-// Which column group (of the block) and which 16 rows a thread owns.
-template <int R>
-__device__ __forceinline__ void scan_place(int& group, int& r) {
-  constexpr int per_warp = 32 / R;
-  const int lane = threadIdx.x & 31;
-  r = lane / per_warp;
-  group = (threadIdx.x >> 5) * per_warp + lane % per_warp;
-}
-
-// The thread's 8 rows of two neighbouring columns (dkp floats apart), as pairs (column, column + 1); the second column
-// is read and written only where it exists.
-__device__ __forceinline__ void load_state(const float* __restrict__ p, int dkp, bool first, bool second, float2* S) {
-#pragma unroll
-  for (int i = 0; i < DPT; i += 4) {
-    const float4 a = first ? *(const float4*)(p + i) : make_float4(0.f, 0.f, 0.f, 0.f);
-    const float4 b = second ? *(const float4*)(p + dkp + i) : make_float4(0.f, 0.f, 0.f, 0.f);
-    S[i] = make_float2(a.x, b.x); S[i + 1] = make_float2(a.y, b.y); S[i + 2] = make_float2(a.z, b.z); S[i + 3] = make_float2(a.w, b.w);
-  }
-}
-__device__ __forceinline__ void store_state(float* __restrict__ p, int dkp, bool first, bool second, const float2* S) {
-#pragma unroll
-  for (int i = 0; i < DPT; i += 4) {
-    if (first) *(float4*)(p + i) = make_float4(S[i].x, S[i + 1].x, S[i + 2].x, S[i + 3].x);
-    if (second) *(float4*)(p + dkp + i) = make_float4(S[i].y, S[i + 1].y, S[i + 2].y, S[i + 3].y);
-  }
-}
-__device__ __forceinline__ void load8(const float* p, float* v) {       // 8 floats from shared memory, 32-byte aligned
-  const float4 a = *(const float4*)p, b = *(const float4*)(p + 4);
-  v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
-}
-__device__ __forceinline__ float2 both(float v) { return make_float2(v, v); }
-
-__device__ __forceinline__ void cp_async16(void* dst, const void* src) {
-  const unsigned d = (unsigned)__cvta_generic_to_shared(dst);
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(d), "l"(src) : "memory");
-}
-__device__ __forceinline__ bool aligned16(const void* p) { return ((uintptr_t)p & 15) == 0; }
-__device__ __forceinline__ void cp_async4(void* dst, const void* src) {
-  const unsigned d = (unsigned)__cvta_generic_to_shared(dst);
-  asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(d), "l"(src) : "memory");
-}
-// Unit i of `vec` four-byte words (1 or 4) from src to dst.
-__device__ __forceinline__ void cp_words(float* dst, const float* src, int i, int vec) {
-  if (vec == 4) cp_async16(dst + 4 * i, src + 4 * i);
-  else cp_async4(dst + i, src + i);
-}
-__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-__device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group 0;" ::: "memory"); }
-
-// Unit i of a run of values of T from global to shared: a four-byte copy in flight (T is float, or a pair of 16-bit
-// values where `words` says that source, destination and length allow it), else one value copied at once.
-template <typename T>
-__device__ __forceinline__ void stage_unit(T* dst, const T* src, int i, bool words) {
-  if (sizeof(T) == 4) cp_async4(dst + i, src + i);
-  else if (words) cp_async4(dst + 2 * i, src + 2 * i);
-  else dst[i] = src[i];
-}
-
+// ------------------------------------------------------------------------------------------------ recurrent scans (see scan.cuh)
 // S = decay * S + k' v^T; o = S^T q'. proj rows: [q heads | k heads | v heads | ...], ld floats apart.
 template <int R>
 __global__ void __launch_bounds__(SCAN_MAX_THREADS)
@@ -1022,74 +942,181 @@ head_norm_gate_kernel(const float* __restrict__ o, int H, int dv, const float* _
   }
 }
 
+// The gate before the norm: u = o * act(gate), out = u / sqrt(mean_c u^2 + eps) * w, a block per (row, part of dv values).
+// Vectorised where dv is a multiple of four, at most 4 * VPT values per thread, and everything is 16-byte aligned: a thread
+// keeps its values in registers; else every value is computed twice.
+__device__ __forceinline__ float gated(float o, float z, int act) {
+  const float sg = 1.0f / (1.0f + expf(-z));
+  return o * (act == 2 ? z * sg : sg);
+}
+__device__ __forceinline__ void store4(float* d, float4 v) { *(float4*)d = v; }
+__device__ __forceinline__ void store4(__nv_bfloat16* d, float4 v) {
+  const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+  *(uint2*)d = make_uint2(*(const uint32_t*)&lo, *(const uint32_t*)&hi);
+}
+template <typename TO, int VPT>
+__global__ void __launch_bounds__(512)
+gate_norm_vec_kernel(const float* __restrict__ o, int H, int dv, const float* __restrict__ w, int w_per_head, float eps,
+                     const float* __restrict__ gate, int ldg, int goff, int act, const int* __restrict__ seq_row,
+                     TO* __restrict__ out) {
+  fz_grid_launch_dependents();
+  const int n = blockIdx.x, h = blockIdx.y, NT = blockDim.x;
+  const int D4 = dv >> 2;
+  const bool pad = seq_row[n] < 0;
+  float4 g[VPT];
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {      // the weights depend on no kernel of the step
+    const int c = threadIdx.x + i * NT;
+    g[i] = w != nullptr && c < D4 ? *(const float4*)(w + (w_per_head ? (size_t)h * dv : 0) + 4 * c) : make_float4(1.f, 1.f, 1.f, 1.f);
+  }
+  fz_grid_wait();
+  __shared__ float scratch[32];
+  const float4* x = (const float4*)(o + ((size_t)n * H + h) * dv);
+  const float4* z = (const float4*)(gate + (size_t)n * ldg + goff + (size_t)h * dv);
+  TO* y = out + ((size_t)n * H + h) * dv;
+  float4 u[VPT];
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = threadIdx.x + i * NT;
+    u[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (c < D4 && !pad) {
+      const float4 a = x[c], b = z[c];
+      u[i] = make_float4(gated(a.x, b.x, act), gated(a.y, b.y, act), gated(a.z, b.z, act), gated(a.w, b.w, act));
+    }
+    ss = fmaf(u[i].x, u[i].x, ss); ss = fmaf(u[i].y, u[i].y, ss); ss = fmaf(u[i].z, u[i].z, ss); ss = fmaf(u[i].w, u[i].w, ss);
+  }
+  const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)dv + eps);
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = threadIdx.x + i * NT;
+    if (c < D4) store4(y + 4 * c, make_float4(u[i].x * inv * g[i].x, u[i].y * inv * g[i].y, u[i].z * inv * g[i].z, u[i].w * inv * g[i].w));
+  }
+}
+
+template <typename TO>
+__global__ void __launch_bounds__(512)
+gate_norm_kernel(const float* __restrict__ o, int H, int dv, const float* __restrict__ w, int w_per_head, float eps,
+                 const float* __restrict__ gate, int ldg, int goff, int act, const int* __restrict__ seq_row,
+                 TO* __restrict__ out) {
+  fz_grid_launch_dependents();
+  fz_grid_wait();
+  __shared__ float scratch[32];
+  const int n = blockIdx.x, h = blockIdx.y;
+  const bool pad = seq_row[n] < 0;
+  const float* x = o + ((size_t)n * H + h) * dv;
+  const float* z = gate + (size_t)n * ldg + goff + (size_t)h * dv;
+  TO* y = out + ((size_t)n * H + h) * dv;
+  float ss = 0.f;
+  for (int c = threadIdx.x; c < dv && !pad; c += blockDim.x) {
+    const float u = gated(x[c], z[c], act);
+    ss = fmaf(u, u, ss);
+  }
+  const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)dv + eps);
+  for (int c = threadIdx.x; c < dv; c += blockDim.x) {
+    float u = pad ? 0.f : gated(x[c], z[c], act) * inv;
+    if (w != nullptr) u *= w[w_per_head ? (size_t)h * dv + c : c];
+    y[c] = Cvt<TO>::from_f(u);
+  }
+}
+
 // ------------------------------------------------------------------------------------------------ router
-// A warp per row: softmax over the E router logits, then lane 0 picks the groups and the experts. Scores of chosen
-// experts are overwritten with -1 in shared memory (scores are never negative), so each is picked once.
+// A warp per row. Scores s: softmax over the E router logits, or the sigmoid of each; choice scores c = s + correction (c = s
+// without one). A group's score is the sum of its `group_top` (1 or 2) largest choice scores; the `keep` best groups stay
+// (the lower index first among equals), the experts of the others get a choice score of minus infinity. Then `top` times
+// the largest remaining choice score (the lower index first among equals). Weights: the picked experts' s, divided by
+// (their sum, added in the order of the picks, + sum_eps) if renorm, times scale. A choice score that is not a number counts
+// as minus infinity; a picked expert's becomes one, so that no expert is picked twice.
+struct RouterRule {
+  int top, groups, keep, renorm, sigmoid, group_top;
+  const float* correction;
+  float sum_eps, scale;
+};
 constexpr int ROUTER_WARPS = 4;
 __global__ void __launch_bounds__(32 * ROUTER_WARPS)
-router_topk_kernel(const float* __restrict__ logits, int ld, int N, int E, int top, int groups, int keep, int renorm,
-                   const int* __restrict__ seq_row, int* __restrict__ choice, float* __restrict__ weight) {
+router_topk_kernel(const float* __restrict__ logits, int ld, int N, int E, const RouterRule p, const int* __restrict__ seq_row,
+                   int* __restrict__ choice, float* __restrict__ weight) {
   fz_grid_launch_dependents();
   fz_grid_wait();
   extern __shared__ __align__(16) float smem[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int n = blockIdx.x * ROUTER_WARPS + warp;
   if (n >= N) return;
-  float* s = smem + (size_t)warp * (E + groups + top);
-  float* gmax = s + E;
-  float* picked = gmax + groups;                       // the chosen scores, until their sum is known
+  const int top = p.top, groups = p.groups;
+  float* s = smem + (size_t)warp * (2 * E + groups + top);
+  float* c = s + E;
+  float* gs = c + E;
+  float* picked = gs + groups;                         // the chosen scores, until their sum is known
   if (seq_row[n] < 0) {
     for (int k = lane; k < top; k += 32) { choice[(size_t)n * top + k] = 0; weight[(size_t)n * top + k] = 0.f; }
     return;
   }
   const float* z = logits + (size_t)n * ld;
-  float mx = -INFINITY;
-  for (int e = lane; e < E; e += 32) mx = fmaxf(mx, z[e]);
-  mx = warp_max(mx);
-  float sum = 0.f;
-  for (int e = lane; e < E; e += 32) { const float v = expf(z[e] - mx); s[e] = v; sum += v; }
-  sum = warp_sum(sum);
-  __syncwarp();
-  for (int e = lane; e < E; e += 32) s[e] = __fdiv_rn(s[e], sum);
-  __syncwarp();
-  const int per = E / groups;
-  for (int g = lane; g < groups; g += 32) {
-    float v = -1.f;
-    for (int e = g * per; e < (g + 1) * per; ++e) v = fmaxf(v, s[e]);
-    gmax[g] = v;
+  if (p.sigmoid) {
+    for (int e = lane; e < E; e += 32) s[e] = 1.0f / (1.0f + expf(-z[e]));
+  } else {
+    float mx = -INFINITY;
+    for (int e = lane; e < E; e += 32) mx = fmaxf(mx, z[e]);
+    mx = warp_max(mx);
+    float sum = 0.f;
+    for (int e = lane; e < E; e += 32) { const float v = expf(z[e] - mx); s[e] = v; sum += v; }
+    sum = warp_sum(sum);
+    for (int e = lane; e < E; e += 32) s[e] = __fdiv_rn(s[e], sum);
+  }
+  for (int e = lane; e < E; e += 32) {                 // (a lane reads what it wrote itself)
+    const float v = p.correction != nullptr ? s[e] + p.correction[e] : s[e];
+    c[e] = isnan(v) ? -INFINITY : v;
   }
   __syncwarp();
-  if (lane == 0) {
-    // the groups that are not kept lose their experts: groups - keep times, strike the worst group (the higher index
-    // among equals, so that the lower index stays)
-    for (int d = 0; d < groups - keep; ++d) {
-      int worst = -1;
-      float wv = 0.f;
-      for (int g = 0; g < groups; ++g) {
-        if (gmax[g] < -1.5f) continue;                 // already struck
-        if (worst < 0 || !(gmax[g] > wv)) { worst = g; wv = gmax[g]; }
+  if (p.keep < groups) {
+    const int per = E / groups;
+    for (int g = lane; g < groups; g += 32) {
+      float first = -INFINITY, second = -INFINITY;
+      for (int e = g * per; e < (g + 1) * per; ++e) {
+        const float v = c[e];
+        if (v > first) { second = first; first = v; }
+        else if (v > second) second = v;
       }
-      gmax[worst] = -2.f;
-      for (int e = worst * per; e < (worst + 1) * per; ++e) s[e] = -1.f;
+      gs[g] = p.group_top == 2 && per > 1 ? first + second : first;
     }
-    float total = 0.f;
-    for (int k = 0; k < top; ++k) {
-      int best = -1;
-      float bv = -1.f;
-      for (int e = 0; e < E; ++e)
-        if (s[e] > bv) { best = e; bv = s[e]; }
-      if (best < 0) {                                  // scores that are not numbers: any expert not yet taken
-        for (int e = 0; e < E && best < 0; ++e)
-          if (!(s[e] == -1.f)) best = e;
-        if (best < 0) best = 0;
-        bv = 0.f;
-      }
+    __syncwarp();
+    for (int g = lane; g < groups; g += 32) {
+      const float v = gs[g];
+      int better = 0;
+      for (int o = 0; o < groups; ++o) better += gs[o] > v || (gs[o] == v && o < g);
+      if (better >= p.keep)
+        for (int e = g * per; e < (g + 1) * per; ++e) c[e] = -INFINITY;
+    }
+    __syncwarp();
+  }
+  float total = 0.f;
+  for (int k = 0; k < top; ++k) {
+    float bv = -INFINITY;
+    int best = 0x7fffffff;
+    for (int e = lane; e < E; e += 32) {
+      const float v = c[e];
+      if (!isnan(v) && (best == 0x7fffffff || v > bv)) { bv = v; best = e; }
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
+      const int oe = __shfl_xor_sync(0xffffffffu, best, o);
+      if (oe != 0x7fffffff && (best == 0x7fffffff || ov > bv || (ov == bv && oe < best))) { bv = ov; best = oe; }
+    }
+    const float sv = s[best];                          // (top <= E: some expert is always left)
+    total += sv;
+    __syncwarp();
+    if (lane == 0) {
       choice[(size_t)n * top + k] = best;
-      picked[k] = bv;
-      total += bv;
-      s[best] = -1.f;
+      picked[k] = sv;
+      c[best] = NAN;
     }
-    for (int k = 0; k < top; ++k) weight[(size_t)n * top + k] = renorm ? __fdiv_rn(picked[k], total) : picked[k];
+    __syncwarp();
+  }
+  for (int k = lane; k < top; k += 32) {
+    float v = p.renorm ? __fdiv_rn(picked[k], total + p.sum_eps) : picked[k];
+    if (p.scale != 1.f) v = __fmul_rn(v, p.scale);
+    weight[(size_t)n * top + k] = v;
   }
 }
 
@@ -1310,25 +1337,8 @@ __global__ void __launch_bounds__(256) weighted_sum_kernel(const Terms p, float*
   }
 }
 
-int lanes_per_column(int dk) {
-  int R = 1;
-  while (R * DPT < dk) R <<= 1;
-  return R;
-}
-
 size_t attn_smem(int dk, int dv, int pairs) {
   return sizeof(float) * ((size_t)CHUNK * (dk + 1) + (size_t)CHUNK * dv + (size_t)pairs * dk);
-}
-
-template <typename K>
-int allow_smem(K kern, size_t smem, size_t& allowed) {
-  if (smem > allowed) {
-    if (smem > 227 * 1024) return FZ_TOO_LARGE;
-    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    if (e != cudaSuccess) return (int)e;
-    allowed = smem;
-  }
-  return FZ_OK;
 }
 
 // rows_per_block: as many rows of a portion as give 32 (row, head) pairs at most.
@@ -1440,11 +1450,6 @@ FZ_API int fz_recurrent_key_pad(int dk) {
 }
 
 // Shared memory of a scan with `tch` tokens per chunk (floats): what the recurrence reads, then the raw staging area.
-// Threads of a scan block: R lanes for each group of DC of the head's value columns, a multiple of 32, SCAN_MAX_THREADS at most.
-static int scan_threads(int dv, int R) {
-  const long long want = ((long long)((dv + DC - 1) / DC) * R + 31) / 32 * 32;
-  return (int)(want < SCAN_MAX_THREADS ? want : SCAN_MAX_THREADS);
-}
 static size_t retention_smem(int dk, int R, int cols, int rotated, int tch) {
   const int dkp = R * DPT;
   return sizeof(float) * (size_t)tch * ((size_t)2 * dkp + cols + 2 * dk + cols + rotated);
@@ -1469,16 +1474,6 @@ static int launch_retention(const float* proj, int ld, int H, int dk, int dv, co
   FZ_LAUNCH_CHECK();
   return FZ_OK;
 }
-
-#define FZ_BY_LANES(R, CALL)          \
-  switch (R) {                        \
-    case 1: return CALL(1);           \
-    case 2: return CALL(2);           \
-    case 4: return CALL(4);           \
-    case 8: return CALL(8);           \
-    case 16: return CALL(16);         \
-    default: return CALL(32);         \
-  }
 
 FZ_API int fz_retention_scan(const float* proj, int ld, int H, int dk, int dv, const float* decay, float key_scale,
                              const float* cos_t, const float* sin_t, int rotated, int pairing, int max_pos, float* state,
@@ -1568,14 +1563,47 @@ FZ_API int fz_head_norm_gate(const float* o, int N, int H, int dv, const float* 
   return FZ_OK;
 }
 
-FZ_API int fz_router_topk(const float* logits, int ld, int N, int E, int top, int groups, int keep, int renorm,
-                          const int* seq_row, int* choice, float* weight, cudaStream_t stream) {
+// The same with the gate before the norm.
+template <typename TO>
+static int launch_gate_norm(const float* o, int N, int H, int dv, const float* w, int w_per_head, float eps, const float* gate,
+                            int ldg, int goff, int act, const int* seq_row, TO* out, cudaStream_t stream) {
+  int threads = ((dv + 3) / 4 + 31) / 32 * 32;
+  if (threads > 512) threads = 512;
+  const bool vec = dv % 4 == 0 && ldg % 4 == 0 && goff % 4 == 0 && dv <= 4 * 512 * 8 &&
+                   (((uintptr_t)o | (uintptr_t)w | (uintptr_t)gate | (uintptr_t)out) & 15) == 0;
+  const int per = (dv / 4 + threads - 1) / threads;
+#define FZ_GNV(V) fz_launch(gate_norm_vec_kernel<TO, V>, dim3(N, H), dim3(threads), 0, stream, o, H, dv, w, w_per_head, eps, gate, ldg, goff, act, seq_row, out)
+  if (!vec) fz_launch(gate_norm_kernel<TO>, dim3(N, H), dim3(threads), 0, stream, o, H, dv, w, w_per_head, eps, gate, ldg, goff, act, seq_row, out);
+  else if (per <= 1) FZ_GNV(1);
+  else if (per <= 2) FZ_GNV(2);
+  else if (per <= 4) FZ_GNV(4);
+  else FZ_GNV(8);
+#undef FZ_GNV
+  FZ_LAUNCH_CHECK();
+  return FZ_OK;
+}
+FZ_API int fz_gate_norm(const float* o, int N, int H, int dv, const float* w, int w_per_head, float eps, const float* gate, int ldg,
+                        int goff, int act, const int* seq_row, void* out, int out_dtype, cudaStream_t stream) {
+  if (N <= 0) return FZ_OK;
+  if (H <= 0 || H > 65535 || dv <= 0 || gate == nullptr || act < 1 || act > 2) return FZ_BAD_SHAPE;
+  if (out_dtype == FZ_F32) return launch_gate_norm<float>(o, N, H, dv, w, w_per_head, eps, gate, ldg, goff, act, seq_row, (float*)out, stream);
+  if (out_dtype == FZ_BF16) return launch_gate_norm<__nv_bfloat16>(o, N, H, dv, w, w_per_head, eps, gate, ldg, goff, act, seq_row, (__nv_bfloat16*)out, stream);
+  return FZ_BAD_DTYPE;
+}
+
+FZ_API int fz_router_topk(const float* logits, int ld, int N, int E, int top, int groups, int keep, int renorm, int sigmoid,
+                          const float* correction, int group_top, float sum_eps, float scale, const int* seq_row, int* choice,
+                          float* weight, cudaStream_t stream) {
   if (N <= 0) return FZ_OK;
   if (E <= 0 || E > 2048 || top <= 0 || top > E || groups <= 0 || E % groups || keep <= 0 || keep > groups ||
-      top > keep * (E / groups)) return FZ_BAD_SHAPE;
-  const size_t smem = sizeof(float) * ROUTER_WARPS * (size_t)(E + groups + top);
+      top > keep * (E / groups) || group_top < 1 || group_top > 2) return FZ_BAD_SHAPE;
+  const size_t smem = sizeof(float) * ROUTER_WARPS * (size_t)(2 * E + groups + top);
+  static size_t allowed = 48 * 1024;
+  int st = allow_smem(router_topk_kernel, smem, allowed);
+  if (st != FZ_OK) return st;
+  const RouterRule rule = {top, groups, keep, renorm, sigmoid, group_top, correction, sum_eps, scale};
   fz_launch(router_topk_kernel, dim3((N + ROUTER_WARPS - 1) / ROUTER_WARPS), dim3(32 * ROUTER_WARPS), smem, stream, logits, ld,
-            N, E, top, groups, keep, renorm, seq_row, choice, weight);
+            N, E, rule, seq_row, choice, weight);
   FZ_LAUNCH_CHECK();
   return FZ_OK;
 }

@@ -26,6 +26,8 @@ _DEVICE_ERRORS = {1: "a token id lies outside the embedding table", 2: "a positi
 
 _ACTIVATIONS = {"tanh": 0, "sigmoid": 1, "silu": 2, "gelu_tanh": 3, "identity": 4}
 RGLRU_COOK_ROWS = 4  # recurrent unit: steps whose longest portion is longer compute the recurrence's coefficients in a launch of their own
+SSD_SPREAD_ROWS = 16    # state space scan: in steps whose longest portion has this many rows a head's columns are spread over blocks of
+SSD_SPREAD_THREADS = 64  # this many threads (few blocks otherwise); shorter portions take blocks of up to 512 threads
 SINK_MMA_ROWS = 16  # windowed attention with a sink: steps whose longest portion has this many rows go to the tensor-core kernel
 LONG_PORTION = 8    # attention: portions of at least this many tokens go to the tile (prefill) kernels
 TILE_ROWS = 128     # token rows per tile of those kernels
@@ -123,7 +125,7 @@ class CudaOps(Ops):
         if self.dtype == torch.bfloat16:
             self.tc = load("fzb200_tc")      # tcgen05 / TMA kernels
         self.use_tensor_cores = self.tc is not None
-        self._attn_tc = self._mix = self._mix_tc = self._latent = self._latent_tc = self._seq = self._seq_tc = self._rows = None   # libraries loaded (and built) when a part first asks for their kernels
+        self._attn_tc = self._mix = self._mix_tc = self._latent = self._latent_tc = self._seq = self._seq_tc = self._rows = self._ssd = None   # libraries loaded (and built) when a part first asks for their kernels
         self.prefill_tcgen05 = True        # False: long portions on the mma.sync flash-attention kernel
         self.fuse_swiglu = True            # gate/up product and SwiGLU in one kernel where the sizes allow it
         self.fuse_argmax = True            # lm_head product and argmax in one pass where no logits are asked for
@@ -195,6 +197,13 @@ class CudaOps(Ops):
         if self._rows is None:
             self._rows = load("fzb200_rows")
         return self._rows
+
+    @property
+    def ssd(self):
+        """The selective state space scan."""
+        if self._ssd is None:
+            self._ssd = load("fzb200_ssd")
+        return self._ssd
 
     @property
     def mix(self):
@@ -331,7 +340,7 @@ class CudaOps(Ops):
         self._attn_items = min(self._attn_items or items, items)
 
     # ---- kernels
-    def embed(self, table, tokens, x, src=None, prev_ids=None, scale: float = 1.0) -> None:
+    def embed(self, table, tokens, x, src=None, prev_ids=None, scale: float = 1.0, copy=None) -> None:
         self._want(table, "embedding table", (torch.float32, torch.bfloat16), 2)
         self._want(tokens, "tokens", (torch.int32,), 1)
         self._want(x, "x", (torch.float32,), 2)
@@ -341,10 +350,14 @@ class CudaOps(Ops):
         if src is not None:
             self._want(src, "src", (torch.int32,), 1)
             self._want(prev_ids, "prev_ids", (torch.int32,), 1)
+        if copy is not None:
+            self._want(copy, "copy of x", (torch.float32,), 2)
+            if copy.shape != x.shape:
+                raise KernelError(f"embed: copy {tuple(copy.shape)} vs x {tuple(x.shape)}")
         self._check(self.core.fz_embed(_p(table), c_int(_CODE[table.dtype]), _p(tokens), _p(src),
-                                       _p(prev_ids if src is not None else None), _p(x), c_int(n), c_int(d),
+                                       _p(prev_ids if src is not None else None), _p(x), _p(copy), c_int(n), c_int(d),
                                        c_int(table.shape[0]), c_float(scale), _p(self.err), self._stream()), "embed",
-                    n * d * (table.element_size() + 4))
+                    n * d * (table.element_size() + (4 if copy is None else 8)))
 
     def add_rmsnorm(self, x, delta, weight, eps, h, rows=None, groups: int = 1) -> None:
         self._want(x, "x", (torch.float32,), 2)
@@ -374,6 +387,29 @@ class CudaOps(Ops):
                                              c_int(_CODE[h.dtype]), _p(rows), c_int(n_out), c_int(n_src), c_int(d),
                                              c_float(eps), _p(self.err), self._stream()), "add_rmsnorm",
                     n_out * d * (4 + (8 if delta is not None and rows is None else 4 if delta is not None else 0) + h.element_size()))
+
+    def add_layernorm(self, x, delta, extra, weight, eps, h, rows=None) -> None:
+        self._want(x, "x", (torch.float32,), 2)
+        self._want(weight, "norm weight", (torch.float32,), 1)
+        self._want(h, "h", (torch.float32, torch.bfloat16), 2)
+        for t, name in ((delta, "delta"), (extra, "extra")):
+            if t is not None:
+                self._want(t, name, (torch.float32,), 2)
+                if t.shape != x.shape:
+                    raise KernelError(f"add_layernorm: {name} {tuple(t.shape)} vs x {tuple(x.shape)}")
+        n_src, d = x.shape
+        n_out = n_src
+        if rows is not None:
+            self._want(rows, "rows", (torch.int32,), 1)
+            n_out = rows.shape[0]
+            if extra is not None:
+                raise KernelError("add_layernorm: selected rows take no extra stream")
+        if h.shape != (n_out, d) or weight.shape[0] != d:
+            raise KernelError(f"add_layernorm: h {tuple(h.shape)}, expected {(n_out, d)}; weight {tuple(weight.shape)}")
+        adds = (delta is not None) + (extra is not None)
+        self._check(self.core.fz_add_layernorm(_p(x), _p(delta), _p(extra), _p(weight), _p(h), c_int(_CODE[h.dtype]), _p(rows),
+                                               c_int(n_out), c_int(n_src), c_int(d), c_float(eps), _p(self.err), self._stream()),
+                    "add_layernorm", n_out * d * (4 + 4 * adds + (4 if adds and rows is None else 0) + h.element_size()))
 
     def linear(self, a, w, bias, out) -> None:
         self._want(a, "linear input", (self.dtype,), 2)
@@ -633,19 +669,20 @@ class CudaOps(Ops):
             raise KernelError("select_tokens: row counts differ")
         self._check(self.mix.fz_select_tokens(_p(tokens), _p(src), _p(prev_ids), _p(out), c_int(n), self._stream()), "select_tokens")
 
-    def short_conv(self, h, w, state, meta, out, residual: bool = True, activation: str | None = None, bias=None) -> None:
+    def short_conv(self, h, w, state, meta, out, residual: bool = True, activation: str | None = None, bias=None,
+                   offset: int | None = None) -> None:
         if activation not in (None, "silu"):
             raise KernelError(f"short_conv: activation {activation!r} is not one of None, 'silu'")
-        self._want(h, "convolution input", (self.dtype,), 2)
+        self._want(h, "convolution input", (self.dtype if offset is None else torch.float32,), 2)
         self._want(w, "convolution weight", (self.dtype,), 2)
         self._want(out, "convolution output", (self.dtype,), 2)
-        n, c = h.shape
+        n, c = out.shape
         taps = w.shape[1]
         if bias is not None:
             self._want(bias, "convolution bias", (torch.float32,), 1)
             if bias.shape[0] != c:
                 raise KernelError(f"short_conv: bias {tuple(bias.shape)} for {c} channels")
-        if w.shape[0] != c or out.shape != h.shape:
+        if w.shape[0] != c or h.shape[0] != n or (h.shape[1] != c if offset is None else residual or not 0 <= offset <= h.shape[1] - c):
             raise KernelError(f"short_conv: h {tuple(h.shape)}, w {tuple(w.shape)}, out {tuple(out.shape)}")
         if taps > 1:
             if state is None:
@@ -653,11 +690,14 @@ class CudaOps(Ops):
             self._want(state, "convolution state", (torch.float32,), 3)
             if tuple(state.shape[1:]) != (taps - 1, c):
                 raise KernelError(f"short_conv: state {tuple(state.shape)}, expected (slots, {taps - 1}, {c})")
-        self._check(self.mix.fz_short_conv(_p(h), _p(w), _p(state), _p(meta.seg), _p(meta.seq_row), _p(out),
-                                           c_int(_CODE[self.dtype]), c_int(n), c_int(getattr(meta, "max_segments", meta.n_segments)), c_int(c), c_int(taps),
-                                           c_int(1 if residual else 0), c_int(1 if activation else 0), _p(bias), self._stream()), "short_conv",
-                    n * c * 2 * h.element_size())
-        if taps > 1:
+        # a step of single tokens, in a model whose parts make the longest portion part of a step's shape: one launch
+        single = getattr(meta, "portion_tiles", 0) == 1
+        self._check(self.mix.fz_short_conv(_p(h), c_int(_CODE[h.dtype]), c_int(h.shape[1]), c_int(offset or 0), _p(w), _p(state),
+                                           _p(meta.seg), _p(meta.seq_row), _p(out), c_int(_CODE[self.dtype]), c_int(n),
+                                           c_int(getattr(meta, "max_segments", meta.n_segments)), c_int(c), c_int(taps),
+                                           c_int(1 if residual else 0), c_int(1 if activation else 0), _p(bias), c_int(1 if single else 0),
+                                           self._stream()), "short_conv", n * c * (h.element_size() + out.element_size()))
+        if taps > 1 and not single:
             self.launches += 1    # the state update
 
     def gated_sum(self, a, gate_a, f, gate_f, out, f_terms: int = 1, f_weight: float = 1.0) -> None:
@@ -924,7 +964,29 @@ class CudaOps(Ops):
             n * (qkv.shape[1] * qkv.element_size() + heads * (key_dim + value_dim + 1) * 4)
             + 2 * meta.n_segments * heads * value_dim * state.shape[3] * 4)
 
-    def head_norm_gate(self, o, heads, value_dim, weight, eps, gate, gate_offset, activation, out) -> None:
+    def ssd_scan(self, xbc, heads, groups, state_dim, value_dim, dt, dt_offset, dt_bias, a_log, skip, state, meta, out) -> None:
+        self._want(xbc, "x, B and C", (self.dtype,), 2)
+        self._want(dt, "step sizes", (torch.float32,), 2)
+        self._want(out, "state space output", (torch.float32,), 2)
+        n, w = xbc.shape
+        for t, name in ((dt_bias, "step size bias"), (a_log, "decay rates"), (skip, "skip weights")):
+            self._want(t, name, (torch.float32,), 1)
+            if t.shape[0] != heads:
+                raise KernelError(f"ssd_scan: {name} {tuple(t.shape)} for {heads} heads")
+        if heads % groups or w != heads * value_dim + 2 * groups * state_dim or dt.shape[0] != n or dt_offset < 0 or \
+                dt_offset + heads > dt.shape[1] or tuple(out.shape) != (n, heads * value_dim):
+            raise KernelError(f"ssd_scan: rows {tuple(xbc.shape)}, step sizes {tuple(dt.shape)} from column {dt_offset}, out {tuple(out.shape)}")
+        self._state(state, heads, state_dim, value_dim, "ssd_scan")
+        self._meta_rows = meta.seq_row
+        nbytes = n * (w * xbc.element_size() + heads * (value_dim + 1) * 4) + 2 * meta.n_segments * heads * value_dim * state.shape[3] * 4
+        max_portion = max(1, int(getattr(meta, "max_portion", 0)) or n)
+        self._check(self.ssd.fz_ssd_scan(
+            _p(xbc), c_int(_CODE[self.dtype]), c_int(heads), c_int(groups), c_int(state_dim), c_int(value_dim), _p(dt), c_int(dt.shape[1]),
+            c_int(dt_offset), _p(dt_bias), _p(a_log), _p(skip), _p(state), _p(meta.seg),
+            c_int(getattr(meta, "max_segments", meta.n_segments)), c_int(SSD_SPREAD_THREADS if max_portion >= SSD_SPREAD_ROWS else 512),
+            _p(out), self._stream()), "ssd_scan", nbytes)
+
+    def head_norm_gate(self, o, heads, value_dim, weight, eps, gate, gate_offset, activation, out, gate_first: bool = False) -> None:
         self._want(o, "head outputs", (torch.float32,), 2)
         self._want(out, "normed head outputs", (torch.float32, self.dtype), 2)
         n = o.shape[0]
@@ -945,6 +1007,14 @@ class CudaOps(Ops):
                 raise KernelError(f"head_norm_gate: gate {tuple(gate.shape)} from column {gate_offset}, activation {activation!r}")
         seq_row = self._step_rows(n)
         per_head = 1 if weight is not None and heads > 1 and weight.shape[0] == heads * value_dim else 0
+        if gate_first:
+            if gate is None:
+                raise KernelError("head_norm_gate: a gate before the norm needs a gate")
+            self._check(self.seq.fz_gate_norm(_p(o), c_int(n), c_int(heads), c_int(value_dim), _p(weight), c_int(per_head), c_float(eps),
+                                              _p(gate), c_int(ldg), c_int(gate_offset), c_int(act), _p(seq_row), _p(out),
+                                              c_int(_CODE[out.dtype]), self._stream()),
+                        "gate_norm", n * heads * value_dim * (8 + out.element_size()))
+            return
         self._check(self.seq.fz_head_norm_gate(_p(o), c_int(n), c_int(heads), c_int(value_dim), _p(weight), c_int(per_head), c_float(eps),
                                                _p(gate), c_int(ldg), c_int(gate_offset), c_int(act if gate is not None else 0),
                                                _p(seq_row), _p(out), c_int(_CODE[out.dtype]), self._stream()),
@@ -1217,7 +1287,14 @@ class CudaOps(Ops):
                                              c_longlong(out.numel()), self._stream()), "weighted_sum",
                     out.numel() * 4 * (len(terms) + 1))
 
-    def route_by_scores(self, logits, num_experts, top, groups, keep_groups, renormalize, meta, weights, align: int = 1):
+    def route_by_scores(self, logits, num_experts, top, groups, keep_groups, renormalize, meta, weights, align: int = 1,
+                        scoring: str = "softmax", correction=None, group_top: int = 1, sum_eps: float = 0.0, scale: float = 1.0):
+        if scoring not in ("softmax", "sigmoid"):
+            raise KernelError(f"route_by_scores: scoring {scoring!r} is not one of 'softmax', 'sigmoid'")
+        if correction is not None:
+            self._want(correction, "router correction", (torch.float32,), 1)
+            if correction.shape[0] != num_experts:
+                raise KernelError(f"route_by_scores: correction {tuple(correction.shape)} for {num_experts} experts")
         self._want(logits, "router logits", (torch.float32,), 2)
         self._want(weights, "router weights", (torch.float32,), 2)
         n = logits.shape[0]
@@ -1225,8 +1302,9 @@ class CudaOps(Ops):
             raise KernelError(f"route_by_scores: logits {tuple(logits.shape)}, weights {tuple(weights.shape)}, {num_experts} experts")
         choice = self._scratch("router choices", max(n, 1) * top, torch.int32)[:n * top].view(n, top)
         self._check(self.seq.fz_router_topk(_p(logits), c_int(logits.shape[1]), c_int(n), c_int(num_experts), c_int(top),
-                                            c_int(groups), c_int(keep_groups), c_int(1 if renormalize else 0), _p(meta.seq_row),
-                                            _p(choice), _p(weights), self._stream()), "router_topk")
+                                            c_int(groups), c_int(keep_groups), c_int(1 if renormalize else 0),
+                                            c_int(1 if scoring == "sigmoid" else 0), _p(correction), c_int(group_top),
+                                            c_float(sum_eps), c_float(scale), _p(meta.seq_row), _p(choice), _p(weights), self._stream()), "router_topk")
         self._meta_rows = meta.seq_row
         return self._sort_pairs(None, n, meta, choice, num_experts, align)
 
