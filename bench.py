@@ -1,7 +1,7 @@
 """Benchmark: decode tokens per second of the Llama-3.1-8B-sized model (random bf16 weights) on one B200.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--batch 8] [--context 4096] [--layers L] [--impl ours|reference]
-                    [--preset NAME] [--workload decode|stream|pepilix|gizulorn|nepudra|gimotar]
+                    [--preset NAME] [--workload decode|stream|pepilix|gizulorn|nepudra|gimotar|gimupel]
 
 A "step" is one decode step of `--batch` requests whose contexts end at `--context` tokens. Prints ONE JSON line:
   value      decoded tokens per second, timed on the device (CUDA events around K steps: metadata copy + graph replay)
@@ -32,6 +32,9 @@ layers, heads, window and dense feed-forward size.
 `--workload gimotar` (`--sizes m1024,m2048`, `--layers 4`) does the same for the Gimotar design (real-gated recurrent unit,
 latent attention with a sink and an output gate, attention under a chunked mask with blended values, routed experts with a
 shared expert in a parallel block), beside Gizulorn at equal sizes.
+`--workload gimupel` (`--sizes p1024,p2048`, `--layers 4`) does the same for the Gimupel design (selective state space
+layers with a convolution and a gated norm in parts, windowed attention with normed heads, experts chosen by corrected
+sigmoid scores in groups, layers run twice with the embedding added again), beside Gizulorn at equal sizes.
 `--workload pepilix` (`--sizes w1024,w2048`, `--layers 4`) times the Pepilix design beside the dense decoder at equal
 width, layers, heads, vocabulary and active feed-forward size: a 2,048-token prompt and decode steps at `--batch`
 requests through `LLMEngine.step()`, and (unless `--no-points`) a kernel-by-kernel profile of both; its line's `sizes`
@@ -163,7 +166,7 @@ def main() -> int:
     ap.add_argument("--no-points", action="store_true", help="skip the batch 1 and 64 points")
     ap.add_argument("--no-e2e", action="store_true")
     ap.add_argument("--reference-device", default="CUDA", help="the reference's device name for --impl reference")
-    ap.add_argument("--workload", default="decode", choices=["decode", "stream", "pepilix", "gizulorn", "nepudra", "gimotar"],
+    ap.add_argument("--workload", default="decode", choices=["decode", "stream", "pepilix", "gizulorn", "nepudra", "gimotar", "gimupel"],
                     help="pepilix: prefill and decode of the Pepilix design at a few layer sizes, beside the dense decoder "
                          "at equal width, layers, heads and active feed-forward size")
     ap.add_argument("--sizes", default="w1024,w2048", help="pepilix workload: which of its sizes to run")
@@ -199,6 +202,8 @@ def main() -> int:
         return design_workload(a, "nepudra")
     if a.workload == "gimotar":
         return design_workload(a, "gimotar")
+    if a.workload == "gimupel":
+        return design_workload(a, "gimupel")
 
     import numpy as np
     import torch
@@ -521,6 +526,34 @@ def gimotar_configs(name: str, L: int, ctx: int):
     return gim, giz
 
 
+# Layer sizes for the Gimupel workload: (width, heads, value size, state size, groups, parts of the gated norm of the state
+# space layers, heads, kv heads and head size of the windowed attention, window, experts, top, groups, kept groups, expert
+# ff, dense ff, vocab). Layers cycle through state space with a dense feed-forward, attention, state space, state space with
+# routed experts; the last layer listed runs twice (so a model of L layer runs lists L - 1). Gizulorn beside it
+# (`GIZULORN_SIZES` of the same width) has the same width, layer runs, attention heads and window, experts, groups, expert
+# sizes and vocabulary: each of Gimupel's kernels has a like kernel there (the state space scan's are the retention and
+# the delta rule).
+GIMUPEL_SIZES = {
+    "p1024": (1024, 32, 64, 128, 1, 4, 8, 2, 64, 512, 16, 2, 4, 2, 512, 1536, 32768),
+    "p2048": (2048, 64, 64, 128, 8, 8, 16, 4, 128, 1024, 32, 4, 8, 4, 512, 3072, 32768),
+}
+
+
+def gimupel_configs(name: str, L: int, ctx: int):
+    D, H, P, N, G, parts, Ha, kv, hd, window, E, top, groups, keep, ff, dense_ff, V = GIMUPEL_SIZES[name]
+    moe = {"kind": "moe", "router": {"experts": E, "top": top, "groups": {"count": groups, "keep": keep}, "scale": 2.5},
+           "expert": {"ff": ff, "limit": 7.0}}
+    ssm = {"heads": H, "vdim": P, "state": N, "groups": G, "conv": 4, "norm_groups": parts}
+    att = {"heads": Ha, "kv_heads": kv, "dim": hd, "vdim": hd, "scale": hd ** -0.5, "mask": {"size": window}}
+    cycle = [("mamba2", ssm, {"kind": "dense", "ff": dense_ff}), ("attention", att, moe), ("mamba2_2", ssm, moe), ("mamba2", ssm, moe)]
+    layers = [dict(zip(("type", "mixer", "mlp"), cycle[i % 4])) for i in range(max(1, L - 1))]
+    gip = {"architecture": "Gimupel", "vocab": V, "width": D, "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0}, "layers": layers}
+    if L > 1:
+        gip["loop"] = {"start": L - 2, "stop": L - 1, "times": 2}
+    giz, _ = gizulorn_configs("g" + name[1:], L, ctx)
+    return gip, giz
+
+
 def pepilix_workload(a) -> int:
     return design_workload(a, "pepilix")
 
@@ -541,8 +574,9 @@ def design_workload(a, design: str) -> int:
     pk = peaks()
     rng = np.random.default_rng(5)
 
-    SIZES = {"pepilix": PEPILIX_SIZES, "gizulorn": GIZULORN_SIZES, "nepudra": NEPUDRA_SIZES, "gimotar": GIMOTAR_SIZES}[design]
-    twin = "gizulorn" if design in ("nepudra", "gimotar") else "dense"        # the model timed beside the design
+    SIZES = {"pepilix": PEPILIX_SIZES, "gizulorn": GIZULORN_SIZES, "nepudra": NEPUDRA_SIZES, "gimotar": GIMOTAR_SIZES,
+             "gimupel": GIMUPEL_SIZES}[design]
+    twin = "gizulorn" if design in ("nepudra", "gimotar", "gimupel") else "dense"        # the model timed beside the design
 
     def configs(name):
         if design == "gizulorn":
@@ -551,6 +585,8 @@ def design_workload(a, design: str) -> int:
             return nepudra_configs(name, L, ctx)
         if design == "gimotar":
             return gimotar_configs(name, L, ctx)
+        if design == "gimupel":
+            return gimupel_configs(name, L, ctx)
         D, H, dn, dr, dv, r, E, top, ff, V = PEPILIX_SIZES[name]
         mixer = {"heads": H, "dim": dn, "rot_dim": dr, "vdim": dv, "kv_rank": r, "scale": (dn + dr) ** -0.5,
                  "rot": {"base": 10000.0, "dims": dr}}
@@ -655,6 +691,9 @@ def design_workload(a, design: str) -> int:
                                          ("width", "rglru_width", "rglru_blocks", "latent_heads", "dim", "rot_dim", "vdim", "kv_rank",
                                           "heads", "kv_heads", "head_dim", "chunk", "experts", "top", "ff", "shared_ff", "vocab")
                                          if design == "gimotar" else
+                                         ("width", "ssm_heads", "ssm_vdim", "state", "groups", "norm_groups", "heads", "kv_heads", "head_dim",
+                                          "window", "experts", "top", "expert_groups", "keep", "ff", "dense_ff", "vocab")
+                                         if design == "gimupel" else
                                          ("width", "heads", "dim", "vdim", "kv_heads", "window", "key_heads", "experts", "top", "groups",
                                           "keep", "ff", "shared_ff", "vocab"), SIZES[n])) for n in sizes},
                    "beside": twin,

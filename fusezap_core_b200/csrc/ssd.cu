@@ -20,19 +20,20 @@ __device__ __forceinline__ void stage_piece(T* dst, const T* src, int i, int byt
   else dst[i] = src[i];
 }
 
-// xbc rows of W values: [x (H dv) | B (G dk) | C (G dk)]. grid (portions, heads, slices of the value columns).
+// xbc rows of W values: [x (H dv) | B (G dk) | C (G dk)]. Portions of more than max_rows rows are left alone. grid
+// (portions, heads, slices of the value columns).
 template <typename T, int R>
 __global__ void __launch_bounds__(SCAN_MAX_THREADS)
 ssd_scan_kernel(const T* __restrict__ xbc, int W, int H, int G, int dk, int dv, int tch, int bytes,
                 const float* __restrict__ dt, int ldt, int off_dt, const float* __restrict__ dt_bias,
                 const float* __restrict__ a_log, const float* __restrict__ skip, float* __restrict__ state,
-                const int* __restrict__ seg, float* __restrict__ out) {
+                const int* __restrict__ seg, int max_rows, float* __restrict__ out) {
   fz_grid_launch_dependents();
   const int s = blockIdx.x, h = blockIdx.y;
   const int row0 = seg[4 * s], cnt = seg[4 * s + 1], slot = seg[4 * s + 3];
   const float rate = expf(a_log[h]), bias = dt_bias[h], D = skip[h];
   fz_grid_wait();
-  if (cnt <= 0 || slot < 0) return;
+  if (cnt <= 0 || cnt > max_rows || slot < 0) return;
   extern __shared__ __align__(16) float smem[];
   const int NT = blockDim.x;
   const int dkp = R * DPT, COLS = NT / R * DC;
@@ -142,7 +143,7 @@ size_t ssd_smem(int dk, int R, int cols, int tch, size_t elem) {
 
 template <typename T, int R>
 int launch_ssd(const void* xbc, int W, int H, int G, int dk, int dv, const float* dt, int ldt, int off_dt, const float* dt_bias,
-               const float* a_log, const float* skip, float* state, const int* seg, int n_seg, int cap, float* out,
+               const float* a_log, const float* skip, float* state, const int* seg, int n_seg, int max_rows, int cap, float* out,
                cudaStream_t stream) {
   int threads = scan_threads(dv, R);
   if (threads > cap) threads = cap;      // long portions: a head's columns are spread over several blocks
@@ -163,22 +164,23 @@ int launch_ssd(const void* xbc, int W, int H, int G, int dk, int dv, const float
   };
   const int bytes = fits(16) ? 16 : fits(4) ? 4 : 0;
   fz_launch(ssd_scan_kernel<T, R>, dim3(n_seg, H, (dv + cols - 1) / cols), dim3(threads), smem, stream, (const T*)xbc, W, H, G,
-            dk, dv, tch, bytes, dt, ldt, off_dt, dt_bias, a_log, skip, state, seg, out);
+            dk, dv, tch, bytes, dt, ldt, off_dt, dt_bias, a_log, skip, state, seg, max_rows, out);
   FZ_LAUNCH_CHECK();
   return FZ_OK;
 }
 }  // namespace
 
-// threads: the most threads a block may have (a multiple of 32, at most 512).
+// Portions of more than max_rows rows are passed over. threads: the most threads a block may have (a multiple of 32, at
+// most 512).
 FZ_API int fz_ssd_scan(const void* xbc, int dtype, int H, int G, int dk, int dv, const float* dt, int ldt, int off_dt,
                        const float* dt_bias, const float* a_log, const float* skip, float* state, const int* seg, int n_seg,
-                       int threads, float* out, cudaStream_t stream) {
+                       int max_rows, int threads, float* out, cudaStream_t stream) {
   if (n_seg <= 0) return FZ_OK;
   if (H <= 0 || H > 65535 || G <= 0 || H % G || dk <= 0 || dk > 32 * DPT || dv <= 0 || threads < 32 || threads % 32 ||
       threads > SCAN_MAX_THREADS) return FZ_BAD_SHAPE;
   const int W = H * dv + 2 * G * dk;
-#define FZ_CALL_F(R) launch_ssd<float, R>(xbc, W, H, G, dk, dv, dt, ldt, off_dt, dt_bias, a_log, skip, state, seg, n_seg, threads, out, stream)
-#define FZ_CALL_B(R) launch_ssd<__nv_bfloat16, R>(xbc, W, H, G, dk, dv, dt, ldt, off_dt, dt_bias, a_log, skip, state, seg, n_seg, threads, out, stream)
+#define FZ_CALL_F(R) launch_ssd<float, R>(xbc, W, H, G, dk, dv, dt, ldt, off_dt, dt_bias, a_log, skip, state, seg, n_seg, max_rows, threads, out, stream)
+#define FZ_CALL_B(R) launch_ssd<__nv_bfloat16, R>(xbc, W, H, G, dk, dv, dt, ldt, off_dt, dt_bias, a_log, skip, state, seg, n_seg, max_rows, threads, out, stream)
   if (dtype == FZ_F32) { FZ_BY_LANES(lanes_per_column(dk), FZ_CALL_F) }
   if (dtype == FZ_BF16) { FZ_BY_LANES(lanes_per_column(dk), FZ_CALL_B) }
 #undef FZ_CALL_F

@@ -176,6 +176,10 @@ class Ops:
         the norm: u = o * act(gate), out = T(u / sqrt(mean_c(u[n, h]^2) + eps) * weight)."""
         raise NotImplementedError
 
+    def check_ssd_scan(self, heads: int, groups: int, state_dim: int, value_dim: int) -> None:
+        """Raise ValueError if `ssd_scan` cannot take these sizes."""
+        raise NotImplementedError
+
     def ssd_scan(self, xbc: torch.Tensor, heads: int, groups: int, state_dim: int, value_dim: int, dt: torch.Tensor,
                  dt_offset: int, dt_bias: torch.Tensor, a_log: torch.Tensor, skip: torch.Tensor, state: torch.Tensor,
                  meta: Any, out: torch.Tensor) -> None:

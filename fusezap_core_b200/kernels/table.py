@@ -26,6 +26,7 @@ _DEVICE_ERRORS = {1: "a token id lies outside the embedding table", 2: "a positi
 
 _ACTIVATIONS = {"tanh": 0, "sigmoid": 1, "silu": 2, "gelu_tanh": 3, "identity": 4}
 RGLRU_COOK_ROWS = 4  # recurrent unit: steps whose longest portion is longer compute the recurrence's coefficients in a launch of their own
+SSD_CHUNK_ROWS = 16     # state space scan (bfloat16): portions of this many rows and more go to the tensor-core kernel where the sizes allow it
 SSD_SPREAD_ROWS = 16    # state space scan: in steps whose longest portion has this many rows a head's columns are spread over blocks of
 SSD_SPREAD_THREADS = 64  # this many threads (few blocks otherwise); shorter portions take blocks of up to 512 threads
 SINK_MMA_ROWS = 16  # windowed attention with a sink: steps whose longest portion has this many rows go to the tensor-core kernel
@@ -125,7 +126,7 @@ class CudaOps(Ops):
         if self.dtype == torch.bfloat16:
             self.tc = load("fzb200_tc")      # tcgen05 / TMA kernels
         self.use_tensor_cores = self.tc is not None
-        self._attn_tc = self._mix = self._mix_tc = self._latent = self._latent_tc = self._seq = self._seq_tc = self._rows = self._ssd = None   # libraries loaded (and built) when a part first asks for their kernels
+        self._attn_tc = self._mix = self._mix_tc = self._latent = self._latent_tc = self._seq = self._seq_tc = self._rows = self._ssd = self._ssd_tc = None   # libraries loaded (and built) when a part first asks for their kernels
         self.prefill_tcgen05 = True        # False: long portions on the mma.sync flash-attention kernel
         self.fuse_swiglu = True            # gate/up product and SwiGLU in one kernel where the sizes allow it
         self.fuse_argmax = True            # lm_head product and argmax in one pass where no logits are asked for
@@ -141,6 +142,7 @@ class CudaOps(Ops):
         self.cut_prefill_keys = True       # few query tiles with many keys behind them are cut along the keys
         self._profile = None               # a StepProfile while the engine profiles its steps
         self._meta_rows = None             # meta.seq_row of the step being run, for ops that take no `meta`
+        self.ssd_tensor_cores = True       # state space scan of long portions on tensor cores (bfloat16)
         self.split_decode_keys = True      # windowed attention with a sink: steps of single tokens cut a row's keys into runs
         self.sink_tensor_cores = True      # that attention on tensor cores for portions of SINK_MMA_ROWS rows and more (bfloat16)
         # the fewest query heads, and the fewest items of a query tile on the prompt kernel, among the attention layers
@@ -204,6 +206,13 @@ class CudaOps(Ops):
         if self._ssd is None:
             self._ssd = load("fzb200_ssd")
         return self._ssd
+
+    @property
+    def ssd_tc(self):
+        """That scan for long portions on tensor cores (bfloat16)."""
+        if self._ssd_tc is None:
+            self._ssd_tc = load("fzb200_ssd_tc")
+        return self._ssd_tc
 
     @property
     def mix(self):
@@ -910,6 +919,17 @@ class CudaOps(Ops):
             raise ValueError(f"a recurrent state with {key_dim} key dimensions is not supported (1..256)")
         return (heads, value_dim, pad)
 
+    def check_ssd_scan(self, heads: int, groups: int, state_dim: int, value_dim: int) -> None:
+        """Builds and loads the libraries with the model, not at its first step; raises for sizes the scan cannot take."""
+        self.recurrent_state_shape(heads, state_dim, value_dim)
+        self.ssd
+        if self._ssd_chunked(None, heads, groups, state_dim, value_dim):
+            self.ssd_tc
+
+    def _ssd_chunked(self, xbc, heads: int, groups: int, state_dim: int, value_dim: int) -> bool:
+        return bool(self.use_tensor_cores and self.ssd_tensor_cores and self.dtype == torch.bfloat16 and state_dim % 16 == 0 and
+                    value_dim % 16 == 0 and self.ssd_tc.fz_ssd_chunk_check(_p(xbc), c_int(heads), c_int(groups), c_int(state_dim), c_int(value_dim)) == 0)
+
     def _state(self, state, heads, key_dim, value_dim, what):
         self._want(state, f"{what} state", (torch.float32,), 4)
         if tuple(state.shape[1:]) != self.recurrent_state_shape(heads, key_dim, value_dim):
@@ -980,10 +1000,22 @@ class CudaOps(Ops):
         self._meta_rows = meta.seq_row
         nbytes = n * (w * xbc.element_size() + heads * (value_dim + 1) * 4) + 2 * meta.n_segments * heads * value_dim * state.shape[3] * 4
         max_portion = max(1, int(getattr(meta, "max_portion", 0)) or n)
+        max_rows = 2 ** 31 - 1
+        n_seg = getattr(meta, "max_segments", meta.n_segments)
+        if max_portion >= SSD_CHUNK_ROWS and self._ssd_chunked(xbc, heads, groups, state_dim, value_dim):
+            # long portions 64 tokens at a time on tensor cores, the step's short ones (if it can have any: its rows are
+            # more than the longest portion's) token by token
+            self._check(self.ssd_tc.fz_ssd_chunk(
+                _p(xbc), c_int(heads), c_int(groups), c_int(state_dim), c_int(value_dim), _p(dt), c_int(dt.shape[1]), c_int(dt_offset),
+                _p(dt_bias), _p(a_log), _p(skip), _p(state), c_int(state.shape[3]), _p(meta.seg), c_int(n_seg), c_int(SSD_CHUNK_ROWS),
+                _p(out), self._stream()), "ssd_scan (tensor cores)", nbytes)
+            if max_portion == n:
+                return
+            max_rows, nbytes = SSD_CHUNK_ROWS - 1, 0
         self._check(self.ssd.fz_ssd_scan(
             _p(xbc), c_int(_CODE[self.dtype]), c_int(heads), c_int(groups), c_int(state_dim), c_int(value_dim), _p(dt), c_int(dt.shape[1]),
             c_int(dt_offset), _p(dt_bias), _p(a_log), _p(skip), _p(state), _p(meta.seg),
-            c_int(getattr(meta, "max_segments", meta.n_segments)), c_int(SSD_SPREAD_THREADS if max_portion >= SSD_SPREAD_ROWS else 512),
+            c_int(n_seg), c_int(max_rows), c_int(SSD_SPREAD_THREADS if max_portion >= SSD_SPREAD_ROWS and max_rows >= max_portion else 512),
             _p(out), self._stream()), "ssd_scan", nbytes)
 
     def head_norm_gate(self, o, heads, value_dim, weight, eps, gate, gate_offset, activation, out, gate_first: bool = False) -> None:

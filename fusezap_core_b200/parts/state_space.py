@@ -57,6 +57,7 @@ class StateSpace(Mixer):
         self.w_in, self.wo = tensors[n["in"]], tensors[n["out"]]
         self.dt_bias, self.a_log, self.skip, self.norm_w = (tensors[n[k]].float().contiguous()
                                                             for k in ("dt_bias", "decay_log", "skip", "norm"))
+        ops.check_ssd_scan(self.H, self.G, self.N, self.P)
         self.state_shape = ops.recurrent_state_shape(self.H, self.N, self.P)
 
     def children(self):

@@ -3,9 +3,12 @@ token by token where the design is a recurrence. It shares no code with the pack
 of config.json, which are the design's own).
 
 A model is (config dict, {tensor name: float64 tensor}). `forward(config, tensors, tokens)` returns the logits of every
-position, and with `layers=True` also the residual stream after every layer that ran.
+position, and with `layers=True` also the residual stream after every layer that ran. Inside `with rounded_operands():`
+what a 16-bit engine hands to its matrix products, its cache and its scan is rounded to bfloat16 on the way, which shows
+how far rounding alone moves the logits.
 """
 from __future__ import annotations
+import contextlib
 import math
 
 import torch
@@ -13,6 +16,23 @@ import torch
 F = torch.float64
 GATE_SHARPNESS = 1.702       # an expert's gate: g * sigmoid(1.702 g)
 SUM_EPS = 1e-20              # added to the sum of the chosen scores
+
+
+_rounding = False
+
+
+@contextlib.contextmanager
+def rounded_operands():
+    global _rounding
+    _rounding = True
+    try:
+        yield
+    finally:
+        _rounding = False
+
+
+def R(x: torch.Tensor) -> torch.Tensor:
+    return x.to(torch.bfloat16).to(x.dtype) if _rounding else x
 
 
 def sigmoid(z: torch.Tensor) -> torch.Tensor:
@@ -92,11 +112,11 @@ def state_space(cfg: dict, w: dict, p: str, m: dict, h: torch.Tensor) -> torch.T
     inner = H * P
     proj = h @ w[p + "in"].T
     z, xbc, dt = proj[:, :inner], proj[:, inner: 2 * inner + 2 * G * N], proj[:, 2 * inner + 2 * G * N:]
-    xbc = silu(causal_conv(xbc, w[p + "conv"], w[p + "conv.b"]))
+    xbc = R(silu(causal_conv(xbc, w[p + "conv"], w[p + "conv.b"])))
     x, B, C = xbc[:, :inner], xbc[:, inner: inner + G * N], xbc[:, inner + G * N:]
     dt = softplus(dt + w[p + "dt_bias"])
     y, _ = ssd_recurrence_fast(x.reshape(T, H, P), B.reshape(T, G, N), C.reshape(T, G, N), dt, w[p + "A_log"], w[p + "D"])
-    return gated_norm(y.reshape(T, inner), z, m["norm_groups"], cfg["norm"]["eps"], w[p + "norm"]) @ w[p + "o"].T
+    return R(gated_norm(y.reshape(T, inner), z, m["norm_groups"], cfg["norm"]["eps"], w[p + "norm"])) @ w[p + "o"].T
 
 
 # ---- attention
@@ -110,7 +130,7 @@ def window_mask(T: int, size: int) -> torch.Tensor:
 def masked_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, scale: float, visible) -> torch.Tensor:
     """q: (T, H, d), k: (T, H, d), v: (T, H, dv), already per query head. `visible(i, j)`: does position i see key j."""
     T, H, _ = q.shape
-    out = torch.zeros(T, H, v.shape[-1], dtype=F)
+    out = torch.zeros(T, H, v.shape[-1], dtype=q.dtype)
     for i in range(T):
         js = [j for j in range(T) if visible(i, j)]
         for h in range(H):
@@ -129,23 +149,23 @@ def masked_attention_fast(q, k, v, scale, mask):
 def attention(cfg: dict, w: dict, p: str, m: dict, h: torch.Tensor) -> torch.Tensor:
     T = h.shape[0]
     H, G, d, dv, eps = m["heads"], m["kv_heads"], m["dim"], m["vdim"], cfg["norm"]["eps"]
-    q = rms((h @ w[p + "q"].T).view(T, H, d), eps)
-    k = rms((h @ w[p + "k"].T).view(T, G, d), eps)
-    v = (h @ w[p + "v"].T).view(T, G, dv)
+    q = R(rms((h @ w[p + "q"].T).view(T, H, d), eps))
+    k = R(rms((h @ w[p + "k"].T).view(T, G, d), eps))
+    v = R((h @ w[p + "v"].T).view(T, G, dv))
     o = masked_attention_fast(q, k.repeat_interleave(H // G, 1), v.repeat_interleave(H // G, 1), m["scale"],
                               window_mask(T, m["mask"]["size"]))
-    return o.reshape(T, H * dv) @ w[p + "o"].T
+    return R(o.reshape(T, H * dv)) @ w[p + "o"].T
 
 
 # ---- feed-forward
 def dense(w: dict, p: str, h: torch.Tensor) -> torch.Tensor:
-    return (silu(h @ w[p + "gate"].T) * (h @ w[p + "up"].T)) @ w[p + "down"].T
+    return R(silu(h @ w[p + "gate"].T) * (h @ w[p + "up"].T)) @ w[p + "down"].T
 
 
 def expert(w: dict, p: str, h: torch.Tensor, limit: float) -> torch.Tensor:
     g = torch.clamp(h @ w[p + "gate"].T, max=limit)
     u = torch.clamp(h @ w[p + "up"].T, -limit, limit)
-    return (g * sigmoid(GATE_SHARPNESS * g) * (u + 1.0)) @ w[p + "down"].T
+    return R(g * sigmoid(GATE_SHARPNESS * g) * (u + 1.0)) @ w[p + "down"].T
 
 
 def route(z: torch.Tensor, correction: torch.Tensor, top: int, groups: int, keep: int, scale: float):
@@ -171,7 +191,7 @@ def route(z: torch.Tensor, correction: torch.Tensor, top: int, groups: int, keep
 def mixture(w: dict, p: str, mlp: dict, h: torch.Tensor) -> torch.Tensor:
     r = mlp["router"]
     idx, wt = route(h @ w[p + "router"].T, w[p + "correction"], r["top"], r["groups"]["count"], r["groups"]["keep"], r["scale"])
-    out = torch.zeros(h.shape[0], w[p + "e0.down"].shape[0], dtype=F)
+    out = torch.zeros(h.shape[0], w[p + "e0.down"].shape[0], dtype=h.dtype)
     for e in range(r["experts"]):
         rows, n = torch.nonzero(idx == e, as_tuple=True)
         if len(rows):
@@ -202,12 +222,12 @@ def forward(cfg: dict, w: dict, tokens: list[int], layers: bool = False):
         L, p = cfg["layers"][n], f"l{n}."
         if again:
             x = x + x0
-        h = layer_norm(x, w[p + "norm1"], eps)
+        h = R(layer_norm(x, w[p + "norm1"], eps))
         mixer = attention if L["type"] == "attention" else state_space
         x = x + mixer(cfg, w, p + "mix.", L["mixer"], h)
         if L.get("mlp") is not None:
-            h = layer_norm(x, w[p + "norm2"], eps)
+            h = R(layer_norm(x, w[p + "norm2"], eps))
             x = x + (dense(w, p + "mlp.", h) if L["mlp"]["kind"] == "dense" else mixture(w, p + "mlp.", L["mlp"], h))
         streams.append(x)
-    logits = layer_norm(x, w["final.norm"], eps) @ w["embed"].T
+    logits = R(layer_norm(x, w["final.norm"], eps)) @ w["embed"].T
     return (logits, torch.stack(streams)) if layers else logits

@@ -731,6 +731,10 @@ class PlainOpsSpace(PlainOpsGated):
         w = weight.float() if weight is not None else torch.ones(1)
         out.copy_((y * (w.repeat(heads) if w.shape[0] == value_dim and heads > 1 else w)).to(out.dtype))
 
+    def check_ssd_scan(self, heads, groups, state_dim, value_dim) -> None:
+        if heads % groups:
+            raise ValueError("bad state space sizes")
+
     def ssd_scan(self, xbc, heads, groups, state_dim, value_dim, dt, dt_offset, dt_bias, a_log, skip, state, meta, out) -> None:
         H, G, N, P = heads, groups, state_dim, value_dim
         out.zero_()

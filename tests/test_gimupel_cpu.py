@@ -195,8 +195,8 @@ def test_the_embedding_is_added_again_once_per_later_pass(dirs):
     assert rel_rms(without, ref) > 0.05
 
 
-def test_a_depth_averaged_stream_may_stand_before_an_added_embedding():
-    """The engine resolves whatever is pending before it adds the kept embedding (a generic schedule, not one design's)."""
+def test_a_pending_sum_resolves_to_its_other_stream():
+    """What a norm that cannot take both streams in its own pass does with them."""
     from fusezap_core_b200.parts import PendingSum
 
     class Ctx:
