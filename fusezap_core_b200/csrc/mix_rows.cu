@@ -314,6 +314,78 @@ short_conv_vec_kernel(const TI* __restrict__ h, int ld, const T* __restrict__ w,
   st8(out + (size_t)n * C + c0, acc);
 }
 
+// The same for steps of many rows: a thread takes CONV_ROWS rows in a row and keeps the inputs that the next one needs, so
+// that an input is read about once (the first of a thread's rows, and the first row of another portion, read their own).
+constexpr int CONV_ROWS = 4;
+template <typename TI, typename T, int TAPS>
+__global__ void __launch_bounds__(128)
+short_conv_rows_kernel(const TI* __restrict__ h, int ld, const T* __restrict__ w, const float* __restrict__ state,
+                       const int* __restrict__ seg, const int* __restrict__ seq_row, T* __restrict__ out, int N, int C,
+                       int residual, int act, const float* __restrict__ bias) {
+  fz_grid_launch_dependents();
+  const int n0 = blockIdx.x * CONV_ROWS;
+  const int c0 = (blockIdx.y * blockDim.x + threadIdx.x) * 8;
+  float wv[8 * TAPS], bv[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+  if (c0 < C) {                          // weights and bias depend on no kernel of the step
+#pragma unroll
+    for (int m = 0; m < TAPS; ++m) ld8(w + (size_t)c0 * TAPS + 8 * m, wv + 8 * m);
+    if (bias != nullptr) ld8(bias + c0, bv);
+  }
+  fz_grid_wait();
+  if (c0 >= C) return;
+  float in[CONV_ROWS][8], past[TAPS - 1][8];
+#pragma unroll
+  for (int r = 0; r < CONV_ROWS; ++r) {
+    if (n0 + r < N) ld8(h + (size_t)(n0 + r) * ld + c0, in[r]);
+  }
+  int last = -1;
+#pragma unroll
+  for (int r = 0; r < CONV_ROWS; ++r) {
+    const int n = n0 + r;
+    if (n >= N) break;
+    const int s = seq_row[n];
+    float acc[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+    if (s >= 0) {
+      if (s != last) {                   // the inputs before this row: the portion's own rows, then the request's state
+        const int row0 = seg[4 * s], slot = seg[4 * s + 3];
+        const float* st = state != nullptr && slot >= 0 ? state + (size_t)slot * (TAPS - 1) * C : nullptr;
+#pragma unroll
+        for (int j = 0; j < TAPS - 1; ++j) {
+          const int k = n - row0 - (TAPS - 1) + j;
+          if (k >= 0) ld8(h + (size_t)(row0 + k) * ld + c0, past[j]);
+          else if (st != nullptr) ld8(st + (size_t)(TAPS - 1 + k) * C + c0, past[j]);
+          else {
+#pragma unroll
+            for (int e = 0; e < 8; ++e) past[j][e] = 0.f;
+          }
+        }
+      }
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j)
+#pragma unroll
+        for (int e = 0; e < 8; ++e) acc[e] = fmaf(wv[e * TAPS + j], j < TAPS - 1 ? past[j < TAPS - 1 ? j : 0][e] : in[r][e], acc[e]);
+      if (bias != nullptr) {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) acc[e] += bv[e];
+      }
+      if (residual) {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) acc[e] += in[r][e];
+      }
+      if (act) {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) acc[e] = acc[e] * (1.0f / (1.0f + expf(-acc[e])));
+      }
+#pragma unroll
+      for (int j = 0; j < TAPS - 1; ++j)
+#pragma unroll
+        for (int e = 0; e < 8; ++e) past[j][e] = j + 1 < TAPS - 1 ? past[j + 1 < TAPS - 1 ? j + 1 : j][e] : in[r][e];
+    }
+    last = s;
+    st8(out + (size_t)n * C + c0, acc);
+  }
+}
+
 // After the convolution has read the old state: the state of every portion's request becomes its last taps - 1 inputs
 // (the portion's own rows, and what is left of the old state when the portion is shorter than taps - 1). A thread owns
 // one channel of one portion, reads all it needs and then writes. grid (portions, channel blocks).
@@ -481,12 +553,19 @@ int launch_conv(const TI* h, int ld, const T* w, float* state, const int* seg, c
     const dim3 grid(N, (C / 8 + 127) / 128);
     const bool w_ok = ((uintptr_t)w & 15) == 0;       // the grouped weight loads want 16-byte aligned rows of 8 x taps values
 #define FZ_CV(K) fz_launch(short_conv_vec_kernel<TI, T, K>, grid, dim3(128), 0, stream, h, ld, w, state, seg, seq_row, out, C, taps, residual, act, bias, single)
-    if (w_ok && taps == 2) FZ_CV(2);
+    // steps of hundreds of rows: several rows per thread (a row's bits are the same)
+#define FZ_CR(K) fz_launch(short_conv_rows_kernel<TI, T, K>, dim3((N + CONV_ROWS - 1) / CONV_ROWS, grid.y), dim3(128), 0, stream, h, ld, w, state, seg, seq_row, out, N, C, residual, act, bias)
+    const bool many = w_ok && N >= 256 && !single;
+    if (many && taps == 2) FZ_CR(2);
+    else if (many && taps == 3) FZ_CR(3);
+    else if (many && taps == 4) FZ_CR(4);
+    else if (w_ok && taps == 2) FZ_CV(2);
     else if (w_ok && taps == 3) FZ_CV(3);
     else if (w_ok && taps == 4) FZ_CV(4);
     else if (w_ok && taps == 5) FZ_CV(5);
     else if (w_ok && taps == 8) FZ_CV(8);
     else FZ_CV(0);
+#undef FZ_CR
 #undef FZ_CV
   } else {
     fz_launch(short_conv_kernel<TI, T>, dim3(N, (C + 255) / 256), dim3(256), 0, stream, h, ld, w, state, seg, seq_row, out, C, taps,

@@ -10,18 +10,28 @@
 // the sum of two bfloat16 numbers, its rounding and the rounding of what is left, and both are multiplied: a relative
 // error of 2^-17 per term.
 //
-// A block owns PB value columns of one head of one portion. Warps 0 .. 3 compute the results of a chunk (16 tokens each),
-// warps 4 .. 7 the state after it (rows 16 (warp - 4 + 4 i) of the state each) and leave it as operands for the next
-// chunk's results; one barrier per chunk. The next chunk's rows travel by cp.async meanwhile.
+// A block owns PB value columns of one head of one portion. Eight warps compute the results of a chunk: a warp takes 16
+// tokens and half of what they need, first every second 16 x 16 tile of the weighted C . B (left in shared memory as
+// operands), then half of the value columns. Eight others compute the state after the chunk: first the weighted x (left in
+// shared memory as operands), then units of 16 state rows x 16 columns, which they leave as operands for the next chunk's
+// results. Each group has a barrier between its two halves, the block one per chunk. The next chunk's rows travel by
+// cp.async meanwhile.
 #include "attn_mma.cuh"
 #include <math.h>
 
 namespace {
 using namespace fzattn;
 constexpr int Q = 64;                       // tokens per chunk
-constexpr int SSD_THREADS = 256;
+constexpr int SSD_THREADS = 512;        // eight warps for the results, eight for the state
 constexpr float LOG2E = 1.4426950408889634f;
 
+// 2^x for x <= 0 (results below the normal range are zero)
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ void group_barrier(int id) { asm volatile("bar.sync %0, 256;" ::"r"(id) : "memory"); }
 __device__ __forceinline__ float softplus32(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
 
 // Two 32-bit values as bfloat16 pairs: their roundings, and the roundings of what is left.
@@ -48,8 +58,9 @@ struct SsdChunkArgs {
 
 __host__ __device__ constexpr int pad_units(int n) { return n + 8; }      // an odd number of 16-byte units per row: no bank conflicts
 
-// PB: value columns per block (16 or 32). MT: state rows / 64, rounded up (1, 2 or 4). grid (portions, heads, P / PB).
-template <int PB, int MT>
+// PB: value columns per block (16 or 32). UM: units of 16 state rows x 16 columns per warp (1 or 2). grid (portions, heads,
+// P / PB).
+template <int PB, int UM>
 __global__ void __launch_bounds__(SSD_THREADS)
 ssd_chunk_kernel(const SsdChunkArgs p) {
   fz_grid_launch_dependents();
@@ -60,12 +71,14 @@ ssd_chunk_kernel(const SsdChunkArgs p) {
   if (cnt < p.min_rows || cnt <= 0 || slot < 0) return;
   extern __shared__ __align__(16) unsigned char smem_raw[];
   const int N = p.N, KN = N >> 4, SN = pad_units(N);
-  constexpr int SP = PB + 8;
+  constexpr int SP = pad_units(PB), SQ = pad_units(Q), NT = PB / 16;      // NT: 8-column tiles per result warp
   __nv_bfloat16* Cs = (__nv_bfloat16*)smem_raw;            // [2][Q][SN]
   __nv_bfloat16* Bs = Cs + 2 * Q * SN;                     // [2][Q][SN]
   __nv_bfloat16* Xs = Bs + 2 * Q * SN;                     // [2][Q][SP]
   __nv_bfloat16* Ms = Xs + 2 * Q * SP;                     // [2][2][N][SP]: the state before a chunk, rounding and rest
-  float* scal = (float*)(Ms + 4 * N * SP);                 // [2][4][Q]: L in powers of two, exp(L), d, exp(L_last - L) d
+  __nv_bfloat16* Gs = Ms + 4 * N * SP;                     // [2][Q][SQ]: the weighted C . B, rounding and rest
+  __nv_bfloat16* Ws = Gs + 2 * Q * SQ;                     // [2][Q][SP]: the weighted x, rounding and rest
+  float* scal = (float*)(Ws + 2 * Q * SP);                 // [2][4][Q]: L in powers of two, exp(L), d, exp(L_last - L) d
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int gq = lane >> 2, q2 = (lane & 3) * 2;           // an accumulator's row (and row + 8) and first column
   const int g = h / (p.H / p.G);
@@ -73,15 +86,15 @@ ssd_chunk_kernel(const SsdChunkArgs p) {
   const size_t off_x = (size_t)h * p.P + p0, off_b = (size_t)p.H * p.P + (size_t)g * N, off_c = off_b + (size_t)p.G * N;
 
   auto load_chunk = [&](int c) {
-    const int st = c & 1, r = tid >> 2;                    // four threads per token
+    const int st = c & 1, r = tid >> 3;                    // eight threads per token
     const bool ok = c * Q + r < cnt;
     const __nv_bfloat16* in = p.xbc + (size_t)(row0 + (ok ? c * Q + r : 0)) * p.W;
     const uint32_t dc = smem_u32(Cs + (st * Q + r) * SN), db = smem_u32(Bs + (st * Q + r) * SN), dx = smem_u32(Xs + (st * Q + r) * SP);
-    for (int j = tid & 3; j < 2 * KN; j += 4) {
+    for (int j = tid & 7; j < 2 * KN; j += 8) {
       cp_async16(dc + 16 * j, in + off_c + 8 * j, ok);
       cp_async16(db + 16 * j, in + off_b + 8 * j, ok);
     }
-    for (int j = tid & 3; j < PB / 8; j += 4) cp_async16(dx + 16 * j, in + off_x + 8 * j, ok);
+    if ((tid & 7) < PB / 8) cp_async16(dx + 16 * (tid & 7), in + off_x + 8 * (tid & 7), ok);
     cp_async_commit();
   };
   // the scalars of a chunk, two tokens per lane of one warp; r0, r1: the tokens' raw step sizes
@@ -106,22 +119,23 @@ ssd_chunk_kernel(const SsdChunkArgs p) {
     const float l0 = before + a0, l1 = incl;
     float* sc = scal + (c & 1) * 4 * Q + 2 * lane;
     *(float2*)sc = make_float2(l0, l1);
-    *(float2*)(sc + Q) = make_float2(exp2f(l0), exp2f(l1));
+    *(float2*)(sc + Q) = make_float2(ex2(l0), ex2(l1));
     *(float2*)(sc + 2 * Q) = make_float2(d0, d1);
-    *(float2*)(sc + 3 * Q) = make_float2(exp2f(last - l0) * d0, exp2f(last - l1) * d1);
+    *(float2*)(sc + 3 * Q) = make_float2(ex2(last - l0) * d0, ex2(last - l1) * d1);
   };
 
-  float S[MT][PB / 8][4];                                  // warps 4 .. 7: the state's rows 16 (warp - 4 + 4 i)
+  const int sw = warp - 8;                                 // of the warps that keep the state: units sw, sw + 8, ...
+  float S[UM][2][4];                                       // a unit: rows 16 (u % KN), columns 16 (u / KN)
   auto leave_state = [&](int buf) {
     __nv_bfloat16* hi = Ms + (size_t)buf * 2 * N * SP;
     __nv_bfloat16* lo = hi + (size_t)N * SP;
 #pragma unroll
-    for (int i = 0; i < MT; ++i) {
-      const int mt = warp - 4 + 4 * i;
-      if (mt >= KN) continue;
+    for (int i = 0; i < UM; ++i) {
+      const int u = sw + 8 * i;
+      if (u >= KN * NT) break;
 #pragma unroll
-      for (int n = 0; n < PB / 8; ++n) {
-        const int at = (16 * mt + gq) * SP + 8 * n + q2;
+      for (int n = 0; n < 2; ++n) {
+        const int at = (16 * (u % KN) + gq) * SP + 16 * (u / KN) + 8 * n + q2;
         uint32_t a, b;
         split2(S[i][n][0], S[i][n][1], a, b);
         *(uint32_t*)(hi + at) = a; *(uint32_t*)(lo + at) = b;
@@ -130,22 +144,23 @@ ssd_chunk_kernel(const SsdChunkArgs p) {
       }
     }
   };
-  float* sp = p.state + ((size_t)slot * p.H + h) * p.P * p.npad;
+  float* sp = p.state + (((size_t)slot * p.H + h) * p.P + p0) * p.npad;
+  auto state_at = [&](int u, int n, int e) {
+    return (size_t)(16 * (u / KN) + 8 * n + q2 + (e & 1)) * p.npad + 16 * (u % KN) + gq + (e & 2) * 4;
+  };
 
   load_chunk(0);
-  if (warp >= 4) {
+  if (sw >= 0) {
 #pragma unroll
-    for (int i = 0; i < MT; ++i) {
-      const int mt = warp - 4 + 4 * i;
+    for (int i = 0; i < UM; ++i) {
+      const int u = sw + 8 * i;
 #pragma unroll
-      for (int n = 0; n < PB / 8; ++n) {
+      for (int n = 0; n < 2; ++n)
 #pragma unroll
-        for (int e = 0; e < 4; ++e)
-          S[i][n][e] = mt < KN ? sp[(size_t)(p0 + 8 * n + q2 + (e & 1)) * p.npad + 16 * mt + gq + (e & 2) * 4] : 0.f;
-      }
+        for (int e = 0; e < 4; ++e) S[i][n][e] = u < KN * NT ? sp[state_at(u, n, e)] : 0.f;
     }
     leave_state(0);
-    if (warp == 7) {
+    if (sw == 7) {
       float r0, r1;
       raw_steps(0, r0, r1);
       scalars(0, r0, r1);
@@ -162,161 +177,184 @@ ssd_chunk_kernel(const SsdChunkArgs p) {
     const __nv_bfloat16* Bc = Bs + st * Q * SN;
     const __nv_bfloat16* Xc = Xs + st * Q * SP;
     const float* sc = scal + st * 4 * Q;
-    if (warp < 4) {
-      if (16 * warp < valid) {
-        float G[8][4], Y[PB / 8][4];
+    if (sw < 0) {
+      const int rt = warp >> 1, half = warp & 1;           // 16 tokens; which tiles and which columns
+      const bool live = 16 * rt < valid;
+      const int ta = 16 * rt + gq, tb = ta + 8;            // this thread's two tokens
+      float Y[NT][4];
 #pragma unroll
-        for (int j = 0; j < 8; ++j)
+      for (int n = 0; n < NT; ++n)
 #pragma unroll
-          for (int e = 0; e < 4; ++e) G[j][e] = 0.f;
+        for (int e = 0; e < 4; ++e) Y[n][e] = 0.f;
+      if (live) {
+        float G[2][2][4];                                  // tiles half and half + 2
 #pragma unroll
-        for (int n = 0; n < PB / 8; ++n)
+        for (int i = 0; i < 2; ++i)
 #pragma unroll
-          for (int e = 0; e < 4; ++e) Y[n][e] = 0.f;
-        const __nv_bfloat16* hi = Ms + (size_t)st * 2 * N * SP;
-        const uint32_t ac = smem_u32(Cc + (16 * warp + (lane & 15)) * SN + 8 * (lane >> 4));
-        const uint32_t ab = smem_u32(Bc + (((lane >> 4) << 3) + (lane & 7)) * SN + 8 * ((lane >> 3) & 1));
-        const uint32_t am = smem_u32(hi + (lane & 15) * SP + 8 * (lane >> 4));
-        const uint32_t rest = (uint32_t)(N * SP * 2);
-#pragma unroll 2
+          for (int u = 0; u < 2; ++u)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) G[i][u][e] = 0.f;
+        const uint32_t ac = smem_u32(Cc + (16 * rt + (lane & 15)) * SN + 8 * (lane >> 4));
+        const uint32_t ab = smem_u32(Bc + (16 * half + ((lane >> 4) << 3) + (lane & 7)) * SN + 8 * ((lane >> 3) & 1));
+        // the state's rounding and rest in one load: lanes 0 .. 15 the rounding's rows, 16 .. 31 the rest's
+        const uint32_t am = smem_u32(Ms + ((size_t)st * 2 + (lane >> 4)) * N * SP + (lane & 15) * SP + 8 * NT * half);
+#pragma unroll 4
         for (int k = 0; k < KN; ++k) {
           uint32_t a[4], b[4];
           ldmatrix_x4(a, ac + 32 * k);
 #pragma unroll
-          for (int j = 0; j < 4; ++j) {
-            if (j > warp) break;                           // tokens after this warp's: not seen
-            ldmatrix_x4(b, ab + (16 * j * SN) * 2 + 32 * k);
-            mma_bf16(G[2 * j], a, b[0], b[1]);
-            mma_bf16(G[2 * j + 1], a, b[2], b[3]);
+          for (int i = 0; i < 2; ++i) {
+            if (half + 2 * i > rt) break;                  // tokens after this warp's: not seen
+            ldmatrix_x4(b, ab + (32 * i * SN) * 2 + 32 * k);
+            mma_bf16(G[i][0], a, b[0], b[1]);
+            mma_bf16(G[i][1], a, b[2], b[3]);
           }
 #pragma unroll
-          for (int n = 0; n < PB / 16; ++n) {
-            const uint32_t at = am + (16 * k * SP) * 2 + 32 * n;
-            ldmatrix_x4_trans(b, at);
-            mma_bf16(Y[2 * n], a, b[0], b[1]);
-            mma_bf16(Y[2 * n + 1], a, b[2], b[3]);
-            ldmatrix_x4_trans(b, at + rest);
-            mma_bf16(Y[2 * n], a, b[0], b[1]);
-            mma_bf16(Y[2 * n + 1], a, b[2], b[3]);
+          for (int n = 0; n < NT; ++n) {
+            ldmatrix_x4_trans(b, am + (16 * k * SP) * 2 + 16 * n);
+            mma_bf16(Y[n], a, b[0], b[1]);
+            mma_bf16(Y[n], a, b[2], b[3]);
           }
         }
-        const int ta = 16 * warp + gq, tb = ta + 8;        // this thread's two tokens
         const float la = sc[ta], lb = sc[tb], ea = sc[Q + ta], eb = sc[Q + tb];
 #pragma unroll
-        for (int n = 0; n < PB / 8; ++n) { Y[n][0] *= ea; Y[n][1] *= ea; Y[n][2] *= eb; Y[n][3] *= eb; }
-        const uint32_t ax = smem_u32(Xc + (lane & 15) * SP + 8 * (lane >> 4));
+        for (int n = 0; n < NT; ++n) { Y[n][0] *= ea; Y[n][1] *= ea; Y[n][2] *= eb; Y[n][3] *= eb; }
 #pragma unroll
-        for (int j = 0; j < 4; ++j) {
-          if (j > warp) break;
-          uint32_t hi4[4], lo4[4];
+        for (int i = 0; i < 2; ++i) {
+          const int j = half + 2 * i;
+          if (j > rt) break;
 #pragma unroll
           for (int u = 0; u < 2; ++u) {
             const int t = 16 * j + 8 * u + q2;             // the earlier tokens of this thread's columns: t, t + 1
             const float2 l = *(const float2*)(sc + t), d = *(const float2*)(sc + 2 * Q + t);
-            const float* w = G[2 * j + u];
-            const float w0 = t <= ta ? w[0] * (exp2f(la - l.x) * d.x) : 0.f, w1 = t + 1 <= ta ? w[1] * (exp2f(la - l.y) * d.y) : 0.f;
-            const float w2 = t <= tb ? w[2] * (exp2f(lb - l.x) * d.x) : 0.f, w3 = t + 1 <= tb ? w[3] * (exp2f(lb - l.y) * d.y) : 0.f;
-            split2(w0, w1, hi4[2 * u], lo4[2 * u]);
-            split2(w2, w3, hi4[2 * u + 1], lo4[2 * u + 1]);
+            const float* w = G[i][u];
+            const float w0 = t <= ta ? w[0] * (ex2(la - l.x) * d.x) : 0.f, w1 = t + 1 <= ta ? w[1] * (ex2(la - l.y) * d.y) : 0.f;
+            const float w2 = t <= tb ? w[2] * (ex2(lb - l.x) * d.x) : 0.f, w3 = t + 1 <= tb ? w[3] * (ex2(lb - l.y) * d.y) : 0.f;
+            uint32_t hi, lo;
+            split2(w0, w1, hi, lo);
+            *(uint32_t*)(Gs + ta * SQ + t) = hi; *(uint32_t*)(Gs + (Q + ta) * SQ + t) = lo;
+            split2(w2, w3, hi, lo);
+            *(uint32_t*)(Gs + tb * SQ + t) = hi; *(uint32_t*)(Gs + (Q + tb) * SQ + t) = lo;
           }
+        }
+      }
+      group_barrier(1);
+      if (live) {
+        const uint32_t ag = smem_u32(Gs + (16 * rt + (lane & 15)) * SQ + 8 * (lane >> 4));
+        const uint32_t ax = smem_u32(Xc + lane * SP + 8 * NT * half);      // 32 tokens of one 8-column tile per load
 #pragma unroll
-          for (int n = 0; n < PB / 16; ++n) {
-            uint32_t b[4];
-            ldmatrix_x4_trans(b, ax + (16 * j * SP) * 2 + 32 * n);
-            mma_bf16(Y[2 * n], hi4, b[0], b[1]);
-            mma_bf16(Y[2 * n + 1], hi4, b[2], b[3]);
-            mma_bf16(Y[2 * n], lo4, b[0], b[1]);
-            mma_bf16(Y[2 * n + 1], lo4, b[2], b[3]);
+        for (int jj = 0; jj < 2; ++jj) {
+          if (2 * jj > rt) break;
+          uint32_t b[NT][4];
+#pragma unroll
+          for (int n = 0; n < NT; ++n) ldmatrix_x4_trans(b[n], ax + (32 * jj * SP) * 2 + 16 * n);
+#pragma unroll
+          for (int u = 0; u < 2; ++u) {
+            const int j = 2 * jj + u;
+            if (j > rt) break;
+            uint32_t hi[4], lo[4];
+            ldmatrix_x4(hi, ag + 32 * j);
+            ldmatrix_x4(lo, ag + (Q * SQ) * 2 + 32 * j);
+#pragma unroll
+            for (int n = 0; n < NT; ++n) {
+              mma_bf16(Y[n], hi, b[n][2 * u], b[n][2 * u + 1]);
+              mma_bf16(Y[n], lo, b[n][2 * u], b[n][2 * u + 1]);
+            }
           }
         }
         const size_t ld = (size_t)p.H * p.P;
-        float* dst = p.out + (size_t)(row0 + c * Q) * ld + off_x + q2;
+        const int col = 8 * NT * half + q2;
+        float* dst = p.out + (size_t)(row0 + c * Q) * ld + off_x + col;
 #pragma unroll
-        for (int n = 0; n < PB / 8; ++n) {
+        for (int n = 0; n < NT; ++n) {
           if (ta < valid) {
-            const float2 x = unpack2(*(const uint32_t*)(Xc + ta * SP + 8 * n + q2));
+            const float2 x = unpack2(*(const uint32_t*)(Xc + ta * SP + col + 8 * n));
             *(float2*)(dst + ta * ld + 8 * n) = make_float2(fmaf(D, x.x, Y[n][0]), fmaf(D, x.y, Y[n][1]));
           }
           if (tb < valid) {
-            const float2 x = unpack2(*(const uint32_t*)(Xc + tb * SP + 8 * n + q2));
+            const float2 x = unpack2(*(const uint32_t*)(Xc + tb * SP + col + 8 * n));
             *(float2*)(dst + tb * ld + 8 * n) = make_float2(fmaf(D, x.x, Y[n][2]), fmaf(D, x.y, Y[n][3]));
           }
         }
       }
     } else {
       float r0 = 0.f, r1 = 0.f;
-      if (warp == 7 && more) raw_steps(c + 1, r0, r1);
+      if (sw == 7 && more) raw_steps(c + 1, r0, r1);
+      {                                                    // the weighted x: four threads per token, PB / 4 columns each
+        const int t = (tid - 256) >> 2, c0 = (tid & 3) * (PB / 4);
+        const float w = sc[3 * Q + t];
+#pragma unroll
+        for (int i = 0; i < PB / 16; ++i) {
+          const int at = t * SP + c0 + 4 * i;
+          const uint2 v = *(const uint2*)(Xc + at);
+          const float2 a = unpack2(v.x), b = unpack2(v.y);
+          uint2 hi, lo;
+          split2(a.x * w, a.y * w, hi.x, lo.x);
+          split2(b.x * w, b.y * w, hi.y, lo.y);
+          *(uint2*)(Ws + at) = hi;
+          *(uint2*)(Ws + Q * SP + at) = lo;
+        }
+      }
       const float all = sc[Q + Q - 1];                     // exp(L_last): tokens past the end decay nothing
 #pragma unroll
-      for (int i = 0; i < MT; ++i)
+      for (int i = 0; i < UM; ++i)
 #pragma unroll
-        for (int n = 0; n < PB / 8; ++n)
+        for (int n = 0; n < 2; ++n)
 #pragma unroll
           for (int e = 0; e < 4; ++e) S[i][n][e] *= all;
-      const uint32_t ax = smem_u32(Xc + (lane & 15) * SP + 8 * (lane >> 4));
+      group_barrier(2);
+      const uint32_t aw = smem_u32(Ws + (lane & 15) * SP + 8 * (lane >> 4));
       const uint32_t at = smem_u32(Bc + (((lane >> 4) << 3) + (lane & 7)) * SN + 8 * ((lane >> 3) & 1));
 #pragma unroll
       for (int k = 0; k < Q / 16; ++k) {
         if (16 * k >= valid) break;
-        const float2 wa = *(const float2*)(sc + 3 * Q + 16 * k + q2), wb = *(const float2*)(sc + 3 * Q + 16 * k + 8 + q2);
-        uint32_t xh[PB / 8][2], xl[PB / 8][2];
 #pragma unroll
-        for (int n = 0; n < PB / 16; ++n) {
-          uint32_t b[4];
-          ldmatrix_x4_trans(b, ax + (16 * k * SP) * 2 + 32 * n);
-#pragma unroll
-          for (int u = 0; u < 2; ++u) {
-            const float2 va = unpack2(b[2 * u]), vb = unpack2(b[2 * u + 1]);
-            split2(va.x * wa.x, va.y * wa.y, xh[2 * n + u][0], xl[2 * n + u][0]);
-            split2(vb.x * wb.x, vb.y * wb.y, xh[2 * n + u][1], xl[2 * n + u][1]);
-          }
-        }
-#pragma unroll
-        for (int i = 0; i < MT; ++i) {
-          const int mt = warp - 4 + 4 * i;
-          if (mt >= KN) break;
-          uint32_t a[4];
-          ldmatrix_x4_trans(a, at + (16 * k * SN) * 2 + 32 * mt);
-#pragma unroll
-          for (int n = 0; n < PB / 8; ++n) {
-            mma_bf16(S[i][n], a, xh[n][0], xh[n][1]);
-            mma_bf16(S[i][n], a, xl[n][0], xl[n][1]);
-          }
+        for (int i = 0; i < UM; ++i) {
+          const int u = sw + 8 * i;
+          if (u >= KN * NT) break;
+          uint32_t a[4], b[4];
+          ldmatrix_x4_trans(a, at + (16 * k * SN) * 2 + 32 * (u % KN));
+          ldmatrix_x4_trans(b, aw + (16 * k * SP) * 2 + 32 * (u / KN));
+          mma_bf16(S[i][0], a, b[0], b[1]);
+          mma_bf16(S[i][1], a, b[2], b[3]);
+          ldmatrix_x4_trans(b, aw + ((Q + 16 * k) * SP) * 2 + 32 * (u / KN));
+          mma_bf16(S[i][0], a, b[0], b[1]);
+          mma_bf16(S[i][1], a, b[2], b[3]);
         }
       }
       if (more) {
         leave_state(st ^ 1);
-        if (warp == 7) scalars(c + 1, r0, r1);
+        if (sw == 7) scalars(c + 1, r0, r1);
       }
     }
     cp_async_wait<0>();
     __syncthreads();
   }
-  if (warp >= 4) {
+  if (sw >= 0) {
 #pragma unroll
-    for (int i = 0; i < MT; ++i) {
-      const int mt = warp - 4 + 4 * i;
-      if (mt >= KN) continue;
+    for (int i = 0; i < UM; ++i) {
+      const int u = sw + 8 * i;
+      if (u >= KN * NT) break;
 #pragma unroll
-      for (int n = 0; n < PB / 8; ++n)
+      for (int n = 0; n < 2; ++n)
 #pragma unroll
-        for (int e = 0; e < 4; ++e)
-          sp[(size_t)(p0 + 8 * n + q2 + (e & 1)) * p.npad + 16 * mt + gq + (e & 2) * 4] = S[i][n][e];
+        for (int e = 0; e < 4; ++e) sp[state_at(u, n, e)] = S[i][n][e];
     }
   }
 }
 
-template <int PB, int MT>
+template <int PB, int UM>
 int launch_chunk(const SsdChunkArgs& a, int n_seg, cudaStream_t stream) {
-  const size_t smem = 2 * (4 * (size_t)Q * pad_units(a.N) + 2 * Q * (PB + 8) + 4 * (size_t)a.N * (PB + 8)) + sizeof(float) * 8 * Q;
+  const size_t smem = 2 * (4 * (size_t)Q * pad_units(a.N) + 4 * Q * pad_units(PB) + 4 * (size_t)a.N * pad_units(PB) + 2 * Q * pad_units(Q)) +
+                      sizeof(float) * 8 * Q;
   static size_t allowed = 48 * 1024;
   if (smem > allowed) {
     if (smem > 227 * 1024) return FZ_TOO_LARGE;
-    cudaError_t e = cudaFuncSetAttribute(ssd_chunk_kernel<PB, MT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t e = cudaFuncSetAttribute(ssd_chunk_kernel<PB, UM>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
     allowed = smem;
   }
-  fz_launch(ssd_chunk_kernel<PB, MT>, dim3(n_seg, a.H, a.P / PB), dim3(SSD_THREADS), smem, stream, a);
+  fz_launch(ssd_chunk_kernel<PB, UM>, dim3(n_seg, a.H, a.P / PB), dim3(SSD_THREADS), smem, stream, a);
   FZ_LAUNCH_CHECK();
   return FZ_OK;
 }
@@ -337,13 +375,9 @@ FZ_API int fz_ssd_chunk(const void* xbc, int H, int G, int N, int P, const float
   if (npad < N || ((uintptr_t)out & 7)) return FZ_BAD_SHAPE;
   const SsdChunkArgs a = {(const __nv_bfloat16*)xbc, H * P + 2 * G * N, H, G, N, P, dt, ldt, off_dt, dt_bias, a_log, skip, state, npad,
                           seg, min_rows, out};
-  if (P % 32 == 0 && N <= 128) {
-    if (N <= 64) return launch_chunk<32, 1>(a, n_seg, stream);
-    return launch_chunk<32, 2>(a, n_seg, stream);
-  }
-  if (N <= 64) return launch_chunk<16, 1>(a, n_seg, stream);
-  if (N <= 128) return launch_chunk<16, 2>(a, n_seg, stream);
-  return launch_chunk<16, 4>(a, n_seg, stream);
+  // units of 16 state rows x 16 columns: N / 16 * PB / 16, eight warps
+  if (P % 32 == 0 && N <= 128) return N <= 64 ? launch_chunk<32, 1>(a, n_seg, stream) : launch_chunk<32, 2>(a, n_seg, stream);
+  return N <= 128 ? launch_chunk<16, 1>(a, n_seg, stream) : launch_chunk<16, 2>(a, n_seg, stream);
 }
 
 #ifdef FZ_TIMELINE

@@ -297,6 +297,41 @@ def test_convolution_over_columns_of_a_wider_product(dtype, C, taps, off, width)
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("wide", [True, False])
+@pytest.mark.parametrize("taps", [2, 3, 4])
+def test_convolution_of_steps_of_hundreds_of_rows(dtype, wide, taps):
+    """Portions whose borders fall anywhere among the rows that one thread takes, with single tokens and padding between
+    them: the same bits as the rows of small steps."""
+    ops, g, dt, C, T = cuda_ops(dtype), torch.Generator().manual_seed(taps), DT[dtype], 72, 330
+    width = 96 if wide else C
+    off = 16 if wide else None
+    tin = torch.float32 if wide else dt
+    x = [torch.randn(T, width, generator=g).to(tin) for _ in range(3)]
+    w, b = torch.randn(C, taps, generator=g).to(dt), torch.randn(C, generator=g)
+    outs = []
+    for steps in ([[(0, 0, 201), (1, 0, 1), (2, 0, 102)], [(0, 201, 129), (1, 1, 3), (2, 102, 228)], [(1, 4, 326)]],
+                  [[(r, at, min(50, T - at)) for r in range(3)] for at in range(0, T, 50)]):
+        state = torch.zeros(5, taps - 1, C, device=DEV)
+        got = [torch.zeros(T, C, dtype=dt) for _ in range(3)]
+        for step in steps:
+            meta = Meta([(n, at, (2, 0, 4)[r]) for r, at, n in step], pad=3)
+            rows = torch.cat([x[r][at: at + n] for r, at, n in step] + [torch.zeros(3, width, dtype=tin)]).to(DEV)
+            out = torch.full((meta.n_rows, C), 7.0, dtype=dt, device=DEV)
+            kw = {"offset": off} if wide else {}
+            ops.short_conv(rows, w.to(DEV), state, meta, out, not wide, "silu", bias=b.to(DEV), **kw)
+            assert float(out[-3:].float().abs().max()) == 0.0
+            k = 0
+            for r, at, n in step:
+                got[r][at: at + n] = out[k: k + n].cpu()
+                k += n
+        outs.append(got)
+    for r in range(3):
+        xr = (x[r][:, off: off + C] if wide else x[r]).to(F)
+        close(outs[0][r], plain.silu(plain.causal_conv(xr, w.to(F), b.to(F)) + (0 if wide else xr)), dtype, f"request {r}")
+        assert torch.equal(outs[0][r], outs[1][r])
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 @pytest.mark.parametrize("parts,size,off,extra", [(4, 20, 0, 0), (1, 384, 8, 24), (3, 7, 2, 5), (2, 2048, 0, 64), (1, 4500, 4, 4), (5, 1, 0, 3), (1, 20000, 0, 0), (8, 130, 0, 2)])
 def test_norm_in_parts_with_the_gate_first(dtype, parts, size, off, extra):
     ops, g, n = cuda_ops(dtype), torch.Generator().manual_seed(size), 9
