@@ -177,6 +177,12 @@ add_rmsnorm_groups_vec_kernel(float* __restrict__ x, const float* __restrict__ d
 // seg: (first row, rows, first position, state slot) per portion. state: (slots, taps - 1, C) float32, oldest first. The
 // inputs are C neighbouring columns of rows of ld values of TI (TI = T and ld = C, or a range of a wider float32 product).
 // `single`: every portion of the step is one token; the thread that owns a channel then also moves its state on.
+template <typename T>
+__device__ __forceinline__ float silu32(float z) { return z * (1.0f / (1.0f + expf(-z))); }
+// where the result is rounded to bfloat16: the short exponential and quotient (a few 32-bit roundings off, a fifth of the
+// instructions, which is what bounds these kernels)
+template <>
+__device__ __forceinline__ float silu32<__nv_bfloat16>(float z) { return __fdividef(z, 1.0f + __expf(-z)); }
 template <typename TI>
 __device__ __forceinline__ void conv_state_single(float* __restrict__ st, const TI* __restrict__ own, int C, int taps) {
   for (int m = 0; m + 1 < taps - 1; ++m) st[(size_t)m * C] = st[(size_t)(m + 1) * C];
@@ -213,7 +219,7 @@ short_conv_kernel(const TI* __restrict__ h, int ld, const T* __restrict__ w, flo
     }
     if (bias != nullptr) acc += bias[c];
     if (residual) acc += Cvt<TI>::to_f(h[(size_t)n * ld + c]);
-    if (act) acc = acc * (1.0f / (1.0f + expf(-acc)));      // silu of the 32-bit sum
+    if (act) acc = silu32<T>(acc);      // silu of the 32-bit sum
     orow[c] = Cvt<T>::from_f(acc);
   }
   if (single && st != nullptr && taps > 1) conv_state_single(st + c, h + (size_t)n * ld + c, C, taps);
@@ -299,7 +305,7 @@ short_conv_vec_kernel(const TI* __restrict__ h, int ld, const T* __restrict__ w,
     }
     if (act) {
 #pragma unroll
-      for (int e = 0; e < 8; ++e) acc[e] = acc[e] * (1.0f / (1.0f + expf(-acc[e])));      // silu of the 32-bit sum
+      for (int e = 0; e < 8; ++e) acc[e] = silu32<T>(acc[e]);      // silu of the 32-bit sum
     }
     if (single && st != nullptr && taps > 1) {
       float v[8];
@@ -314,9 +320,24 @@ short_conv_vec_kernel(const TI* __restrict__ h, int ld, const T* __restrict__ w,
   st8(out + (size_t)n * C + c0, acc);
 }
 
-// The same for steps of many rows: a thread takes CONV_ROWS rows in a row and keeps the inputs that the next one needs, so
+// The same for steps of many rows: a thread takes four channels (more leave too few threads per SM to cover the loads) of
+// CONV_ROWS rows in a row and keeps the inputs that the next one needs, so
 // that an input is read about once (the first of a thread's rows, and the first row of another portion, read their own).
 constexpr int CONV_ROWS = 4;
+__device__ __forceinline__ void ldq(const float* p, float* v) {
+  const float4 a = *(const float4*)p;
+  v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+}
+__device__ __forceinline__ void ldq(const __nv_bfloat16* p, float* v) {
+  const uint2 u = *(const uint2*)p;
+  const float2 a = __bfloat1622float2(*(const __nv_bfloat162*)&u.x), b = __bfloat1622float2(*(const __nv_bfloat162*)&u.y);
+  v[0] = a.x; v[1] = a.y; v[2] = b.x; v[3] = b.y;
+}
+__device__ __forceinline__ void stq(float* p, const float* v) { *(float4*)p = make_float4(v[0], v[1], v[2], v[3]); }
+__device__ __forceinline__ void stq(__nv_bfloat16* p, const float* v) {
+  const __nv_bfloat162 a = __floats2bfloat162_rn(v[0], v[1]), b = __floats2bfloat162_rn(v[2], v[3]);
+  *(uint2*)p = make_uint2(*(const uint32_t*)&a, *(const uint32_t*)&b);
+}
 template <typename TI, typename T, int TAPS>
 __global__ void __launch_bounds__(128)
 short_conv_rows_kernel(const TI* __restrict__ h, int ld, const T* __restrict__ w, const float* __restrict__ state,
@@ -324,19 +345,19 @@ short_conv_rows_kernel(const TI* __restrict__ h, int ld, const T* __restrict__ w
                        int residual, int act, const float* __restrict__ bias) {
   fz_grid_launch_dependents();
   const int n0 = blockIdx.x * CONV_ROWS;
-  const int c0 = (blockIdx.y * blockDim.x + threadIdx.x) * 8;
-  float wv[8 * TAPS], bv[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+  const int c0 = (blockIdx.y * blockDim.x + threadIdx.x) * 4;
+  float wv[4 * TAPS], bv[4] = {0.f, 0.f, 0.f, 0.f};
   if (c0 < C) {                          // weights and bias depend on no kernel of the step
 #pragma unroll
-    for (int m = 0; m < TAPS; ++m) ld8(w + (size_t)c0 * TAPS + 8 * m, wv + 8 * m);
-    if (bias != nullptr) ld8(bias + c0, bv);
+    for (int m = 0; m < TAPS; ++m) ldq(w + (size_t)c0 * TAPS + 4 * m, wv + 4 * m);
+    if (bias != nullptr) ldq(bias + c0, bv);
   }
   fz_grid_wait();
   if (c0 >= C) return;
-  float in[CONV_ROWS][8], past[TAPS - 1][8];
+  float in[CONV_ROWS][4], past[TAPS - 1][4];
 #pragma unroll
   for (int r = 0; r < CONV_ROWS; ++r) {
-    if (n0 + r < N) ld8(h + (size_t)(n0 + r) * ld + c0, in[r]);
+    if (n0 + r < N) ldq(h + (size_t)(n0 + r) * ld + c0, in[r]);
   }
   int last = -1;
 #pragma unroll
@@ -344,7 +365,7 @@ short_conv_rows_kernel(const TI* __restrict__ h, int ld, const T* __restrict__ w
     const int n = n0 + r;
     if (n >= N) break;
     const int s = seq_row[n];
-    float acc[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+    float acc[4] = {0.f, 0.f, 0.f, 0.f};
     if (s >= 0) {
       if (s != last) {                   // the inputs before this row: the portion's own rows, then the request's state
         const int row0 = seg[4 * s], slot = seg[4 * s + 3];
@@ -352,37 +373,37 @@ short_conv_rows_kernel(const TI* __restrict__ h, int ld, const T* __restrict__ w
 #pragma unroll
         for (int j = 0; j < TAPS - 1; ++j) {
           const int k = n - row0 - (TAPS - 1) + j;
-          if (k >= 0) ld8(h + (size_t)(row0 + k) * ld + c0, past[j]);
-          else if (st != nullptr) ld8(st + (size_t)(TAPS - 1 + k) * C + c0, past[j]);
+          if (k >= 0) ldq(h + (size_t)(row0 + k) * ld + c0, past[j]);
+          else if (st != nullptr) ldq(st + (size_t)(TAPS - 1 + k) * C + c0, past[j]);
           else {
 #pragma unroll
-            for (int e = 0; e < 8; ++e) past[j][e] = 0.f;
+            for (int e = 0; e < 4; ++e) past[j][e] = 0.f;
           }
         }
       }
 #pragma unroll
       for (int j = 0; j < TAPS; ++j)
 #pragma unroll
-        for (int e = 0; e < 8; ++e) acc[e] = fmaf(wv[e * TAPS + j], j < TAPS - 1 ? past[j < TAPS - 1 ? j : 0][e] : in[r][e], acc[e]);
+        for (int e = 0; e < 4; ++e) acc[e] = fmaf(wv[e * TAPS + j], j < TAPS - 1 ? past[j < TAPS - 1 ? j : 0][e] : in[r][e], acc[e]);
       if (bias != nullptr) {
 #pragma unroll
-        for (int e = 0; e < 8; ++e) acc[e] += bv[e];
+        for (int e = 0; e < 4; ++e) acc[e] += bv[e];
       }
       if (residual) {
 #pragma unroll
-        for (int e = 0; e < 8; ++e) acc[e] += in[r][e];
+        for (int e = 0; e < 4; ++e) acc[e] += in[r][e];
       }
       if (act) {
 #pragma unroll
-        for (int e = 0; e < 8; ++e) acc[e] = acc[e] * (1.0f / (1.0f + expf(-acc[e])));
+        for (int e = 0; e < 4; ++e) acc[e] = silu32<T>(acc[e]);
       }
 #pragma unroll
       for (int j = 0; j < TAPS - 1; ++j)
 #pragma unroll
-        for (int e = 0; e < 8; ++e) past[j][e] = j + 1 < TAPS - 1 ? past[j + 1 < TAPS - 1 ? j + 1 : j][e] : in[r][e];
+        for (int e = 0; e < 4; ++e) past[j][e] = j + 1 < TAPS - 1 ? past[j + 1 < TAPS - 1 ? j + 1 : j][e] : in[r][e];
     }
     last = s;
-    st8(out + (size_t)n * C + c0, acc);
+    stq(out + (size_t)n * C + c0, acc);
   }
 }
 
@@ -554,7 +575,7 @@ int launch_conv(const TI* h, int ld, const T* w, float* state, const int* seg, c
     const bool w_ok = ((uintptr_t)w & 15) == 0;       // the grouped weight loads want 16-byte aligned rows of 8 x taps values
 #define FZ_CV(K) fz_launch(short_conv_vec_kernel<TI, T, K>, grid, dim3(128), 0, stream, h, ld, w, state, seg, seq_row, out, C, taps, residual, act, bias, single)
     // steps of hundreds of rows: several rows per thread (a row's bits are the same)
-#define FZ_CR(K) fz_launch(short_conv_rows_kernel<TI, T, K>, dim3((N + CONV_ROWS - 1) / CONV_ROWS, grid.y), dim3(128), 0, stream, h, ld, w, state, seg, seq_row, out, N, C, residual, act, bias)
+#define FZ_CR(K) fz_launch(short_conv_rows_kernel<TI, T, K>, dim3((N + CONV_ROWS - 1) / CONV_ROWS, (C / 4 + 127) / 128), dim3(128), 0, stream, h, ld, w, state, seg, seq_row, out, N, C, residual, act, bias)
     const bool many = w_ok && N >= 256 && !single;
     if (many && taps == 2) FZ_CR(2);
     else if (many && taps == 3) FZ_CR(3);

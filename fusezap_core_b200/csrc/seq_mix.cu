@@ -945,8 +945,10 @@ head_norm_gate_kernel(const float* __restrict__ o, int H, int dv, const float* _
 // The gate before the norm: u = o * act(gate), out = u / sqrt(mean_c u^2 + eps) * w, a block per (row, part of dv values).
 // Vectorised where dv is a multiple of four, at most 4 * VPT values per thread, and everything is 16-byte aligned: a thread
 // keeps its values in registers; else every value is computed twice.
+// Where the result is rounded to bfloat16 the sigmoid takes the short exponential and quotient (a few 32-bit roundings off).
+template <typename TO>
 __device__ __forceinline__ float gated(float o, float z, int act) {
-  const float sg = 1.0f / (1.0f + expf(-z));
+  const float sg = sizeof(TO) == 2 ? __fdividef(1.0f, 1.0f + __expf(-z)) : 1.0f / (1.0f + expf(-z));
   return o * (act == 2 ? z * sg : sg);
 }
 __device__ __forceinline__ void store4(float* d, float4 v) { *(float4*)d = v; }
@@ -982,7 +984,7 @@ gate_norm_vec_kernel(const float* __restrict__ o, int H, int dv, const float* __
     u[i] = make_float4(0.f, 0.f, 0.f, 0.f);
     if (c < D4 && !pad) {
       const float4 a = x[c], b = z[c];
-      u[i] = make_float4(gated(a.x, b.x, act), gated(a.y, b.y, act), gated(a.z, b.z, act), gated(a.w, b.w, act));
+      u[i] = make_float4(gated<TO>(a.x, b.x, act), gated<TO>(a.y, b.y, act), gated<TO>(a.z, b.z, act), gated<TO>(a.w, b.w, act));
     }
     ss = fmaf(u[i].x, u[i].x, ss); ss = fmaf(u[i].y, u[i].y, ss); ss = fmaf(u[i].z, u[i].z, ss); ss = fmaf(u[i].w, u[i].w, ss);
   }
@@ -1009,12 +1011,12 @@ gate_norm_kernel(const float* __restrict__ o, int H, int dv, const float* __rest
   TO* y = out + ((size_t)n * H + h) * dv;
   float ss = 0.f;
   for (int c = threadIdx.x; c < dv && !pad; c += blockDim.x) {
-    const float u = gated(x[c], z[c], act);
+    const float u = gated<TO>(x[c], z[c], act);
     ss = fmaf(u, u, ss);
   }
   const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)dv + eps);
   for (int c = threadIdx.x; c < dv; c += blockDim.x) {
-    float u = pad ? 0.f : gated(x[c], z[c], act) * inv;
+    float u = pad ? 0.f : gated<TO>(x[c], z[c], act) * inv;
     if (w != nullptr) u *= w[w_per_head ? (size_t)h * dv + c : c];
     y[c] = Cvt<TO>::from_f(u);
   }

@@ -14,15 +14,16 @@
 // tokens and half of what they need, first every second 16 x 16 tile of the weighted C . B (left in shared memory as
 // operands), then half of the value columns. Eight others compute the state after the chunk: first the weighted x (left in
 // shared memory as operands), then units of 16 state rows x 16 columns, which they leave as operands for the next chunk's
-// results. Each group has a barrier between its two halves, the block one per chunk. The next chunk's rows travel by
-// cp.async meanwhile.
+// results, and bring the rows of the next one or two chunks in (cp.async; bulk copies of a row each took twice as long as the
+// arithmetic). One more warp computes the next chunk's decays. Each group of eight has a barrier between its two halves,
+// the block one per chunk.
 #include "attn_mma.cuh"
 #include <math.h>
 
 namespace {
 using namespace fzattn;
 constexpr int Q = 64;                       // tokens per chunk
-constexpr int SSD_THREADS = 512;        // eight warps for the results, eight for the state
+constexpr int SSD_THREADS = 544;        // eight warps for the results, eight for the state, one for the decays
 constexpr float LOG2E = 1.4426950408889634f;
 
 // 2^x for x <= 0 (results below the normal range are zero)
@@ -58,9 +59,9 @@ struct SsdChunkArgs {
 
 __host__ __device__ constexpr int pad_units(int n) { return n + 8; }      // an odd number of 16-byte units per row: no bank conflicts
 
-// PB: value columns per block (16 or 32). UM: units of 16 state rows x 16 columns per warp (1 or 2). grid (portions, heads,
-// P / PB).
-template <int PB, int UM>
+// PB: value columns per block (16 or 32). UM: units of 16 state rows x 16 columns per warp (1 or 2). ST: chunks in shared
+// memory at a time (3, or 2 where three do not fit). grid (portions, heads, P / PB).
+template <int PB, int UM, int ST>
 __global__ void __launch_bounds__(SSD_THREADS)
 ssd_chunk_kernel(const SsdChunkArgs p) {
   fz_grid_launch_dependents();
@@ -72,10 +73,10 @@ ssd_chunk_kernel(const SsdChunkArgs p) {
   extern __shared__ __align__(16) unsigned char smem_raw[];
   const int N = p.N, KN = N >> 4, SN = pad_units(N);
   constexpr int SP = pad_units(PB), SQ = pad_units(Q), NT = PB / 16;      // NT: 8-column tiles per result warp
-  __nv_bfloat16* Cs = (__nv_bfloat16*)smem_raw;            // [2][Q][SN]
-  __nv_bfloat16* Bs = Cs + 2 * Q * SN;                     // [2][Q][SN]
-  __nv_bfloat16* Xs = Bs + 2 * Q * SN;                     // [2][Q][SP]
-  __nv_bfloat16* Ms = Xs + 2 * Q * SP;                     // [2][2][N][SP]: the state before a chunk, rounding and rest
+  __nv_bfloat16* Cs = (__nv_bfloat16*)smem_raw;            // [ST][Q][SN]
+  __nv_bfloat16* Bs = Cs + ST * Q * SN;                    // [ST][Q][SN]
+  __nv_bfloat16* Xs = Bs + ST * Q * SN;                    // [ST][Q][SP]
+  __nv_bfloat16* Ms = Xs + ST * Q * SP;                    // [2][2][N][SP]: the state before a chunk, rounding and rest
   __nv_bfloat16* Gs = Ms + 4 * N * SP;                     // [2][Q][SQ]: the weighted C . B, rounding and rest
   __nv_bfloat16* Ws = Gs + 2 * Q * SQ;                     // [2][Q][SP]: the weighted x, rounding and rest
   float* scal = (float*)(Ws + 2 * Q * SP);                 // [2][4][Q]: L in powers of two, exp(L), d, exp(L_last - L) d
@@ -85,17 +86,26 @@ ssd_chunk_kernel(const SsdChunkArgs p) {
   const int nc = (cnt + Q - 1) / Q;
   const size_t off_x = (size_t)h * p.P + p0, off_b = (size_t)p.H * p.P + (size_t)g * N, off_c = off_b + (size_t)p.G * N;
 
-  auto load_chunk = [&](int c) {
-    const int st = c & 1, r = tid >> 3;                    // eight threads per token
-    const bool ok = c * Q + r < cnt;
-    const __nv_bfloat16* in = p.xbc + (size_t)(row0 + (ok ? c * Q + r : 0)) * p.W;
-    const uint32_t dc = smem_u32(Cs + (st * Q + r) * SN), db = smem_u32(Bs + (st * Q + r) * SN), dx = smem_u32(Xs + (st * Q + r) * SP);
-    for (int j = tid & 7; j < 2 * KN; j += 8) {
-      cp_async16(dc + 16 * j, in + off_c + 8 * j, ok);
-      cp_async16(db + 16 * j, in + off_b + 8 * j, ok);
+  const int per = KN >= 8 ? 3 : 2;           // 2^per threads side by side on a token's run of B or C
+  auto load_chunk = [&](int c) {                           // by the state's warps; past the portion's end: zeros
+    if (c < nc) {
+      const int st = c % ST, me = tid & 255;
+      const __nv_bfloat16* in = p.xbc + (size_t)(row0 + c * Q) * p.W;
+      for (int r = me >> per; r < Q; r += 256 >> per) {
+        const bool ok = c * Q + r < cnt;
+        const __nv_bfloat16* row = in + (ok ? (size_t)r * p.W : 0);
+        const uint32_t at = (uint32_t)((st * Q + r) * SN * 2);
+        for (int j = me & ((1 << per) - 1); j < 2 * KN; j += 1 << per) {
+          cp_async16(smem_u32(Cs) + at + 16 * j, row + off_c + 8 * j, ok);
+          cp_async16(smem_u32(Bs) + at + 16 * j, row + off_b + 8 * j, ok);
+        }
+      }
+      const int r = me >> 2;
+      const bool ok = c * Q + r < cnt;
+      if ((me & 3) < PB / 8)
+        cp_async16(smem_u32(Xs + (st * Q + r) * SP) + 16 * (me & 3), in + (ok ? (size_t)r * p.W : 0) + off_x + 8 * (me & 3), ok);
     }
-    if ((tid & 7) < PB / 8) cp_async16(dx + 16 * (tid & 7), in + off_x + 8 * (tid & 7), ok);
-    cp_async_commit();
+    cp_async_commit();                                     // (an empty group past the last chunk keeps the count)
   };
   // the scalars of a chunk, two tokens per lane of one warp; r0, r1: the tokens' raw step sizes
   auto raw_steps = [&](int c, float& r0, float& r1) {
@@ -124,18 +134,27 @@ ssd_chunk_kernel(const SsdChunkArgs p) {
     *(float2*)(sc + 3 * Q) = make_float2(ex2(last - l0) * d0, ex2(last - l1) * d1);
   };
 
-  const int sw = warp - 8;                                 // of the warps that keep the state: units sw, sw + 8, ...
-  float S[UM][2][4];                                       // a unit: rows 16 (u % KN), columns 16 (u / KN)
+  // of the warps that keep the state: units sw, sw + 8; unit u: state rows 16 (u % KN), columns 16 (u / KN)
+  const int sw = warp - 8;
+  int ur[UM], uc[UM];
+  bool own[UM];
+#pragma unroll
+  for (int i = 0; i < UM; ++i) {
+    const int u = max(sw, 0) + 8 * i;
+    own[i] = u < KN * NT;
+    ur[i] = 16 * (u % KN);
+    uc[i] = 16 * (u / KN);
+  }
+  float S[UM][2][4];
   auto leave_state = [&](int buf) {
     __nv_bfloat16* hi = Ms + (size_t)buf * 2 * N * SP;
     __nv_bfloat16* lo = hi + (size_t)N * SP;
 #pragma unroll
     for (int i = 0; i < UM; ++i) {
-      const int u = sw + 8 * i;
-      if (u >= KN * NT) break;
+      if (!own[i]) break;
 #pragma unroll
       for (int n = 0; n < 2; ++n) {
-        const int at = (16 * (u % KN) + gq) * SP + 16 * (u / KN) + 8 * n + q2;
+        const int at = (ur[i] + gq) * SP + uc[i] + 8 * n + q2;
         uint32_t a, b;
         split2(S[i][n][0], S[i][n][1], a, b);
         *(uint32_t*)(hi + at) = a; *(uint32_t*)(lo + at) = b;
@@ -145,47 +164,57 @@ ssd_chunk_kernel(const SsdChunkArgs p) {
     }
   };
   float* sp = p.state + (((size_t)slot * p.H + h) * p.P + p0) * p.npad;
-  auto state_at = [&](int u, int n, int e) {
-    return (size_t)(16 * (u / KN) + 8 * n + q2 + (e & 1)) * p.npad + 16 * (u % KN) + gq + (e & 2) * 4;
+  auto state_at = [&](int i, int n, int e) {
+    return (size_t)(uc[i] + 8 * n + q2 + (e & 1)) * p.npad + ur[i] + gq + (e & 2) * 4;
   };
 
-  load_chunk(0);
+  if (sw == 8) {                                           // the warp that computes the decays
+    float r0, r1;
+    raw_steps(0, r0, r1);
+    scalars(0, r0, r1);
+    raw_steps(1, r0, r1);                                  // (zeros past the end)
+    __syncthreads();
+    for (int c = 0; c < nc; ++c) {
+      if (c + 1 < nc) {
+        const float n0 = r0, n1 = r1;
+        raw_steps(c + 2, r0, r1);
+        scalars(c + 1, n0, n1);
+      }
+      __syncthreads();
+    }
+    return;
+  }
   if (sw >= 0) {
 #pragma unroll
-    for (int i = 0; i < UM; ++i) {
-      const int u = sw + 8 * i;
+    for (int c = 0; c < ST - 1; ++c) load_chunk(c);
+#pragma unroll
+    for (int i = 0; i < UM; ++i)
 #pragma unroll
       for (int n = 0; n < 2; ++n)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) S[i][n][e] = u < KN * NT ? sp[state_at(u, n, e)] : 0.f;
-    }
+        for (int e = 0; e < 4; ++e) S[i][n][e] = own[i] ? sp[state_at(i, n, e)] : 0.f;
     leave_state(0);
-    if (sw == 7) {
-      float r0, r1;
-      raw_steps(0, r0, r1);
-      scalars(0, r0, r1);
-    }
+    cp_async_wait<ST - 2>();
   }
-  cp_async_wait<0>();
   __syncthreads();
 
   for (int c = 0; c < nc; ++c) {
     const int st = c & 1, valid = min(Q, cnt - c * Q);
     const bool more = c + 1 < nc;
-    if (more) load_chunk(c + 1);
-    const __nv_bfloat16* Cc = Cs + st * Q * SN;
-    const __nv_bfloat16* Bc = Bs + st * Q * SN;
-    const __nv_bfloat16* Xc = Xs + st * Q * SP;
+    const int slot_in = c % ST;
+    const __nv_bfloat16* Cc = Cs + slot_in * Q * SN;
+    const __nv_bfloat16* Bc = Bs + slot_in * Q * SN;
+    const __nv_bfloat16* Xc = Xs + slot_in * Q * SP;
     const float* sc = scal + st * 4 * Q;
     if (sw < 0) {
       const int rt = warp >> 1, half = warp & 1;           // 16 tokens; which tiles and which columns
       const bool live = 16 * rt < valid;
       const int ta = 16 * rt + gq, tb = ta + 8;            // this thread's two tokens
-      float Y[NT][4];
+      float Y[NT][4], Z[NT][4];                            // products with the roundings and with the rests
 #pragma unroll
       for (int n = 0; n < NT; ++n)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) Y[n][e] = 0.f;
+        for (int e = 0; e < 4; ++e) Y[n][e] = Z[n][e] = 0.f;
       if (live) {
         float G[2][2][4];                                  // tiles half and half + 2
 #pragma unroll
@@ -213,12 +242,15 @@ ssd_chunk_kernel(const SsdChunkArgs p) {
           for (int n = 0; n < NT; ++n) {
             ldmatrix_x4_trans(b, am + (16 * k * SP) * 2 + 16 * n);
             mma_bf16(Y[n], a, b[0], b[1]);
-            mma_bf16(Y[n], a, b[2], b[3]);
+            mma_bf16(Z[n], a, b[2], b[3]);
           }
         }
         const float la = sc[ta], lb = sc[tb], ea = sc[Q + ta], eb = sc[Q + tb];
 #pragma unroll
-        for (int n = 0; n < NT; ++n) { Y[n][0] *= ea; Y[n][1] *= ea; Y[n][2] *= eb; Y[n][3] *= eb; }
+        for (int n = 0; n < NT; ++n) {
+          Y[n][0] *= ea; Y[n][1] *= ea; Y[n][2] *= eb; Y[n][3] *= eb;
+          Z[n][0] *= ea; Z[n][1] *= ea; Z[n][2] *= eb; Z[n][3] *= eb;
+        }
 #pragma unroll
         for (int i = 0; i < 2; ++i) {
           const int j = half + 2 * i;
@@ -245,23 +277,29 @@ ssd_chunk_kernel(const SsdChunkArgs p) {
 #pragma unroll
         for (int jj = 0; jj < 2; ++jj) {
           if (2 * jj > rt) break;
-          uint32_t b[NT][4];
+          uint32_t b[NT][4], hi[2][4], lo[2][4];
+#pragma unroll
+          for (int u = 0; u < 2; ++u) {
+            if (2 * jj + u > rt) break;
+            ldmatrix_x4(hi[u], ag + 32 * (2 * jj + u));
+            ldmatrix_x4(lo[u], ag + (Q * SQ) * 2 + 32 * (2 * jj + u));
+          }
 #pragma unroll
           for (int n = 0; n < NT; ++n) ldmatrix_x4_trans(b[n], ax + (32 * jj * SP) * 2 + 16 * n);
 #pragma unroll
           for (int u = 0; u < 2; ++u) {
-            const int j = 2 * jj + u;
-            if (j > rt) break;
-            uint32_t hi[4], lo[4];
-            ldmatrix_x4(hi, ag + 32 * j);
-            ldmatrix_x4(lo, ag + (Q * SQ) * 2 + 32 * j);
+            if (2 * jj + u > rt) break;
 #pragma unroll
             for (int n = 0; n < NT; ++n) {
-              mma_bf16(Y[n], hi, b[n][2 * u], b[n][2 * u + 1]);
-              mma_bf16(Y[n], lo, b[n][2 * u], b[n][2 * u + 1]);
+              mma_bf16(Y[n], hi[u], b[n][2 * u], b[n][2 * u + 1]);
+              mma_bf16(Z[n], lo[u], b[n][2 * u], b[n][2 * u + 1]);
             }
           }
         }
+#pragma unroll
+        for (int n = 0; n < NT; ++n)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) Y[n][e] += Z[n][e];
         const size_t ld = (size_t)p.H * p.P;
         const int col = 8 * NT * half + q2;
         float* dst = p.out + (size_t)(row0 + c * Q) * ld + off_x + col;
@@ -278,8 +316,6 @@ ssd_chunk_kernel(const SsdChunkArgs p) {
         }
       }
     } else {
-      float r0 = 0.f, r1 = 0.f;
-      if (sw == 7 && more) raw_steps(c + 1, r0, r1);
       {                                                    // the weighted x: four threads per token, PB / 4 columns each
         const int t = (tid - 256) >> 2, c0 = (tid & 3) * (PB / 4);
         const float w = sc[3 * Q + t];
@@ -310,51 +346,47 @@ ssd_chunk_kernel(const SsdChunkArgs p) {
         if (16 * k >= valid) break;
 #pragma unroll
         for (int i = 0; i < UM; ++i) {
-          const int u = sw + 8 * i;
-          if (u >= KN * NT) break;
+          if (!own[i]) break;
           uint32_t a[4], b[4];
-          ldmatrix_x4_trans(a, at + (16 * k * SN) * 2 + 32 * (u % KN));
-          ldmatrix_x4_trans(b, aw + (16 * k * SP) * 2 + 32 * (u / KN));
+          ldmatrix_x4_trans(a, at + (16 * k * SN) * 2 + 2 * ur[i]);
+          ldmatrix_x4_trans(b, aw + (16 * k * SP) * 2 + 2 * uc[i]);
           mma_bf16(S[i][0], a, b[0], b[1]);
           mma_bf16(S[i][1], a, b[2], b[3]);
-          ldmatrix_x4_trans(b, aw + ((Q + 16 * k) * SP) * 2 + 32 * (u / KN));
+          ldmatrix_x4_trans(b, aw + ((Q + 16 * k) * SP) * 2 + 2 * uc[i]);
           mma_bf16(S[i][0], a, b[0], b[1]);
           mma_bf16(S[i][1], a, b[2], b[3]);
         }
       }
-      if (more) {
-        leave_state(st ^ 1);
-        if (sw == 7) scalars(c + 1, r0, r1);
-      }
+      if (more) leave_state(st ^ 1);
+      load_chunk(c + ST - 1);                              // into the place of chunk c - 1
+      cp_async_wait<ST - 2>();
     }
-    cp_async_wait<0>();
     __syncthreads();
   }
   if (sw >= 0) {
 #pragma unroll
     for (int i = 0; i < UM; ++i) {
-      const int u = sw + 8 * i;
-      if (u >= KN * NT) break;
+      if (!own[i]) break;
 #pragma unroll
       for (int n = 0; n < 2; ++n)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) sp[state_at(u, n, e)] = S[i][n][e];
+        for (int e = 0; e < 4; ++e) sp[state_at(i, n, e)] = S[i][n][e];
     }
   }
 }
 
-template <int PB, int UM>
+template <int PB, int UM, int ST>
 int launch_chunk(const SsdChunkArgs& a, int n_seg, cudaStream_t stream) {
-  const size_t smem = 2 * (4 * (size_t)Q * pad_units(a.N) + 4 * Q * pad_units(PB) + 4 * (size_t)a.N * pad_units(PB) + 2 * Q * pad_units(Q)) +
-                      sizeof(float) * 8 * Q;
+  const size_t smem = 2 * (ST * Q * (2 * (size_t)pad_units(a.N) + pad_units(PB)) + 2 * Q * pad_units(PB) + 4 * (size_t)a.N * pad_units(PB) +
+                           2 * Q * pad_units(Q)) + sizeof(float) * 8 * Q;
   static size_t allowed = 48 * 1024;
   if (smem > allowed) {
     if (smem > 227 * 1024) return FZ_TOO_LARGE;
-    cudaError_t e = cudaFuncSetAttribute(ssd_chunk_kernel<PB, UM>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t e = cudaFuncSetAttribute(ssd_chunk_kernel<PB, UM, ST>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
     allowed = smem;
   }
-  fz_launch(ssd_chunk_kernel<PB, UM>, dim3(n_seg, a.H, a.P / PB), dim3(SSD_THREADS), smem, stream, a);
+  fz_launch(ssd_chunk_kernel<PB, UM, ST>, dim3(n_seg, a.H, a.P / PB), dim3(SSD_THREADS), smem, stream, a);
   FZ_LAUNCH_CHECK();
   return FZ_OK;
 }
@@ -376,8 +408,8 @@ FZ_API int fz_ssd_chunk(const void* xbc, int H, int G, int N, int P, const float
   const SsdChunkArgs a = {(const __nv_bfloat16*)xbc, H * P + 2 * G * N, H, G, N, P, dt, ldt, off_dt, dt_bias, a_log, skip, state, npad,
                           seg, min_rows, out};
   // units of 16 state rows x 16 columns: N / 16 * PB / 16, eight warps
-  if (P % 32 == 0 && N <= 128) return N <= 64 ? launch_chunk<32, 1>(a, n_seg, stream) : launch_chunk<32, 2>(a, n_seg, stream);
-  return N <= 128 ? launch_chunk<16, 1>(a, n_seg, stream) : launch_chunk<16, 2>(a, n_seg, stream);
+  if (P % 32 == 0 && N <= 128) return N <= 64 ? launch_chunk<32, 1, 3>(a, n_seg, stream) : launch_chunk<32, 2, 3>(a, n_seg, stream);
+  return N <= 128 ? launch_chunk<16, 1, 3>(a, n_seg, stream) : launch_chunk<16, 2, 2>(a, n_seg, stream);
 }
 
 #ifdef FZ_TIMELINE
