@@ -78,6 +78,15 @@ def _gimupel(c: dict):
 register_architecture("Gimupel", _gimupel)
 
 
+def _muretar(c: dict):
+    from .muretar import MuretarConfig
+    cfg = MuretarConfig.from_json(c)
+    return cfg, cfg.spec()
+
+
+register_architecture("Muretar", _muretar)
+
+
 def read_config_json(model_dir: str) -> dict:
     path = os.path.join(model_dir, "config.json")
     if not os.path.isfile(path):

@@ -37,9 +37,11 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
 }
 
 // Byte offset of the 16-byte chunk `chunk` of row `row` in a [rows][HD] bf16 tile: chunks of a row are permuted by the
-// row's low three bits, so that the eight rows one ldmatrix reads fall into different banks.
+// row's low three bits, so that the eight rows one ldmatrix reads fall into different banks. (HD 32: a row is half of the
+// 128 bytes that span the banks, so two rows share a permutation of their four chunks.)
 template <int HD>
 __device__ __forceinline__ uint32_t swz(int row, int chunk) {
+  if constexpr (HD == 32) return (uint32_t)(row * 64 + ((chunk ^ ((row >> 1) & 3)) << 4));
   return (uint32_t)(row * (HD * 2) + ((chunk ^ (row & 7)) << 4));
 }
 

@@ -1,5 +1,5 @@
 // Attention over a sliding window that keeps the first tokens, with a sink in the softmax, for prompt portions over the
-// paged bf16 cache, on tensor cores (mma.sync m16n8k16): key and value size 64 or 128.
+// paged bf16 cache, on tensor cores (mma.sync m16n8k16): key sizes 64 or 128, value sizes 32, 64 or 128.
 //
 // grid (portions + 1, tiles of 64 rows of a portion, query heads), 128 threads; warp w owns rows 16 w .. 16 w + 15 of its
 // tile. Key tiles of 64 start at multiples of 64 in absolute position: first the tiles of the kept first tokens that
@@ -8,31 +8,42 @@
 // and sum, P is rounded to bf16 for the second product; a row sees key j if j <= p and (p - j < window or j <
 // keep_first); the sink (a learned number per head, not scaled) joins the denominator at the end. The block after the
 // last portion's writes zeros into the rows of padding.
+//
+// Two maps per head (MAPS = 2, differential attention): a cached key holds one vector per map, the maps share the values.
+// Four more warps walk the same key tiles for the second map, so keys and values are fetched once; at the end they hand
+// their results over in shared memory and the first four write (a1 - lam a2) / sqrt(mean(.^2) + eps) * mult.
 #include "attn_mma.cuh"
 #include <math.h>
 
 namespace {
 using namespace fzattn;
 
-constexpr int BM = 64, BN = 64, THREADS = 128;
+constexpr int BM = 64, BN = 64;
 constexpr float LOG2E = 1.4426950408889634f;
 
-template <int HD>
-__global__ void __launch_bounds__(THREADS)
+struct MapMix {            // MAPS = 2 only
+  const float* lam;        // one number
+  float eps, mult;
+};
+
+template <int KD, int VD, int MAPS>      // size of a cached key (all maps), of a value, maps per head
+__global__ void __launch_bounds__(128 * MAPS)
 sink_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ k_pool,
                           const __nv_bfloat16* __restrict__ v_pool, const int* __restrict__ seg,
                           const int* __restrict__ seq_row, const int* __restrict__ table, int mb, long long page_stride,
                           long long head_stride, long long tok_stride, int page_size, int n_pages,
                           __nv_bfloat16* __restrict__ out, int Hq, int Hkv, float scale_log2, int window, int keep_first,
                           const float* __restrict__ sink, float cap_log2, float over_cap, const float* __restrict__ gate,
-                          int gate_ld, int gate_off, int N, int* err, int span) {
+                          int gate_ld, int gate_off, int N, int* err, int span, const MapMix mix) {
   fz_grid_launch_dependents();
   fz_grid_wait();
-  constexpr int KSTEPS = HD / 16, NB = HD / 8, TILE_BYTES = BN * HD * 2;
+  constexpr int THREADS = 128 * MAPS;
+  constexpr int KSTEPS = KD / MAPS / 16, NB = VD / 8, K_BYTES = BN * KD * 2, STAGE = K_BYTES + BN * VD * 2;
   extern __shared__ __align__(128) uint8_t smem[];
   const uint32_t s_base = smem_u32(smem);          // [2 stages][K | V], then Q
-  const uint32_t s_q = s_base + 4 * TILE_BYTES;
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const uint32_t s_q = s_base + 2 * STAGE;
+  const int tid = threadIdx.x, warp = (tid >> 5) & 3, lane = tid & 31;
+  const int map = MAPS > 1 ? tid >> 7 : 0;         // which map this warp computes
   // grid (portions + 1, heads, row tiles): blocks are handed out with the tile index falling, so a portion's last
   // tiles, which have the most keys behind them under a causal or chunked mask, start first and the short ones fill
   // the tail
@@ -41,7 +52,7 @@ sink_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat
     if (tile == 0)
       for (int n = 0; n < N; ++n)
         if (seq_row[n] < 0)
-          for (int i = tid; i < HD; i += THREADS) out[((size_t)n * Hq + h) * HD + i] = __float2bfloat16_rn(0.f);
+          for (int i = tid; i < VD; i += THREADS) out[((size_t)n * Hq + h) * VD + i] = __float2bfloat16_rn(0.f);
     return;
   }
   const int s_idx = blockIdx.x, r_off = BM * tile;
@@ -61,17 +72,18 @@ sink_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat
   const long long head_off = (long long)kvh * head_stride;
 
   {
-    const __nv_bfloat16* qbase = q + (size_t)(row0 + r_off) * Hq * HD + (size_t)h * HD;
-    for (int e = tid; e < BM * (HD / 8); e += THREADS) {
-      const int r = e / (HD / 8), c = e - r * (HD / 8);
-      cp_async16(s_q + swz<HD>(r, c), qbase + (size_t)r * Hq * HD + c * 8, r < valid_rows);
+    const __nv_bfloat16* qbase = q + (size_t)(row0 + r_off) * Hq * KD + (size_t)h * KD;
+    for (int e = tid; e < BM * (KD / 8); e += THREADS) {
+      const int r = e / (KD / 8), c = e - r * (KD / 8);
+      cp_async16(s_q + swz<KD>(r, c), qbase + (size_t)r * Hq * KD + c * 8, r < valid_rows);
     }
   }
   auto key_tile = [&](int it) { return (it <= first_end ? it : c2 + (it - first_end - 1)) * BN; };
   auto issue = [&](int it) {
-    const uint32_t sk = s_base + (it & 1) * 2 * TILE_BYTES, sv = sk + TILE_BYTES;
-    constexpr int TPR = THREADS / BN, CPT = (HD / 8) / TPR;      // threads per key row, 16-byte chunks per thread
-    const int r = tid / TPR, cfirst = (tid % TPR) * CPT;
+    const uint32_t sk = s_base + (it & 1) * STAGE, sv = sk + K_BYTES;
+    constexpr int TPR = THREADS / BN, CPK = (KD / 8) / TPR, CPV = (VD / 8) / TPR;      // threads per key row, 16-byte chunks per thread
+    static_assert((KD / 8) % TPR == 0 && (VD / 8) % TPR == 0, "tile shape");
+    const int r = tid / TPR, part = tid % TPR;
     const int key = key_tile(it) + r;
     bool valid = key <= last_pos && (key >= lo_tile || key < keep_first);
     long long off = 0;
@@ -81,10 +93,14 @@ sink_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat
       else off = (long long)page * page_stride + head_off + (long long)(key % page_size) * tok_stride;
     }
 #pragma unroll
-    for (int i = 0; i < CPT; ++i) {
-      const int c = cfirst + i;
-      cp_async16(sk + swz<HD>(r, c), k_pool + off + c * 8, valid);
-      cp_async16(sv + swz<HD>(r, c), v_pool + off + c * 8, valid);
+    for (int i = 0; i < CPK; ++i) {
+      const int c = part * CPK + i;
+      cp_async16(sk + swz<KD>(r, c), k_pool + off + c * 8, valid);
+    }
+#pragma unroll
+    for (int i = 0; i < CPV; ++i) {
+      const int c = part * CPV + i;
+      cp_async16(sv + swz<VD>(r, c), v_pool + off + c * 8, valid);
     }
     cp_async_commit();
   };
@@ -105,7 +121,7 @@ sink_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat
     if (t == 0) {
 #pragma unroll
       for (int ks = 0; ks < KSTEPS; ++ks)
-        ldmatrix_x4(qf[ks], s_q + swz<HD>(warp * 16 + (lane & 15), ks * 2 + (lane >> 4)));
+        ldmatrix_x4(qf[ks], s_q + swz<KD>(warp * 16 + (lane & 15), (map * KSTEPS + ks) * 2 + (lane >> 4)));
     }
     const int key0 = key_tile(t);
     // a warp whose rows all lie before this key tile, or whose windows all ended before it (and that is not a tile of
@@ -114,7 +130,7 @@ sink_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat
                         (window <= 0 || key0 + BN - 1 >= warp_first - window + 1 || key0 < keep_first) &&
                         (span <= 0 || key0 + BN - 1 >= warp_first - warp_first % span);
     if (active) {
-      const uint32_t sk = s_base + (t & 1) * 2 * TILE_BYTES, sv = sk + TILE_BYTES;
+      const uint32_t sk = s_base + (t & 1) * STAGE, sv = sk + K_BYTES;
       float s[BN / 8][4];
 #pragma unroll
       for (int j = 0; j < BN / 8; ++j) { s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.f; }
@@ -124,7 +140,7 @@ sink_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat
         for (int jb = 0; jb < BN / 16; ++jb) {
           uint32_t kf[4];
           const int mi = lane >> 3;
-          ldmatrix_x4(kf, sk + swz<HD>(jb * 16 + (mi >> 1) * 8 + (lane & 7), ks * 2 + (mi & 1)));
+          ldmatrix_x4(kf, sk + swz<KD>(jb * 16 + (mi >> 1) * 8 + (lane & 7), (map * KSTEPS + ks) * 2 + (mi & 1)));
           mma_bf16(s[2 * jb], qf[ks], kf[0], kf[1]);
           mma_bf16(s[2 * jb + 1], qf[ks], kf[2], kf[3]);
         }
@@ -177,7 +193,7 @@ sink_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat
         for (int nb = 0; nb < NB; nb += 2) {
           uint32_t vf[4];
           const int mi = lane >> 3;
-          ldmatrix_x4_trans(vf, sv + swz<HD>(kk * 16 + (mi & 1) * 8 + (lane & 7), nb + (mi >> 1)));
+          ldmatrix_x4_trans(vf, sv + swz<VD>(kk * 16 + (mi & 1) * 8 + (lane & 7), nb + (mi >> 1)));
           mma_bf16(o[nb], pf, vf[0], vf[1]);
           mma_bf16(o[nb + 1], pf, vf[2], vf[3]);
         }
@@ -189,6 +205,46 @@ sink_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat
   for (int hh = 0; hh < 2; ++hh) {
     l_run[hh] += __shfl_xor_sync(0xffffffffu, l_run[hh], 1);
     l_run[hh] += __shfl_xor_sync(0xffffffffu, l_run[hh], 2);
+  }
+  if constexpr (MAPS == 2) {
+    constexpr int LD = VD + 4;                     // (the stages are free: every copy has landed and was consumed)
+    float* other = (float*)smem;                   // [BM][LD]: the second map's results
+    if (map == 1) {
+#pragma unroll
+      for (int hh = 0; hh < 2; ++hh) {
+        const float inv = 1.0f / l_run[hh];
+        float* row = other + (r_lo + 8 * hh) * LD + 2 * (lane & 3);
+#pragma unroll
+        for (int i = 0; i < NB; ++i) *(float2*)(row + 8 * i) = make_float2(o[i][2 * hh] * inv, o[i][2 * hh + 1] * inv);
+      }
+    }
+    __syncthreads();
+    if (map == 1) return;
+    const float lam = mix.lam[0];
+#pragma unroll
+    for (int hh = 0; hh < 2; ++hh) {
+      const int r = r_lo + 8 * hh;
+      const float inv = 1.0f / l_run[hh];
+      const float* row = other + r * LD + 2 * (lane & 3);
+      float ss = 0.f;
+#pragma unroll
+      for (int i = 0; i < NB; ++i) {
+        const float2 b = *(const float2*)(row + 8 * i);
+        o[i][2 * hh] = fmaf(-lam, b.x, o[i][2 * hh] * inv);
+        o[i][2 * hh + 1] = fmaf(-lam, b.y, o[i][2 * hh + 1] * inv);
+        ss = fmaf(o[i][2 * hh], o[i][2 * hh], ss);
+        ss = fmaf(o[i][2 * hh + 1], o[i][2 * hh + 1], ss);
+      }
+      ss += __shfl_xor_sync(0xffffffffu, ss, 1);   // the four lanes that share the row
+      ss += __shfl_xor_sync(0xffffffffu, ss, 2);
+      const float f = mix.mult / sqrtf(ss * (1.0f / VD) + mix.eps);
+      if (r >= valid_rows) continue;
+      __nv_bfloat16* orow = out + (size_t)(row0 + r_off + r) * Hq * VD + (size_t)h * VD + 2 * (lane & 3);
+#pragma unroll
+      for (int i = 0; i < NB; ++i)
+        *(uint32_t*)(orow + 8 * i) = pack_bf16(o[i][2 * hh] * f, o[i][2 * hh + 1] * f);
+    }
+    return;
   }
 #pragma unroll
   for (int hh = 0; hh < 2; ++hh) {
@@ -204,61 +260,88 @@ sink_attention_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat
     float inv = corr / l;
     if (gate != nullptr)                           // a gate per head: the result times its sigmoid
       inv *= 1.0f / (1.0f + expf(-gate[(size_t)(row0 + r_off + r) * gate_ld + gate_off + h]));
-    __nv_bfloat16* orow = out + (size_t)(row0 + r_off + r) * Hq * HD + (size_t)h * HD + 2 * (lane & 3);
+    __nv_bfloat16* orow = out + (size_t)(row0 + r_off + r) * Hq * VD + (size_t)h * VD + 2 * (lane & 3);
 #pragma unroll
     for (int i = 0; i < NB; ++i)
       *(uint32_t*)(orow + 8 * i) = pack_bf16(o[i][2 * hh] * inv, o[i][2 * hh + 1] * inv);
   }
 }
 
-template <int HD>
-int launch(const void* q, const void* k_pool, const void* v_pool, const int* seg, const int* seq_row, int n_seg, int max_portion,
-           const int* table, int mb, long long page_stride, long long head_stride, long long tok_stride, int page_size,
-           int n_pages, void* out, int N, int Hq, int Hkv, float scale, int window, int keep_first, const float* sink,
-           float softcap, const float* gate, int gate_ld, int gate_off, int span, int* err, cudaStream_t stream) {
-  constexpr size_t smem = 4 * (BN * HD * 2) + BM * HD * 2;
+struct Step {
+  const void *q, *k_pool, *v_pool;
+  const int *seg, *seq_row, *table;
+  int n_seg, max_portion, mb;
+  long long page_stride, head_stride, tok_stride;
+  int page_size, n_pages;
+  void* out;
+  int N, Hq, Hkv;
+  float scale;
+  int window, keep_first;
+  const float* sink;
+  float softcap;
+  const float* gate;
+  int gate_ld, gate_off, span;
+  MapMix mix;
+  int* err;
+};
+
+template <int KD, int VD, int MAPS>
+int launch(const Step& a, cudaStream_t stream) {
+  constexpr size_t tiles_smem = 2 * BN * (KD + VD) * 2 + BM * KD * 2, other = MAPS == 2 ? (size_t)BM * (VD + 4) * 4 : 0;
+  constexpr size_t smem = tiles_smem > other ? tiles_smem : other;
   static bool raised = false;
   if (smem > 48 * 1024 && !raised) {
-    cudaError_t e = cudaFuncSetAttribute(sink_attention_mma_kernel<HD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t e = cudaFuncSetAttribute(sink_attention_mma_kernel<KD, VD, MAPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
     raised = true;
   }
-  const int tiles = (max_portion + BM - 1) / BM;
-  if (tiles > 65535 || Hq > 65535) return FZ_TOO_LARGE;
-  fz_launch(sink_attention_mma_kernel<HD>, dim3(n_seg + 1, Hq, tiles), dim3(THREADS), smem, stream, (const __nv_bfloat16*)q,
-            (const __nv_bfloat16*)k_pool, (const __nv_bfloat16*)v_pool, seg, seq_row, table, mb, page_stride, head_stride,
-            tok_stride, page_size, n_pages, (__nv_bfloat16*)out, Hq, Hkv, scale * LOG2E, window, keep_first, sink,
-            softcap > 0.f ? softcap * LOG2E : 0.f, softcap > 0.f ? scale / softcap : 0.f, gate, gate_ld, gate_off, N, err,
-            span);
+  const int tiles = (a.max_portion + BM - 1) / BM;
+  if (tiles > 65535 || a.Hq > 65535) return FZ_TOO_LARGE;
+  fz_launch(sink_attention_mma_kernel<KD, VD, MAPS>, dim3(a.n_seg + 1, a.Hq, tiles), dim3(128 * MAPS), smem, stream,
+            (const __nv_bfloat16*)a.q, (const __nv_bfloat16*)a.k_pool, (const __nv_bfloat16*)a.v_pool, a.seg, a.seq_row, a.table, a.mb,
+            a.page_stride, a.head_stride, a.tok_stride, a.page_size, a.n_pages, (__nv_bfloat16*)a.out, a.Hq, a.Hkv, a.scale * LOG2E,
+            a.window, a.keep_first, a.sink, a.softcap > 0.f ? a.softcap * LOG2E : 0.f, a.softcap > 0.f ? a.scale / a.softcap : 0.f,
+            a.gate, a.gate_ld, a.gate_off, a.N, a.err, a.span, a.mix);
   FZ_LAUNCH_CHECK();
   return FZ_OK;
 }
+
+int dispatch(const Step& a, int dk, int dv, int maps, cudaStream_t stream) {
+#define FZ_GO(K, V, M) if (dk == K && dv == V && maps == M) return launch<K, V, M>(a, stream)
+  FZ_GO(64, 64, 1); FZ_GO(128, 128, 1); FZ_GO(64, 32, 1); FZ_GO(64, 128, 1); FZ_GO(128, 64, 1);
+  FZ_GO(64, 64, 2); FZ_GO(128, 128, 2); FZ_GO(64, 128, 2); FZ_GO(128, 64, 2);
+#undef FZ_GO
+  return FZ_BAD_SHAPE;
+}
 }  // namespace
 
-// Sizes taken: keys and values of one size, 64 or 128; strides of the pools that keep every row 16-byte aligned.
-FZ_API int fz_sink_attention_mma_check(int Hq, int Hkv, int dk, int dv, const void* k_pool, const void* v_pool,
+// Sizes taken: cached keys (of all maps of a head together) of 64 or 128, values of 64 or 128, and one map with keys of 64
+// and values of 32; strides of the pools that keep every row 16-byte aligned.
+FZ_API int fz_sink_attention_mma_check(int Hq, int Hkv, int dk, int dv, int maps, const void* k_pool, const void* v_pool,
                                        long long page_stride, long long head_stride, long long tok_stride) {
-  if (Hq <= 0 || Hkv <= 0 || Hq % Hkv || dk != dv || (dk != 64 && dk != 128)) return FZ_BAD_SHAPE;
+  if (Hq <= 0 || Hkv <= 0 || Hq % Hkv || (maps != 1 && maps != 2) || (dk != 64 && dk != 128) ||
+      (dv != 64 && dv != 128 && !(dv == 32 && dk == 64 && maps == 1))) return FZ_BAD_SHAPE;
   if ((page_stride | head_stride | tok_stride) & 7 || ((uintptr_t)k_pool | (uintptr_t)v_pool) & 15) return FZ_BAD_ALIGNMENT;
   return FZ_OK;
 }
 
+// maps 2: two maps per head (Hq counts heads): q rows [heads][2][dk / 2]; lam, mix_eps, mix_mult as in the kernel's head. maps 1: they are not read.
 FZ_API int fz_sink_attention_mma(const void* q, const void* k_pool, const void* v_pool, const int* seg, const int* seq_row,
                                  int n_seg, int max_portion, const int* table, int mb, long long page_stride,
                                  long long head_stride, long long tok_stride, int page_size, int n_pages, void* out, int N,
-                                 int Hq, int Hkv, int hd, float scale, int window, int keep_first, const float* sink,
-                                 float softcap, const float* gate, int gate_ld, int gate_off, int span, int* err,
-                                 cudaStream_t stream) {
+                                 int Hq, int Hkv, int dk, int dv, float scale, int window, int keep_first, const float* sink,
+                                 float softcap, const float* gate, int gate_ld, int gate_off, int span, int maps,
+                                 const float* lam, float mix_eps, float mix_mult, int* err, cudaStream_t stream) {
   if (N <= 0 || n_seg <= 0) return FZ_OK;
   if (span < 0 || (span > 0 && keep_first > 0)) return FZ_BAD_SHAPE;
   if (softcap < 0.f || (gate != nullptr && (gate_off < 0 || gate_off + Hq > gate_ld))) return FZ_BAD_SHAPE;
-  if (fz_sink_attention_mma_check(Hq, Hkv, hd, hd, k_pool, v_pool, page_stride, head_stride, tok_stride) != FZ_OK ||
+  if (fz_sink_attention_mma_check(Hq, Hkv, dk, dv, maps, k_pool, v_pool, page_stride, head_stride, tok_stride) != FZ_OK ||
       page_size <= 0 || max_portion <= 0 || window < 0 || keep_first < 0 || ((uintptr_t)q & 15)) return FZ_BAD_SHAPE;
-  if (hd == 64)
-    return launch<64>(q, k_pool, v_pool, seg, seq_row, n_seg, max_portion, table, mb, page_stride, head_stride, tok_stride,
-                      page_size, n_pages, out, N, Hq, Hkv, scale, window, keep_first, sink, softcap, gate, gate_ld, gate_off, span, err, stream);
-  return launch<128>(q, k_pool, v_pool, seg, seq_row, n_seg, max_portion, table, mb, page_stride, head_stride, tok_stride,
-                     page_size, n_pages, out, N, Hq, Hkv, scale, window, keep_first, sink, softcap, gate, gate_ld, gate_off, span, err, stream);
+  if (maps == 2 && (lam == nullptr || sink != nullptr || gate != nullptr)) return FZ_BAD_SHAPE;
+  const Step a = {q, k_pool, v_pool, seg, seq_row, table, n_seg, max_portion, mb, page_stride, head_stride, tok_stride, page_size,
+                  n_pages, out, N, Hq, Hkv, scale, window, keep_first, sink, softcap, gate, gate_ld, gate_off, span,
+                  {lam, mix_eps, mix_mult}, err};
+  return dispatch(a, dk, dv, maps, stream);
 }
 
 #ifdef FZ_TIMELINE

@@ -103,12 +103,20 @@ struct Params {
   __nv_bfloat16* v_pool;
   long long page_stride;
   int page_size, write, Hq, Hkv, hd, max_len;
+  // relu2 != 0: every output goes out as max(y, 0)^2 of the biased sum y
+  int relu2;
   // argmax != 0 (few tokens, no split): nothing is stored but, per token row and 128-feature tile, the largest value
   // and its feature index (numpy's order: a NaN is the maximum, the lower index wins among equals)
   int argmax;
   float* am_val;           // [rows][tiles]
   int* am_idx;
 };
+
+__device__ __forceinline__ float finished(const Params& p, float y) {
+  if (!p.relu2) return y;
+  y = fmaxf(y, 0.f);
+  return y * y;
+}
 
 template <int BN>
 __global__ void __launch_bounds__(NUM_THREADS, 1)
@@ -244,7 +252,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
         for (int j = 0; j < 16; ++j) {
           const int m = b0 + c + j;
           if (m < b_limit) {
-            const float y = x[j] + bv;
+            const float y = finished(p, x[j] + bv);
             if (p.c_f32) p.c_f32[(size_t)m * p.feats + a_row] = y;
             else p.c_bf16[(size_t)m * p.feats + a_row] = __float2bfloat16_rn(y);
           }
@@ -253,7 +261,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
         const int n = b0 + c;
         float y[16];
 #pragma unroll
-        for (int j = 0; j < 16; ++j) y[j] = x[j] + (p.bias ? p.bias[n + j] : 0.f);
+        for (int j = 0; j < 16; ++j) y[j] = finished(p, x[j] + (p.bias ? p.bias[n + j] : 0.f));
         if (p.c_f32) {
           float4* dst = (float4*)(p.c_f32 + (size_t)a_row * p.feats + n);
 #pragma unroll
@@ -274,7 +282,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
         for (int j = 0; j < 16; ++j) {
           const int n = b0 + c + j;
           if (n < b_limit) {
-            const float y = x[j] + (p.bias ? p.bias[n] : 0.f);
+            const float y = finished(p, x[j] + (p.bias ? p.bias[n] : 0.f));
             if (p.c_f32) p.c_f32[(size_t)a_row * p.feats + n] = y;
             else p.c_bf16[(size_t)a_row * p.feats + n] = __float2bfloat16_rn(y);
           }
@@ -375,8 +383,9 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
           for (int sp = 0; sp < 8; ++sp) acc += v[sp];
           if (feat < p.feats) {
             const int m = tile_b * BN + c;
-            if (p.c_f32) p.c_f32[(size_t)m * p.feats + feat] = acc + bv;
-            else p.c_bf16[(size_t)m * p.feats + feat] = __float2bfloat16_rn(acc + bv);
+            const float y = finished(p, acc + bv);
+            if (p.c_f32) p.c_f32[(size_t)m * p.feats + feat] = y;
+            else p.c_bf16[(size_t)m * p.feats + feat] = __float2bfloat16_rn(y);
           }
         }
         n_my = 0;
@@ -517,6 +526,10 @@ __device__ __forceinline__ void rows_store_tile(const Params& p, uint32_t taddr,
 #pragma unroll
         for (int i = 0; i < 16; ++i) v[i] += p.bias[n + i];
       }
+      if (p.relu2) {
+#pragma unroll
+        for (int i = 0; i < 16; ++i) v[i] = finished(p, v[i]);
+      }
       if (p.c_f32) {
         float4* dst = (float4*)(p.c_f32 + (size_t)row * p.feats + n);
 #pragma unroll
@@ -536,7 +549,7 @@ __device__ __forceinline__ void rows_store_tile(const Params& p, uint32_t taddr,
 #pragma unroll
       for (int i = 0; i < 16; ++i) {
         if (n + i < p.feats) {
-          const float y = v[i] + (p.bias ? p.bias[n + i] : 0.f);
+          const float y = finished(p, v[i] + (p.bias ? p.bias[n + i] : 0.f));
           if (p.c_f32) p.c_f32[(size_t)row * p.feats + n + i] = y;
           else p.c_bf16[(size_t)row * p.feats + n + i] = __float2bfloat16_rn(y);
         }
@@ -962,6 +975,8 @@ __device__ __forceinline__ void split_reduce_rows(const Params& p, uint32_t base
 #pragma unroll
           for (int j = 0; j < 4; ++j) y[j] += p.bias[n + j];
         }
+#pragma unroll
+        for (int j = 0; j < 4; ++j) y[j] = finished(p, y[j]);
         if (p.c_f32) {
           *(float4*)(p.c_f32 + (size_t)row * p.feats + n) = make_float4(y[0], y[1], y[2], y[3]);
         } else {
@@ -972,7 +987,7 @@ __device__ __forceinline__ void split_reduce_rows(const Params& p, uint32_t base
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
           if (n + j < p.feats) {
-            const float yj = y[j] + (p.bias ? p.bias[n + j] : 0.f);
+            const float yj = finished(p, y[j] + (p.bias ? p.bias[n + j] : 0.f));
             if (p.c_f32) p.c_f32[(size_t)row * p.feats + n + j] = yj;
             else p.c_bf16[(size_t)row * p.feats + n + j] = __float2bfloat16_rn(yj);
           }
@@ -1389,6 +1404,14 @@ FZ_API int fz_gemm_tc_swiglu(const void* x, const void* w_packed, const float* b
   Params f{};
   f.swiglu = kind;
   return gemm_tc_impl(x, w_packed, bias_packed, out, FZ_BF16, M, 2 * I, K, f, err, stream);
+}
+
+// c = max(x . w^T + bias, 0)^2, from the unrounded sums.
+FZ_API int fz_gemm_tc_relu2(const void* x, const void* w, const float* bias, void* c, int out_dtype, int M, int N, int K,
+                            int* err, cudaStream_t stream) {
+  Params f{};
+  f.relu2 = 1;
+  return gemm_tc_impl(x, w, bias, c, out_dtype, M, N, K, f, err, stream);
 }
 
 static int gemm_tc_impl(const void* x, const void* w, const float* bias, void* c, int out_dtype, int M, int N, int K,

@@ -22,6 +22,7 @@ struct GroupedArgs {
   const int* tiles;                                     // experts mode: (group, first, count) per row tile; else null
   const int* a_idx; const int* c_idx;                   // experts mode: row maps (null: identity)
   float alpha, limit, up_shift;                         // GLU: g sigmoid(alpha g) (u + up_shift), g and u clamped by limit
+  int relu2;                                            // without GLU: the sums go out as max(sum, 0)^2
   const int* pad_rows; int pad_n, pad_top;              // experts mode, scatter: rows n with pad_rows[n] < 0 have no
                                                         // pairs; their pad_top output rows are written as zeros
 };
@@ -124,6 +125,9 @@ grouped_gemm_kernel(const GroupedArgs p) {
         const float g = fminf(v, p.limit);
         const float u = fminf(fmaxf(acu[i][j], -p.limit), p.limit);
         v = g * (1.0f / (1.0f + expf(-p.alpha * g))) * (u + p.up_shift);
+      } else if (p.relu2) {
+        v = fmaxf(v, 0.f);
+        v *= v;
       }
       C[(long long)cr * p.ldc + n] = Cvt<TC>::from_f(v);
     }
@@ -132,11 +136,12 @@ grouped_gemm_kernel(const GroupedArgs p) {
 
 // One block sorts the step's N * top (row, choice) pairs by expert. Outputs: a_idx[s] = row and c_idx[s] = row * top +
 // choice of the pair at sorted place s; tiles (expert, first place, pairs) for row tiles of tile_rows pairs, the unused ones
-// with 0 pairs; rows of padding (seq_row < 0) have no pairs. The order of pairs within an expert is whatever the atomic
+// with 0 pairs; rows of padding (seq_row < 0) have no pairs, and neither have choices E .. E + skip - 1 (experts without
+// products of their own). The order of pairs within an expert is whatever the atomic
 // counters give: no result depends on it.
 __global__ void __launch_bounds__(1024)
 route_by_table_kernel(const int* __restrict__ token_ids, const int* __restrict__ seq_row, const int* __restrict__ table,
-                      int N, int V, int top, int E, int* __restrict__ a_idx, int* __restrict__ c_idx,
+                      int N, int V, int top, int E, int skip, int* __restrict__ a_idx, int* __restrict__ c_idx,
                       int* __restrict__ tiles, int max_tiles, int tile_rows, int* err) {
   fz_grid_launch_dependents();
   fz_grid_wait();
@@ -153,6 +158,7 @@ route_by_table_kernel(const int* __restrict__ token_ids, const int* __restrict__
     const int tok = token_ids != nullptr ? token_ids[n] : n;      // no ids: row n of the table belongs to row n
     if (tok < 0 || tok >= V) { atomicOr(err, FZ_ERR_TOKEN_RANGE); continue; }
     const int e = table[(size_t)tok * top + (a - n * top)];
+    if (e >= E && e < E + skip) continue;
     if (e < 0 || e >= E) { atomicOr(err, FZ_ERR_TOKEN_RANGE); continue; }
     atomicAdd(&count[e], 1);
   }
@@ -207,31 +213,32 @@ FZ_API int fz_linear_heads(const void* A, long long lda, long long a_head, const
   if (M <= 0 || N <= 0 || H <= 0) return FZ_OK;
   if (K <= 0) return FZ_BAD_SHAPE;
   if (H > 65535 || (M + BM - 1) / BM > 65535) return FZ_TOO_LARGE;
-  GroupedArgs p = {A, lda, a_head, W, (long long)N * K, C, ldc, c_head, M, N, K, nullptr, nullptr, nullptr, 0.f, 0.f, 0.f, nullptr, 0, 0};
+  GroupedArgs p = {A, lda, a_head, W, (long long)N * K, C, ldc, c_head, M, N, K, nullptr, nullptr, nullptr, 0.f, 0.f, 0.f, 0, nullptr, 0, 0};
   return dispatch(p, dim3((N + BN - 1) / BN, (M + BM - 1) / BM, H), in_dtype, out_dtype, false, stream);
 }
 
-FZ_API int fz_route_by_table(const int* token_ids, const int* seq_row, const int* table, int N, int V, int top, int E,
+FZ_API int fz_route_by_table(const int* token_ids, const int* seq_row, const int* table, int N, int V, int top, int E, int skip,
                              int* a_idx, int* c_idx, int* tiles, int max_tiles, int tile_rows, int* err,
                              cudaStream_t stream) {
   if (N <= 0) return FZ_OK;
   if (E <= 0 || E > 4096 || top <= 0 || tile_rows <= 0 || tile_rows > 128) return FZ_BAD_SHAPE;
   fz_launch(route_by_table_kernel, dim3(1), dim3(1024), (size_t)3 * E * sizeof(int), stream, token_ids, seq_row, table, N, V,
-            top, E, a_idx, c_idx, tiles, max_tiles, tile_rows, err);
+            top, E, skip, a_idx, c_idx, tiles, max_tiles, tile_rows, err);
   FZ_LAUNCH_CHECK();
   return FZ_OK;
 }
 
-// Experts mode. glu != 0: W (E, 2N, K), C (pairs, N) in sorted order, A rows through a_idx. glu == 0: W (E, N, K), A
-// (pairs, K) in sorted order, C rows through c_idx; pad_rows (may be null): see GroupedArgs.
+// Experts mode. glu 1: W (E, 2N, K), C (pairs, N) in sorted order, A rows through a_idx. glu 0: W (E, N, K), A (pairs, K) in
+// sorted order, C rows through c_idx; pad_rows (may be null): see GroupedArgs. glu 2: W (E, N, K), A rows through a_idx, C
+// (pairs, N) = max(sum, 0)^2 in sorted order.
 FZ_API int fz_grouped_linear(const void* A, const void* W, void* C, const int* tiles, int max_tiles, int tile_rows, const int* a_idx,
                              const int* c_idx, int in_dtype, int out_dtype, int N, int K, int glu, float alpha,
                              float limit, float up_shift, const int* pad_rows, int pad_n, int pad_top, cudaStream_t stream) {
   if (max_tiles <= 0 || N <= 0) return FZ_OK;
   if (K <= 0 || tile_rows > BM) return FZ_BAD_SHAPE;      // a tile list built for larger row tiles than this kernel's
   if (max_tiles > 65535) return FZ_TOO_LARGE;
-  GroupedArgs p = {A, K, 0, W, (long long)(glu ? 2 : 1) * N * K, C, N, 0, 0, N, K, tiles, a_idx, c_idx, alpha, limit, up_shift, pad_rows, pad_n, pad_top};
-  return dispatch(p, dim3((N + BN - 1) / BN, max_tiles, 1), in_dtype, out_dtype, glu != 0, stream);
+  GroupedArgs p = {A, K, 0, W, (long long)(glu == 1 ? 2 : 1) * N * K, C, N, 0, 0, N, K, tiles, a_idx, c_idx, alpha, limit, up_shift, glu == 2 ? 1 : 0, pad_rows, pad_n, pad_top};
+  return dispatch(p, dim3((N + BN - 1) / BN, max_tiles, 1), in_dtype, out_dtype, glu == 1, stream);
 }
 
 #ifdef FZ_TIMELINE

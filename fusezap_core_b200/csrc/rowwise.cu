@@ -237,13 +237,20 @@ FZ_API int fz_add_rmsnorm(float* x, const float* delta, const void* w, int w_dty
 
 // ------------------------------------------------------------------------------------------------ add + LayerNorm
 // rows == nullptr: x[n] = (x[n] + delta[n]) + extra[n] (each if given, in place), h[n] = w * (x[n] - m) / sqrt(mean((x[n] -
-// m)^2) + eps) with m the row's mean, one block per row n. rows != nullptr: block r reads row rows[r] (x + delta, x
+// m)^2) + eps) (+ b) with m the row's mean, one block per row n. rows != nullptr: block r reads row rows[r] (x + delta, x
 // untouched) and writes h[r]; rows[r] < 0 gives zeros. The squares are taken of the deviations, after the mean is known.
+// A post norm (p.w != nullptr): delta[n] is itself replaced by its layer norm, p.w * ... + p.b, before it is added.
+struct PostNorm {
+  const float* w;
+  const float* b;      // may be null
+  float eps;
+};
+
 template <typename TH>
 __global__ void __launch_bounds__(256)
 add_layernorm_kernel(float* __restrict__ x, const float* __restrict__ delta, const float* __restrict__ extra,
-                     const float* __restrict__ w, TH* __restrict__ h, const int* __restrict__ rows, int n_src, int D, float eps,
-                     int* err) {
+                     const float* __restrict__ w, const float* __restrict__ b, TH* __restrict__ h, const int* __restrict__ rows,
+                     int n_src, int D, float eps, const PostNorm p, int* err) {
   fz_grid_launch_dependents();
   fz_grid_wait();
   __shared__ float scratch[32];
@@ -262,9 +269,23 @@ add_layernorm_kernel(float* __restrict__ x, const float* __restrict__ delta, con
   const float* dr = delta ? delta + (size_t)src * D : nullptr;
   const float* er = extra ? extra + (size_t)src * D : nullptr;
   const bool write_x = rows == nullptr && (dr != nullptr || er != nullptr);
+  const float over = 1.0f / (float)D;
+  float d_mean = 0.f, d_scale = 1.f;
+  if (p.w != nullptr) {
+    float sum = 0.f;
+    for (int d = threadIdx.x; d < D; d += blockDim.x) sum += dr[d];
+    d_mean = block_sum(sum, scratch) * over;
+    float ss = 0.f;
+    for (int d = threadIdx.x; d < D; d += blockDim.x) { const float v = dr[d] - d_mean; ss = fmaf(v, v, ss); }
+    d_scale = 1.0f / sqrtf(block_sum(ss, scratch) * over + p.eps);
+  }
   auto value = [&](int d) {
     float v = xr[d];
-    if (dr) v += dr[d];
+    if (p.w != nullptr) {
+      float y = p.w[d] * ((dr[d] - d_mean) * d_scale);
+      if (p.b != nullptr) y = __fadd_rn(y, p.b[d]);
+      v = __fadd_rn(v, y);
+    } else if (dr) v += dr[d];
     if (er) v += er[d];
     return v;
   };
@@ -274,32 +295,67 @@ add_layernorm_kernel(float* __restrict__ x, const float* __restrict__ delta, con
     if (write_x) xr[d] = v;
     sum += v;
   }
-  const float mean = block_sum(sum, scratch) * (1.0f / (float)D);
+  const float mean = block_sum(sum, scratch) * over;
   float ss = 0.f;
   for (int d = threadIdx.x; d < D; d += blockDim.x) {      // (a thread reads back what it wrote itself)
     const float v = (write_x ? xr[d] : value(d)) - mean;
     ss = fmaf(v, v, ss);
   }
-  const float scale = 1.0f / sqrtf(block_sum(ss, scratch) * (1.0f / (float)D) + eps);
-  for (int d = threadIdx.x; d < D; d += blockDim.x)
-    hr[d] = Cvt<TH>::from_f(w[d] * (((write_x ? xr[d] : value(d)) - mean) * scale));
+  const float scale = 1.0f / sqrtf(block_sum(ss, scratch) * over + eps);
+  for (int d = threadIdx.x; d < D; d += blockDim.x) {
+    const float y = w[d] * (((write_x ? xr[d] : value(d)) - mean) * scale);
+    hr[d] = Cvt<TH>::from_f(b != nullptr ? __fadd_rn(y, b[d]) : y);
+  }
+}
+
+__device__ __forceinline__ float4 times4(float4 a, float4 b) { return make_float4(a.x * b.x, a.y * b.y, a.z * b.z, a.w * b.w); }
+__device__ __forceinline__ float4 times4(float4 a, float s) { return make_float4(a.x * s, a.y * s, a.z * s, a.w * s); }
+// (sums that no multiplication is folded into)
+__device__ __forceinline__ float4 plus4(float4 a, float4 b) {
+  return make_float4(__fadd_rn(a.x, b.x), __fadd_rn(a.y, b.y), __fadd_rn(a.z, b.z), __fadd_rn(a.w, b.w));
+}
+
+// A row's mean taken off the NT * VPT float4 groups that the block holds in registers; the reciprocal root of the mean
+// squared deviation is returned. Groups past the row's end stay as they are.
+template <int NT, int VPT>
+__device__ __forceinline__ float center_row(float4* v, int D4, float over, float eps, float* scratch) {
+  float sum = 0.f;
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) sum += (v[i].x + v[i].y) + (v[i].z + v[i].w);
+  const float mean = block_sum(sum, scratch) * over;
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    if (threadIdx.x + i * NT < D4) {
+      v[i].x -= mean; v[i].y -= mean; v[i].z -= mean; v[i].w -= mean;
+      ss = fmaf(v[i].x, v[i].x, ss); ss = fmaf(v[i].y, v[i].y, ss); ss = fmaf(v[i].z, v[i].z, ss); ss = fmaf(v[i].w, v[i].w, ss);
+    }
+  }
+  return 1.0f / sqrtf(block_sum(ss, scratch) * over + eps);
 }
 
 // The same for D % 4 == 0 and D <= 4 * NT * VPT: a thread keeps its VPT float4 groups of the row in registers, so the row
 // is read once; the weights and the row's index, which no kernel of the step writes, are read ahead of the wait.
-template <typename TH, int NT, int VPT>
+template <typename TH, int NT, int VPT, bool POST>
 __global__ void __launch_bounds__(NT)
 add_layernorm_vec_kernel(float* __restrict__ x, const float* __restrict__ delta, const float* __restrict__ extra,
-                         const float* __restrict__ w, TH* __restrict__ h, const int* __restrict__ rows, int n_src, int D,
-                         float eps, int* err) {
+                         const float* __restrict__ w, const float* __restrict__ b, TH* __restrict__ h,
+                         const int* __restrict__ rows, int n_src, int D, float eps, const PostNorm p, int* err) {
   fz_grid_launch_dependents();
   const int r = blockIdx.x;
   const int D4 = D >> 2;
-  float4 g[VPT];
+  float4 g[VPT], gb[VPT], pw[POST ? VPT : 1], pb[POST ? VPT : 1];
 #pragma unroll
   for (int i = 0; i < VPT; ++i) {
     const int c = threadIdx.x + i * NT;
-    g[i] = c < D4 ? load4f(w + 4 * c) : make_float4(0.f, 0.f, 0.f, 0.f);
+    const bool in = c < D4;
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+    g[i] = in ? load4f(w + 4 * c) : zero;
+    gb[i] = in && b != nullptr ? load4f(b + 4 * c) : zero;
+    if constexpr (POST) {
+      pw[i] = in ? load4f(p.w + 4 * c) : zero;
+      pb[i] = in && p.b != nullptr ? load4f(p.b + 4 * c) : zero;
+    }
   }
   int src = r;
   if (rows != nullptr) src = rows[r];
@@ -311,6 +367,7 @@ add_layernorm_vec_kernel(float* __restrict__ x, const float* __restrict__ delta,
     for (int d = threadIdx.x; d < D; d += blockDim.x) hr[d] = Cvt<TH>::from_f(0.f);
     return;
   }
+  const float over = 1.0f / (float)D;
   float4* xr = (float4*)(x + (size_t)src * D);
   const float4* add[2] = {delta ? (const float4*)(delta + (size_t)src * D) : nullptr,
                           extra ? (const float4*)(extra + (size_t)src * D) : nullptr};
@@ -329,12 +386,19 @@ add_layernorm_vec_kernel(float* __restrict__ x, const float* __restrict__ delta,
       const int c = threadIdx.x + i * NT;
       dv[i] = c < D4 ? add[k][c] : make_float4(0.f, 0.f, 0.f, 0.f);
     }
+    if constexpr (POST) {
+      if (k == 0) {
+        const float ds = center_row<NT, VPT>(dv, D4, over, p.eps, scratch);
 #pragma unroll
-    for (int i = 0; i < VPT; ++i) { v[i].x += dv[i].x; v[i].y += dv[i].y; v[i].z += dv[i].z; v[i].w += dv[i].w; }
+        for (int i = 0; i < VPT; ++i) {
+          dv[i] = times4(pw[i], times4(dv[i], ds));
+          if (p.b != nullptr) dv[i] = plus4(dv[i], pb[i]);
+        }
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) v[i] = plus4(v[i], dv[i]);
   }
-  float sum = 0.f;
-#pragma unroll
-  for (int i = 0; i < VPT; ++i) sum += (v[i].x + v[i].y) + (v[i].z + v[i].w);
   if (rows == nullptr && (add[0] != nullptr || add[1] != nullptr)) {
 #pragma unroll
     for (int i = 0; i < VPT; ++i) {
@@ -342,49 +406,136 @@ add_layernorm_vec_kernel(float* __restrict__ x, const float* __restrict__ delta,
       if (c < D4) xr[c] = v[i];
     }
   }
-  const float mean = block_sum(sum, scratch) * (1.0f / (float)D);
-  float ss = 0.f;
-#pragma unroll
-  for (int i = 0; i < VPT; ++i) {
-    if (threadIdx.x + i * NT < D4) {
-      v[i].x -= mean; v[i].y -= mean; v[i].z -= mean; v[i].w -= mean;
-      ss = fmaf(v[i].x, v[i].x, ss); ss = fmaf(v[i].y, v[i].y, ss); ss = fmaf(v[i].z, v[i].z, ss); ss = fmaf(v[i].w, v[i].w, ss);
-    }
-  }
-  const float scale = 1.0f / sqrtf(block_sum(ss, scratch) * (1.0f / (float)D) + eps);
+  const float scale = center_row<NT, VPT>(v, D4, over, eps, scratch);
 #pragma unroll
   for (int i = 0; i < VPT; ++i) {
     const int c = threadIdx.x + i * NT;
-    if (c < D4)
-      store4f(hr + 4 * c, g[i].x * (v[i].x * scale), g[i].y * (v[i].y * scale), g[i].z * (v[i].z * scale), g[i].w * (v[i].w * scale));
+    if (c < D4) {
+      float4 y = times4(g[i], times4(v[i], scale));
+      if (b != nullptr) y = plus4(y, gb[i]);
+      store4f(hr + 4 * c, y.x, y.y, y.z, y.w);
+    }
   }
 }
 
 template <typename TH>
-static int launch_layernorm(float* x, const float* delta, const float* extra, const float* w, void* h, const int* rows,
-                            int n_out, int n_src, int D, float eps, int* err, cudaStream_t stream) {
-  const bool vec = D % 4 == 0 && D <= 4 * 512 * 8 &&
-                   (((uintptr_t)x | (uintptr_t)delta | (uintptr_t)extra | (uintptr_t)w | (uintptr_t)h) & 15) == 0;
-#define FZ_LN(NT, V) fz_launch(add_layernorm_vec_kernel<TH, NT, V>, dim3(n_out), dim3(NT), 0, stream, x, delta, extra, w, (TH*)h, rows, n_src, D, eps, err)
-  if (!vec) fz_launch(add_layernorm_kernel<TH>, dim3(n_out), dim3(256), 0, stream, x, delta, extra, w, (TH*)h, rows, n_src, D, eps, err);
+static int launch_layernorm(float* x, const float* delta, const float* extra, const float* w, const float* b, void* h, const int* rows,
+                            int n_out, int n_src, int D, float eps, const PostNorm& p, int* err, cudaStream_t stream) {
+  // (with a post norm the registers hold four weight vectors: rows of up to 8,192 values)
+  const bool vec = D % 4 == 0 && D <= 4 * 512 * (p.w != nullptr ? 4 : 8) &&
+                   (((uintptr_t)x | (uintptr_t)delta | (uintptr_t)extra | (uintptr_t)w | (uintptr_t)b | (uintptr_t)h |
+                     (uintptr_t)p.w | (uintptr_t)p.b) & 15) == 0;
+#define FZ_LN(NT, V)                                                                                                             \
+  do {                                                                                                                           \
+    if (p.w != nullptr) fz_launch(add_layernorm_vec_kernel<TH, NT, V, true>, dim3(n_out), dim3(NT), 0, stream, x, delta, extra, w, b, (TH*)h, rows, n_src, D, eps, p, err); \
+    else fz_launch(add_layernorm_vec_kernel<TH, NT, V, false>, dim3(n_out), dim3(NT), 0, stream, x, delta, extra, w, b, (TH*)h, rows, n_src, D, eps, p, err); \
+  } while (0)
+  if (!vec) fz_launch(add_layernorm_kernel<TH>, dim3(n_out), dim3(256), 0, stream, x, delta, extra, w, b, (TH*)h, rows, n_src, D, eps, p, err);
   else if (D <= 4 * 128) FZ_LN(128, 1);
   else if (D <= 4 * 256) FZ_LN(256, 1);
   else if (D <= 4 * 512) FZ_LN(512, 1);
   else if (D <= 8 * 512) FZ_LN(512, 2);
   else if (D <= 16 * 512) FZ_LN(512, 4);
-  else FZ_LN(512, 8);
+  else fz_launch(add_layernorm_vec_kernel<TH, 512, 8, false>, dim3(n_out), dim3(512), 0, stream, x, delta, extra, w, b, (TH*)h, rows, n_src, D, eps, p, err);
 #undef FZ_LN
   FZ_LAUNCH_CHECK();
   return FZ_OK;
 }
 
-FZ_API int fz_add_layernorm(float* x, const float* delta, const float* extra, const float* w, void* h, int h_dtype,
-                            const int* rows, int n_out, int n_src, int D, float eps, int* err, cudaStream_t stream) {
+// post_w null: no post norm. b, post_b may be null.
+FZ_API int fz_add_layernorm(float* x, const float* delta, const float* extra, const float* w, const float* b, void* h, int h_dtype,
+                            const int* rows, int n_out, int n_src, int D, float eps, const float* post_w, const float* post_b,
+                            float post_eps, int* err, cudaStream_t stream) {
   if (n_out <= 0) return FZ_OK;
-  if (D <= 0 || (rows != nullptr && extra != nullptr)) return FZ_BAD_SHAPE;
-  if (h_dtype == FZ_F32) return launch_layernorm<float>(x, delta, extra, w, h, rows, n_out, n_src, D, eps, err, stream);
-  if (h_dtype == FZ_BF16) return launch_layernorm<__nv_bfloat16>(x, delta, extra, w, h, rows, n_out, n_src, D, eps, err, stream);
+  if (D <= 0 || (rows != nullptr && extra != nullptr) || (post_w != nullptr && delta == nullptr)) return FZ_BAD_SHAPE;
+  const PostNorm p = {post_w, post_b, post_eps};
+  if (h_dtype == FZ_F32) return launch_layernorm<float>(x, delta, extra, w, b, h, rows, n_out, n_src, D, eps, p, err, stream);
+  if (h_dtype == FZ_BF16) return launch_layernorm<__nv_bfloat16>(x, delta, extra, w, b, h, rows, n_out, n_src, D, eps, p, err, stream);
   return FZ_BAD_DTYPE;
+}
+
+// ------------------------------------------------------------------------------------------------ sum of normed streams
+// out[n] = sum_i s_i * (w_i * t_i[n] / sqrt(mean(t_i[n]^2) + eps)), each term rounded, added in the order given: one block
+// per row. For D % 4 == 0 and D <= 4 * NT * VPT a thread keeps its groups in registers and every term is read once.
+struct NormedTerms {
+  const float* t[4];
+  const float* w[4];
+  float s[4];
+  int n;
+};
+__global__ void __launch_bounds__(256) normed_sum_kernel(const NormedTerms p, float* __restrict__ out, int D, float eps) {
+  fz_grid_launch_dependents();
+  fz_grid_wait();
+  __shared__ float scratch[32];
+  const size_t at = (size_t)blockIdx.x * D;
+  float inv[4];
+  for (int k = 0; k < p.n; ++k) {
+    float ss = 0.f;
+    for (int d = threadIdx.x; d < D; d += blockDim.x) ss = fmaf(p.t[k][at + d], p.t[k][at + d], ss);
+    inv[k] = 1.0f / sqrtf(block_sum(ss, scratch) * (1.0f / (float)D) + eps);
+  }
+  for (int d = threadIdx.x; d < D; d += blockDim.x) {
+    float acc = 0.f;
+    for (int k = 0; k < p.n; ++k) {
+      const float y = __fmul_rn(p.s[k], __fmul_rn(p.w[k][d], __fmul_rn(p.t[k][at + d], inv[k])));
+      acc = k == 0 ? y : __fadd_rn(acc, y);
+    }
+    out[at + d] = acc;
+  }
+}
+template <int NT, int VPT>
+__global__ void __launch_bounds__(NT) normed_sum_vec_kernel(const NormedTerms p, float* __restrict__ out, int D, float eps) {
+  fz_grid_launch_dependents();
+  fz_grid_wait();
+  __shared__ float scratch[32];
+  const size_t at = (size_t)blockIdx.x * D;
+  const int D4 = D >> 2;
+  float4 acc[VPT];
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) acc[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+  for (int k = 0; k < p.n; ++k) {
+    const float4* t = (const float4*)(p.t[k] + at);
+    const float4* w = (const float4*)p.w[k];
+    float4 v[VPT];
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int c = threadIdx.x + i * NT;
+      v[i] = c < D4 ? t[c] : make_float4(0.f, 0.f, 0.f, 0.f);
+      ss = fmaf(v[i].x, v[i].x, ss); ss = fmaf(v[i].y, v[i].y, ss); ss = fmaf(v[i].z, v[i].z, ss); ss = fmaf(v[i].w, v[i].w, ss);
+    }
+    const float inv = 1.0f / sqrtf(block_sum(ss, scratch) * (1.0f / (float)D) + eps);
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int c = threadIdx.x + i * NT;
+      if (c < D4) acc[i] = plus4(acc[i], times4(times4(w[c], times4(v[i], inv)), p.s[k]));
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = threadIdx.x + i * NT;
+    if (c < D4) ((float4*)(out + at))[c] = acc[i];
+  }
+}
+
+FZ_API int fz_normed_sum(const float* t0, const float* t1, const float* t2, const float* t3, const float* w0, const float* w1,
+                         const float* w2, const float* w3, float s0, float s1, float s2, float s3, int n_terms, float* out, int N,
+                         int D, float eps, cudaStream_t stream) {
+  if (N <= 0 || D <= 0) return FZ_OK;
+  if (n_terms < 1 || n_terms > 4) return FZ_BAD_SHAPE;
+  const NormedTerms p = {{t0, t1, t2, t3}, {w0, w1, w2, w3}, {s0, s1, s2, s3}, n_terms};
+  uintptr_t bits = (uintptr_t)out;
+  for (int k = 0; k < n_terms; ++k) bits |= (uintptr_t)p.t[k] | (uintptr_t)p.w[k];
+#define FZ_NS(NT, V) fz_launch(normed_sum_vec_kernel<NT, V>, dim3(N), dim3(NT), 0, stream, p, out, D, eps)
+  if (D % 4 || D > 4 * 512 * 8 || (bits & 15)) fz_launch(normed_sum_kernel, dim3(N), dim3(256), 0, stream, p, out, D, eps);
+  else if (D <= 4 * 128) FZ_NS(128, 1);
+  else if (D <= 4 * 256) FZ_NS(256, 1);
+  else if (D <= 4 * 512) FZ_NS(512, 1);
+  else if (D <= 8 * 512) FZ_NS(512, 2);
+  else FZ_NS(512, 8);
+#undef FZ_NS
+  FZ_LAUNCH_CHECK();
+  return FZ_OK;
 }
 
 // ------------------------------------------------------------------------------------------------ rotation + cache write

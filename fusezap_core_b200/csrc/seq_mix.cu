@@ -134,6 +134,9 @@ struct AttnArgs {
   float softcap;                                   // > 0: the scaled score s becomes softcap * tanh(s / softcap)
   const float* gate; int gate_ld, gate_off;        // not null: head h's result is multiplied by sigmoid(gate[n gate_ld + gate_off + h])
   int span;                                        // > 0: a row sees only the keys of its own block of `span` positions
+  // maps > 1: Hq counts softmax maps, `maps` neighbouring ones per head, which share the head's values; map m scores the
+  // dq = dk / maps values of a key from m dq on. Results go out as float32 (out is float*).
+  int maps, dq;
 };
 
 // The first key a row at position p sees (kept first tokens aside): the window's start, and with a chunked mask not
@@ -249,11 +252,11 @@ __device__ __forceinline__ void load_chunk(const AttnArgs& a, const int* trow, i
 // One warp, one pair, one chunk: the online-softmax update. A chunk without a visible key changes nothing.
 template <int DPL>
 __device__ __forceinline__ void pair_chunk(const float* qh, const float* Ks, const float* Vs, int c, int p, int lo,
-                                           int keep_first, float scale, float softcap, int dk, int dv, float& m, float& l, float* acc) {
+                                           int keep_first, float scale, float softcap, int ldk, int dk, int dv, float& m, float& l, float* acc) {
   const int lane = threadIdx.x & 31;
   const int key = c * CHUNK + lane;
   const bool valid = key <= p && (key >= lo || key < keep_first);
-  const float* kr = Ks + lane * (dk + 1);
+  const float* kr = Ks + lane * ldk;
   float s = 0.f;
   for (int d = 0; d < dk; ++d) s = fmaf(qh[d], kr[d], s);
   if (softcap > 0.f) {
@@ -293,6 +296,15 @@ __device__ __forceinline__ void pair_finish(const AttnArgs& a, int n, int head, 
   }
   float inv = 1.0f / l;
   if (a.gate != nullptr) inv *= 1.0f / (1.0f + expf(-a.gate[(size_t)n * a.gate_ld + a.gate_off + head]));
+  if (a.maps > 1) {
+    float* o32 = (float*)a.out + ((size_t)n * a.Hq + head) * a.dv;
+#pragma unroll
+    for (int i = 0; i < DPL; ++i) {
+      const int d = lane + 32 * i;
+      if (d < a.dv) o32[d] = acc[i] * corr * inv;
+    }
+    return;
+  }
   T* o = (T*)a.out + ((size_t)n * a.Hq + head) * a.dv;
 #pragma unroll
   for (int i = 0; i < DPL; ++i) {
@@ -312,7 +324,10 @@ sink_attention_tile_kernel(const AttnArgs a) {
     if (blockIdx.y == 0 && blockIdx.z == 0)
       for (int n = 0; n < a.N; ++n)
         if (a.seq_row[n] < 0)
-          for (int i = threadIdx.x; i < a.Hq * a.dv; i += blockDim.x) ((T*)a.out)[(size_t)n * a.Hq * a.dv + i] = Cvt<T>::from_f(0.f);
+          for (int i = threadIdx.x; i < a.Hq * a.dv; i += blockDim.x) {
+            if (a.maps > 1) ((float*)a.out)[(size_t)n * a.Hq * a.dv + i] = 0.f;
+            else ((T*)a.out)[(size_t)n * a.Hq * a.dv + i] = Cvt<T>::from_f(0.f);
+          }
     return;
   }
   const int row0 = a.seg[4 * s], cnt = a.seg[4 * s + 1], pos0 = a.seg[4 * s + 2];
@@ -325,15 +340,15 @@ sink_attention_tile_kernel(const AttnArgs a) {
   const int G = min(MAX_PAIRS, G_all - g_base);
   const int nr = min(a.rows_per_block, cnt - r0);
   const int warp = threadIdx.x >> 5;
-  const int dk = a.dk, dv = a.dv;
+  const int dk = a.dk, dv = a.dv, dq = a.dq;
   float* Ks = smem;                            // [CHUNK][dk + 1]
   float* Vs = Ks + CHUNK * (dk + 1);           // [CHUNK][dv]
-  float* Qs = Vs + CHUNK * dv;                 // [nr * G][dk]
+  float* Qs = Vs + CHUNK * dv;                 // [nr * G][dq]
   const int head0 = kvh * G_all + g_base;
   const T* q = (const T*)a.q;
-  for (int e = threadIdx.x; e < nr * G * dk; e += blockDim.x) {
-    const int pr = e / dk, d = e - pr * dk;
-    Qs[e] = Cvt<T>::to_f(q[((size_t)(row0 + r0 + pr / G) * a.Hq + head0 + pr % G) * dk + d]);
+  for (int e = threadIdx.x; e < nr * G * dq; e += blockDim.x) {
+    const int pr = e / dq, d = e - pr * dq;
+    Qs[e] = Cvt<T>::to_f(q[((size_t)(row0 + r0 + pr / G) * a.Hq + head0 + pr % G) * dq + d]);
   }
   float m[MAX_PPW], l[MAX_PPW], acc[MAX_PPW][DPL];
 #pragma unroll
@@ -358,7 +373,8 @@ sink_attention_tile_kernel(const AttnArgs a) {
       if (pr >= pairs) break;
       const int p = p_first + pr / G;
       const int lo = first_seen(p, a.window, a.span);
-      pair_chunk<DPL>(Qs + pr * dk, Ks, Vs, c, p, lo, a.keep_first, a.scale, a.softcap, dk, dv, m[x], l[x], acc[x]);
+      pair_chunk<DPL>(Qs + pr * dq, Ks + (head0 + pr % G) % a.maps * dq, Vs, c, p, lo, a.keep_first, a.scale, a.softcap, dk + 1, dq, dv,
+                      m[x], l[x], acc[x]);
     }
   }
 #pragma unroll
@@ -388,13 +404,13 @@ sink_attention_unit_kernel(const AttnArgs a) {
   const int kvh = blockIdx.y / slices, g_base = (blockIdx.y % slices) * MAX_PAIRS;
   const int G = min(MAX_PAIRS, G_all - g_base);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int dk = a.dk, dv = a.dv;
+  const int dk = a.dk, dv = a.dv, dq = a.dq;
   float* Ks = smem;
   float* Vs = Ks + CHUNK * (dk + 1);
-  float* Qs = Vs + CHUNK * dv;                 // [G][dk]
+  float* Qs = Vs + CHUNK * dv;                 // [G][dq]
   const int head0 = kvh * G_all + g_base;
-  const T* q = (const T*)a.q + ((size_t)n * a.Hq + head0) * dk;
-  for (int e = threadIdx.x; e < G * dk; e += blockDim.x) Qs[e] = Cvt<T>::to_f(q[e]);
+  const T* q = (const T*)a.q + ((size_t)n * a.Hq + head0) * dq;
+  for (int e = threadIdx.x; e < G * dq; e += blockDim.x) Qs[e] = Cvt<T>::to_f(q[e]);
   float m[MAX_PPW], l[MAX_PPW], acc[MAX_PPW][DPL];
 #pragma unroll
   for (int x = 0; x < MAX_PPW; ++x) {
@@ -413,7 +429,8 @@ sink_attention_unit_kernel(const AttnArgs a) {
     for (int x = 0; x < MAX_PPW; ++x) {
       const int g = warp + x * ATT_WARPS;
       if (g >= G) break;
-      pair_chunk<DPL>(Qs + g * dk, Ks, Vs, c, p, walk.lo, a.keep_first, a.scale, a.softcap, dk, dv, m[x], l[x], acc[x]);
+      pair_chunk<DPL>(Qs + g * dq, Ks + (head0 + g) % a.maps * dq, Vs, c, p, walk.lo, a.keep_first, a.scale, a.softcap, dk + 1, dq, dv,
+                      m[x], l[x], acc[x]);
     }
   }
 #pragma unroll
@@ -443,8 +460,11 @@ sink_attention_merge_kernel(const AttnArgs a) {
   fz_grid_wait();
   const int dv = a.dv;
   if (row < 0) {
-    T* o = (T*)a.out + ((size_t)n * a.Hq + head) * dv;
-    for (int d = threadIdx.x; d < dv; d += blockDim.x) o[d] = Cvt<T>::from_f(0.f);
+    const size_t at = ((size_t)n * a.Hq + head) * dv;
+    for (int d = threadIdx.x; d < dv; d += blockDim.x) {
+      if (a.maps > 1) ((float*)a.out)[at + d] = 0.f;
+      else ((T*)a.out)[at + d] = Cvt<T>::from_f(0.f);
+    }
     return;
   }
   const ChunkWalk walk(p, p, a.window, a.keep_first, a.span);
@@ -482,6 +502,31 @@ sink_attention_merge_kernel(const AttnArgs a) {
     for (int i = 0; i < DPL; ++i) acc[i] += sums[w][lane + 32 * i];
   }
   pair_finish<T, DPL>(a, n, head, m, l, acc);
+}
+
+// out[n, h] = T((a1 - lam * a2) / sqrt(mean((a1 - lam * a2)^2) + eps) * mult) with a1, a2 the two maps' results of head h,
+// (N, H, 2, dv) float32. A warp per (row, head).
+template <typename T>
+__global__ void __launch_bounds__(256)
+combine_maps_kernel(const float* __restrict__ a, int H, int dv, const float* __restrict__ lam, float eps, float mult,
+                    const int* __restrict__ seq_row, T* __restrict__ out) {
+  fz_grid_launch_dependents();
+  const float la = lam[0];
+  fz_grid_wait();
+  const int n = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, W = blockDim.x >> 5;
+  const bool pad = seq_row[n] < 0;
+  for (int h = warp; h < H; h += W) {
+    const float* x = a + ((size_t)n * H + h) * 2 * dv;
+    T* y = out + ((size_t)n * H + h) * dv;
+    if (pad) {
+      for (int c = lane; c < dv; c += 32) y[c] = Cvt<T>::from_f(0.f);
+      continue;
+    }
+    float ss = 0.f;
+    for (int c = lane; c < dv; c += 32) { const float v = fmaf(-la, x[dv + c], x[c]); ss = fmaf(v, v, ss); }
+    const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)dv + eps);
+    for (int c = lane; c < dv; c += 32) y[c] = Cvt<T>::from_f(fmaf(-la, x[dv + c], x[c]) * inv * mult);
+  }
 }
 
 // ------------------------------------------------------------------------------------------------ recurrent scans (see scan.cuh)
@@ -604,11 +649,17 @@ retention_scan_kernel(const float* __restrict__ proj, int ld, int H, int dk, int
   store_state(sp + 2 * (size_t)dkp, dkp, has[2], has[3], S[1]);
 }
 
+__device__ __forceinline__ float decay_of(float a, float rate) {
+  const float soft = a > 20.f ? a : log1pf(expf(a));
+  return expf(-rate * soft);
+}
 // S = g * S (rows); u = beta (v - S^T k^); S += k^ u^T; o = S^T q^. qkv rows: [q (Hk dk) | k (Hk dk) | v (H dv)] of T.
-template <typename T, int R>
+// HEAD: one decay per head (high holds one input per head), else one per head and key channel. high and beta point at
+// their first column; their rows are ldh and ldb floats long.
+template <typename T, int R, bool HEAD>
 __global__ void __launch_bounds__(SCAN_MAX_THREADS)
 gated_delta_scan_kernel(const T* __restrict__ qkv, int H, int Hk, int dk, int dv, int tch,
-                        const float* __restrict__ high, int ldh, const float* __restrict__ beta,
+                        const float* __restrict__ high, int ldh, const float* __restrict__ beta, int ldb,
                         const float* __restrict__ a_log, const float* __restrict__ dt_bias, float unit_eps, float q_scale,
                         float* __restrict__ state, const int* __restrict__ seg, float* __restrict__ out) {
   fz_grid_launch_dependents();
@@ -623,10 +674,11 @@ gated_delta_scan_kernel(const T* __restrict__ qkv, int H, int Hk, int dk, int dv
   float* qs = smem;                    // [tch][dkp]   what the recurrence reads
   float* ks = qs + tch * dkp;
   float* gs = ks + tch * dkp;
-  float* vs = gs + tch * dkp;          // [tch][COLS]
+  const int da = HEAD ? 1 : dk;        // decays per token, and what a token keeps of them below
+  float* vs = gs + tch * (HEAD ? 4 : dkp);   // [tch][COLS]
   float* bs = vs + tch * COLS;         // [tch]
-  float* ra = bs + tch;                // [tch][dk]    raw: decay inputs
-  float* rb = ra + tch * dk;           // [tch]        raw: beta before the sigmoid
+  float* ra = bs + tch;                // [tch][da]    raw: decay inputs
+  float* rb = ra + tch * da;           // [tch]        raw: beta before the sigmoid
   T* rq = (T*)(rb + tch);              // [tch][dke]   raw: q, k, v after the convolution
   T* rk = rq + tch * dke;
   T* rv = rk + tch * dke;              // [tch][cole]
@@ -647,8 +699,8 @@ gated_delta_scan_kernel(const T* __restrict__ qkv, int H, int Hk, int dk, int dv
   const float rate = expf(a_log[h]);
   const bool pairs = sizeof(T) == 2 && words;
   const int uq = pairs ? dk / 2 : dk, uv = pairs ? ncols / 2 : ncols;      // copies per run of q or k, and of v
-  const int avec = ((dk | ldh) & 3) == 0 && aligned16(high) ? 4 : 1;      // the float32 decay inputs: 16 bytes a copy where aligned
-  const int ua = dk / avec;
+  const int avec = !HEAD && ((dk | ldh) & 3) == 0 && aligned16(high) ? 4 : 1;      // the float32 decay inputs: 16 bytes a copy where aligned
+  const int ua = da / avec;
   const int per_token = 2 * uq + uv + ua + 1;
   auto issue = [&](int t0) {
     const int tc = min(tch, cnt - t0);
@@ -663,8 +715,8 @@ gated_delta_scan_kernel(const T* __restrict__ qkv, int H, int Hk, int dk, int dv
       i -= uq;
       if (i < uv) { stage_unit(rv + tt * cole, in + (size_t)2 * Hk * dk + (size_t)h * dv + col0, i, words); continue; }
       i -= uv;
-      if (i < ua) cp_words(ra + tt * dk, high + n * ldh + (size_t)h * dk, i, avec);
-      else cp_async4(rb + tt, beta + n * H + h);
+      if (i < ua) cp_words(ra + tt * da, high + n * ldh + (size_t)h * da, i, avec);
+      else cp_async4(rb + tt, beta + n * ldb + h);
     }
     cp_async_commit();
   };
@@ -685,13 +737,14 @@ gated_delta_scan_kernel(const T* __restrict__ qkv, int H, int Hk, int dk, int dv
         if (i < dk) {
           qv = __fmul_rn(__fdiv_rn(Cvt<T>::to_f(qin[i]), nq), q_scale);
           kv = __fdiv_rn(Cvt<T>::to_f(kin[i]), nk);
-          const float a = ra[tt * dk + i] + dt_bias[(size_t)h * dk + i];
-          const float soft = a > 20.f ? a : log1pf(expf(a));
-          gv = expf(-rate * soft);
+          if constexpr (!HEAD) gv = decay_of(ra[tt * dk + i] + dt_bias[(size_t)h * dk + i], rate);
         }
         qs[tt * dkp + i] = qv;
         ks[tt * dkp + i] = kv;
-        gs[tt * dkp + i] = gv;
+        if constexpr (!HEAD) gs[tt * dkp + i] = gv;
+      }
+      if constexpr (HEAD) {
+        if (lane == 0) gs[tt] = decay_of(ra[tt] + dt_bias[h], rate);
       }
       if (lane == 0) bs[tt] = 1.0f / (1.0f + expf(-rb[tt]));
     }
@@ -718,11 +771,12 @@ gated_delta_scan_kernel(const T* __restrict__ qkv, int H, int Hk, int dk, int dv
       float kk[DPT], qq[DPT], gg[DPT];
       load8(ks + tt * dkp + r * DPT, kk);
       load8(qs + tt * dkp + r * DPT, qq);
-      load8(gs + tt * dkp + r * DPT, gg);
+      if constexpr (!HEAD) load8(gs + tt * dkp + r * DPT, gg);
+      const float2 gh = both(HEAD ? gs[tt] : 0.f);
       float2 ksum[DC / 2] = {make_float2(0.f, 0.f), make_float2(0.f, 0.f)};
 #pragma unroll
       for (int i = 0; i < DPT; ++i) {
-        const float2 g2 = both(gg[i]), k2 = both(kk[i]);
+        const float2 g2 = HEAD ? gh : both(gg[i]), k2 = both(kk[i]);
 #pragma unroll
         for (int j = 0; j < DC / 2; ++j) {
           S[j][i] = __fmul2_rn(g2, S[j][i]);
@@ -1123,11 +1177,14 @@ router_topk_kernel(const float* __restrict__ logits, int ld, int N, int E, const
 }
 
 // out[n] = scale * (add[n] + sum_k w[n, k] terms[n top + k] (+ sigmoid(gl[n, col]) shared[n])); a null gl counts as a gate
-// of 1, a null add as zero, and the product with scale is left out when it is 1; rows of padding give zeros.
+// of 1, a null add as zero, and the product with scale is left out when it is 1; rows of padding give zeros. choice not
+// null: where choice[n, k] >= n_experts the term is the row's input, hin[n], and terms[n top + k] is not read.
+template <typename TH>
 __global__ void __launch_bounds__(256)
 moe_combine_kernel(const float* __restrict__ terms, const float* __restrict__ w, int top, const float* __restrict__ shared,
                    const float* __restrict__ gl, int ldg, int col, const int* __restrict__ seq_row, float* __restrict__ out,
-                   int N, int D, const float* __restrict__ add, float scale) {
+                   int N, int D, const float* __restrict__ add, float scale, const int* __restrict__ choice, int n_experts,
+                   const TH* __restrict__ hin) {
   fz_grid_launch_dependents();
   fz_grid_wait();
   const int n = blockIdx.x;
@@ -1137,7 +1194,11 @@ moe_combine_kernel(const float* __restrict__ terms, const float* __restrict__ w,
   for (int d = blockIdx.y * blockDim.x + threadIdx.x; d < D; d += gridDim.y * blockDim.x) {
     float acc = 0.f;
     if (!pad) {
-      for (int k = 0; k < top; ++k) acc = __fmaf_rn(w[(size_t)n * top + k], terms[((size_t)n * top + k) * D + d], acc);
+      for (int k = 0; k < top; ++k) {
+        const size_t at = (size_t)n * top + k;
+        const bool hand_on = choice != nullptr && choice[at] >= n_experts;
+        acc = __fmaf_rn(w[at], hand_on ? Cvt<TH>::to_f(hin[(size_t)n * D + d]) : terms[at * D + d], acc);
+      }
       if (shared != nullptr) acc = __fmaf_rn(sg, shared[(size_t)n * D + d], acc);
       if (add != nullptr) acc = __fadd_rn(acc, add[(size_t)n * D + d]);
       if (scale != 1.f) acc = __fmul_rn(acc, scale);
@@ -1339,8 +1400,8 @@ __global__ void __launch_bounds__(256) weighted_sum_kernel(const Terms p, float*
   }
 }
 
-size_t attn_smem(int dk, int dv, int pairs) {
-  return sizeof(float) * ((size_t)CHUNK * (dk + 1) + (size_t)CHUNK * dv + (size_t)pairs * dk);
+size_t attn_smem(int dk, int dv, int dq, int pairs) {
+  return sizeof(float) * ((size_t)CHUNK * (dk + 1) + (size_t)CHUNK * dv + (size_t)pairs * dq);
 }
 
 // rows_per_block: as many rows of a portion as give 32 (row, head) pairs at most.
@@ -1350,7 +1411,7 @@ int launch_sink(AttnArgs a, int N, int n_seg, int max_portion, int units, cudaSt
   const int G = G_all < MAX_PAIRS ? G_all : MAX_PAIRS;
   if (units > 0) {                      // single tokens: runs of chunks per block, then the merge
     static size_t allowed_u = 48 * 1024;
-    const size_t smem = attn_smem(a.dk, a.dv, G);
+    const size_t smem = attn_smem(a.dk, a.dv, a.dq, G);
     int st = allow_smem(sink_attention_unit_kernel<T, DPL>, smem, allowed_u);
     if (st != FZ_OK) return st;
     fz_launch(sink_attention_unit_kernel<T, DPL>, dim3(N, a.Hkv * slices, units), dim3(32 * ATT_WARPS), smem, stream, a);
@@ -1361,7 +1422,7 @@ int launch_sink(AttnArgs a, int N, int n_seg, int max_portion, int units, cudaSt
   }
   a.rows_per_block = MAX_PAIRS / G > 0 ? MAX_PAIRS / G : 1;
   static size_t allowed_t = 48 * 1024;
-  const size_t smem = attn_smem(a.dk, a.dv, a.rows_per_block * G);
+  const size_t smem = attn_smem(a.dk, a.dv, a.dq, a.rows_per_block * G);
   int st = allow_smem(sink_attention_tile_kernel<T, DPL>, smem, allowed_t);
   if (st != FZ_OK) return st;
   const int tiles = (max_portion + a.rows_per_block - 1) / a.rows_per_block;
@@ -1427,22 +1488,37 @@ FZ_API int fz_sink_attention_units(int window, int keep_first, int max_context, 
 
 // Portions are rows of `seg` (n_seg of them, max_portion rows at most). units > 0 (every portion a single token): the
 // keys of a row are cut into runs of unit_chunks chunks, `units` at most, with `part` of N * Hq * units * (dv + 2) floats.
+// maps > 1: see AttnArgs (out is float32 then, (N, Hq, dv) with Hq = heads * maps).
 FZ_API int fz_sink_attention(const void* q, const void* k_pool, const void* v_pool, const int* pos, const int* seq_row,
                              const int* seg, int n_seg, int max_portion, const int* table, int mb, long long page_stride,
                              long long head_stride, long long tok_stride, int page_size, int n_pages, void* out, int dtype,
                              int N, int Hq, int Hkv, int dk, int dv, float scale, int window, int keep_first,
                              const float* sink, int unit_chunks, int units, float* part, float softcap, const float* gate,
-                             int gate_ld, int gate_off, int span, int* err, cudaStream_t stream) {
+                             int gate_ld, int gate_off, int span, int maps, int* err, cudaStream_t stream) {
   if (N <= 0 || n_seg <= 0) return FZ_OK;
   if (span < 0 || (span > 0 && keep_first > 0)) return FZ_BAD_SHAPE;
+  if (maps < 1 || dk % maps || Hq % maps || (Hq / Hkv) % maps) return FZ_BAD_SHAPE;
   if (softcap < 0.f || (gate != nullptr && (gate_off < 0 || gate_off + Hq > gate_ld))) return FZ_BAD_SHAPE;
   if (fz_sink_attention_check(Hq, Hkv, dk, dv) != FZ_OK || page_size <= 0 || window < 0 || keep_first < 0 || max_portion <= 0 ||
       (units > 0 && (unit_chunks <= 0 || part == nullptr || units > 65535))) return FZ_BAD_SHAPE;
   AttnArgs a = {q, k_pool, v_pool, pos, seq_row, seg, table, mb, page_stride, head_stride, tok_stride, page_size, n_pages, out,
-                Hq, Hkv, dk, dv, scale, window, keep_first, sink, err, N, 1, unit_chunks, units, part, softcap, gate, gate_ld, gate_off, span};
+                Hq, Hkv, dk, dv, scale, window, keep_first, sink, err, N, 1, unit_chunks, units, part, softcap, gate, gate_ld, gate_off, span, maps, dk / maps};
   if (dtype == FZ_F32) return dispatch_sink<float>(a, N, n_seg, max_portion, units, stream);
   if (dtype == FZ_BF16) return dispatch_sink<__nv_bfloat16>(a, N, n_seg, max_portion, units, stream);
   return FZ_BAD_DTYPE;
+}
+
+// a: (N, H, 2, dv) float32, lam: one float32 on the device.
+FZ_API int fz_combine_maps(const float* a, int N, int H, int dv, const float* lam, float eps, float mult, const int* seq_row,
+                           void* out, int out_dtype, cudaStream_t stream) {
+  if (N <= 0) return FZ_OK;
+  if (H <= 0 || dv <= 0) return FZ_BAD_SHAPE;
+  const int W = H < 8 ? H : 8;
+  if (out_dtype == FZ_F32) fz_launch(combine_maps_kernel<float>, dim3(N), dim3(32 * W), 0, stream, a, H, dv, lam, eps, mult, seq_row, (float*)out);
+  else if (out_dtype == FZ_BF16) fz_launch(combine_maps_kernel<__nv_bfloat16>, dim3(N), dim3(32 * W), 0, stream, a, H, dv, lam, eps, mult, seq_row, (__nv_bfloat16*)out);
+  else return FZ_BAD_DTYPE;
+  FZ_LAUNCH_CHECK();
+  return FZ_OK;
 }
 
 // The padded key size of the recurrent state, (slots, heads, value_dim, this): 8 times a power of two, at most 256.
@@ -1456,9 +1532,9 @@ static size_t retention_smem(int dk, int R, int cols, int rotated, int tch) {
   const int dkp = R * DPT;
   return sizeof(float) * (size_t)tch * ((size_t)2 * dkp + cols + 2 * dk + cols + rotated);
 }
-static size_t delta_smem(int dk, int R, int cols, int tch, size_t elem) {
+static size_t delta_smem(int dk, int R, int cols, int tch, size_t elem, bool head) {
   const int dkp = R * DPT;
-  return sizeof(float) * (size_t)tch * ((size_t)3 * dkp + cols + 1 + dk + 1) + elem * (size_t)tch * (2 * ((dk + 1) & ~1) + ((cols + 1) & ~1)) + 16;
+  return sizeof(float) * (size_t)tch * ((size_t)2 * dkp + (head ? 4 : dkp) + cols + 1 + (head ? 1 : dk) + 1) + elem * (size_t)tch * (2 * ((dk + 1) & ~1) + ((cols + 1) & ~1)) + 16;
 }
 
 template <int R>
@@ -1487,33 +1563,36 @@ FZ_API int fz_retention_scan(const float* proj, int ld, int H, int dk, int dv, c
 #undef FZ_CALL
 }
 
-template <typename T, int R>
-static int launch_delta(const void* qkv, int H, int Hk, int dk, int dv, const float* high, int ldh, const float* beta,
+template <typename T, int R, bool HEAD>
+static int launch_delta(const void* qkv, int H, int Hk, int dk, int dv, const float* high, int ldh, const float* beta, int ldb,
                         const float* a_log, const float* dt_bias, float unit_eps, float q_scale, float* state, const int* seg,
                         int n_seg, float* out, cudaStream_t stream) {
   const int threads = scan_threads(dv, R), cols = threads / R * DC;
-  const int tch = delta_smem(dk, R, cols, 16, sizeof(T)) <= 48 * 1024 ? 16 : 8;
-  const size_t smem = delta_smem(dk, R, cols, tch, sizeof(T));
+  const int tch = delta_smem(dk, R, cols, 16, sizeof(T), HEAD) <= 48 * 1024 ? 16 : 8;
+  const size_t smem = delta_smem(dk, R, cols, tch, sizeof(T), HEAD);
   static size_t allowed = 48 * 1024;
-  int st = allow_smem(gated_delta_scan_kernel<T, R>, smem, allowed);
+  int st = allow_smem(gated_delta_scan_kernel<T, R, HEAD>, smem, allowed);
   if (st != FZ_OK) return st;
-  fz_launch(gated_delta_scan_kernel<T, R>, dim3(n_seg, H, (dv + cols - 1) / cols), dim3(threads), smem, stream, (const T*)qkv,
-            H, Hk, dk, dv, tch, high, ldh, beta, a_log, dt_bias, unit_eps, q_scale, state, seg, out);
+  fz_launch(gated_delta_scan_kernel<T, R, HEAD>, dim3(n_seg, H, (dv + cols - 1) / cols), dim3(threads), smem, stream, (const T*)qkv,
+            H, Hk, dk, dv, tch, high, ldh, beta, ldb, a_log, dt_bias, unit_eps, q_scale, state, seg, out);
   FZ_LAUNCH_CHECK();
   return FZ_OK;
 }
 
+// high: the first decay input of row 0 (head_decay: one per head, else H dk of them), rows ldh floats apart; beta likewise.
 FZ_API int fz_gated_delta_scan(const void* qkv, int dtype, int H, int Hk, int dk, int dv, const float* high, int ldh,
-                               const float* beta, const float* a_log, const float* dt_bias, float unit_eps, float q_scale,
-                               float* state, const int* seg, int n_seg, float* out, cudaStream_t stream) {
+                               const float* beta, int ldb, const float* a_log, const float* dt_bias, float unit_eps, float q_scale,
+                               int head_decay, float* state, const int* seg, int n_seg, float* out, cudaStream_t stream) {
   if (n_seg <= 0) return FZ_OK;
   if (H <= 0 || H > 65535 || Hk <= 0 || H % Hk || dv <= 0 || fz_recurrent_key_pad(dk) < 0) return FZ_BAD_SHAPE;
-#define FZ_CALL_F(R) launch_delta<float, R>(qkv, H, Hk, dk, dv, high, ldh, beta, a_log, dt_bias, unit_eps, q_scale, state, seg, n_seg, out, stream)
-#define FZ_CALL_B(R) launch_delta<__nv_bfloat16, R>(qkv, H, Hk, dk, dv, high, ldh, beta, a_log, dt_bias, unit_eps, q_scale, state, seg, n_seg, out, stream)
+#define FZ_ARGS qkv, H, Hk, dk, dv, high, ldh, beta, ldb, a_log, dt_bias, unit_eps, q_scale, state, seg, n_seg, out, stream
+#define FZ_CALL_F(R) (head_decay ? launch_delta<float, R, true>(FZ_ARGS) : launch_delta<float, R, false>(FZ_ARGS))
+#define FZ_CALL_B(R) (head_decay ? launch_delta<__nv_bfloat16, R, true>(FZ_ARGS) : launch_delta<__nv_bfloat16, R, false>(FZ_ARGS))
   if (dtype == FZ_F32) { FZ_BY_LANES(lanes_per_column(dk), FZ_CALL_F) }
   if (dtype == FZ_BF16) { FZ_BY_LANES(lanes_per_column(dk), FZ_CALL_B) }
 #undef FZ_CALL_F
 #undef FZ_CALL_B
+#undef FZ_ARGS
   return FZ_BAD_DTYPE;
 }
 
@@ -1610,12 +1689,19 @@ FZ_API int fz_router_topk(const float* logits, int ld, int N, int E, int top, in
   return FZ_OK;
 }
 
+// choice (N, top) and hin (N, D) of hin_dtype: see the kernel; choice null: no such experts.
 FZ_API int fz_moe_combine(const float* terms, const float* w, int top, const float* shared, const float* gl, int ldg, int col,
-                          const int* seq_row, float* out, int N, int D, const float* add, float scale, cudaStream_t stream) {
+                          const int* seq_row, float* out, int N, int D, const float* add, float scale, const int* choice,
+                          int n_experts, const void* hin, int hin_dtype, cudaStream_t stream) {
   if (N <= 0 || D <= 0) return FZ_OK;
+  if (choice != nullptr && hin == nullptr) return FZ_BAD_SHAPE;
   const int by = (D + 1023) / 1024 > 0 ? (D + 1023) / 1024 : 1;
-  fz_launch(moe_combine_kernel, dim3(N, by), dim3(256), 0, stream, terms, w, top, shared, gl, ldg, col, seq_row, out, N, D, add,
-            scale);
+  if (hin_dtype == FZ_BF16)
+    fz_launch(moe_combine_kernel<__nv_bfloat16>, dim3(N, by), dim3(256), 0, stream, terms, w, top, shared, gl, ldg, col, seq_row, out, N,
+              D, add, scale, choice, n_experts, (const __nv_bfloat16*)hin);
+  else
+    fz_launch(moe_combine_kernel<float>, dim3(N, by), dim3(256), 0, stream, terms, w, top, shared, gl, ldg, col, seq_row, out, N, D, add,
+              scale, choice, n_experts, (const float*)hin);
   FZ_LAUNCH_CHECK();
   return FZ_OK;
 }

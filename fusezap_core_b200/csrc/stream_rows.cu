@@ -145,7 +145,8 @@ depth_average_norm_kernel(float* __restrict__ streams, int L1, int depth, const 
   for (int d = threadIdx.x; d < D; d += blockDim.x) hr[d] = Cvt<TH>::from_f(w[d] * (avg[d] * scale));
 }
 
-// out[n, j] = act(src[n, off + j]). kind 0: tanh, 1: sigmoid, 2: silu, 3: the tanh form of gelu.
+// out[n, j] = act(src[n, off + j]). kind 0: tanh, 1: sigmoid, 2: silu, 3: the tanh form of gelu, 4: as it is,
+// 5: max(z, 0)^2.
 template <typename T>
 __global__ void __launch_bounds__(256)
 activate_kernel(const float* __restrict__ src, int ld, int off, int kind, T* __restrict__ out, int W, long long total) {
@@ -160,6 +161,7 @@ activate_kernel(const float* __restrict__ src, int ld, int off, int kind, T* __r
     else if (kind == 1) v = 1.0f / (1.0f + expf(-z));
     else if (kind == 2) v = z / (1.0f + expf(-z));
     else if (kind == 3) v = 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+    else if (kind == 5) { v = fmaxf(z, 0.f); v *= v; }
     else v = z;
     out[idx] = Cvt<T>::from_f(v);
   }
@@ -170,6 +172,7 @@ __device__ __forceinline__ float act_of(float z, int kind) {
   if (kind == 1) return 1.0f / (1.0f + expf(-z));
   if (kind == 2) return z / (1.0f + expf(-z));
   if (kind == 3) return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+  if (kind == 5) { const float v = fmaxf(z, 0.f); return v * v; }
   return z;
 }
 __device__ __forceinline__ void st4(float* d, float4 v) { *(float4*)d = v; }
@@ -319,7 +322,7 @@ FZ_API int fz_depth_average_norm(float* streams, int L1, int depth, const float*
 FZ_API int fz_activate(const float* src, int ld, int off, int kind, void* out, int dtype, int N, int W, cudaStream_t stream) {
   const long long total = (long long)N * W;
   if (total <= 0) return FZ_OK;
-  if (kind < 0 || kind > 4 || off < 0 || off + W > ld) return FZ_BAD_SHAPE;
+  if (kind < 0 || kind > 5 || off < 0 || off + W > ld) return FZ_BAD_SHAPE;
   if (W % 4 == 0 && off % 4 == 0 && ld % 4 == 0 && (((uintptr_t)src | (uintptr_t)out) & 15) == 0 && (dtype == FZ_F32 || dtype == FZ_BF16)) {
     const long long quads = total / 4;
     long long vb = (quads + 255) / 256;
@@ -343,7 +346,7 @@ FZ_API int fz_gate_multiply(const void* x, const float* gate, int ld, int off, i
                             cudaStream_t stream) {
   const long long total = (long long)N * W;
   if (total <= 0) return FZ_OK;
-  if (kind < 0 || kind > 4 || off < 0 || off + W > ld) return FZ_BAD_SHAPE;
+  if (kind < 0 || kind > 5 || off < 0 || off + W > ld) return FZ_BAD_SHAPE;
   if (W % 4 == 0 && off % 4 == 0 && ld % 4 == 0 && (((uintptr_t)x | (uintptr_t)gate | (uintptr_t)out) & 15) == 0 &&
       (dtype == FZ_F32 || dtype == FZ_BF16)) {
     const long long quads = total / 4;

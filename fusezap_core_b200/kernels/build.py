@@ -33,6 +33,8 @@ LIBRARIES: dict[str, list[str]] = {
     # the selective state space scan, token by token (both dtypes)
     "fzb200_ssd": ["ssd.cu"],
     "fzb200_ssd_tc": ["ssd_chunk.cu"],                                       # bfloat16 only: long portions of that scan on tensor cores
+    # the scan of gated linear attention, token by token (both dtypes)
+    "fzb200_gla": ["gla.cu"],
     # depth-averaged layers, the hashed pair embedding, a columnwise activation (both dtypes)
     "fzb200_rows": ["stream_rows.cu"],
     "fzb200_seq_tc": ["attn_sink_mma.cu"],                                   # bfloat16 only: that attention on tensor cores

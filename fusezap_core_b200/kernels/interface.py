@@ -52,10 +52,13 @@ class Ops:
         raise NotImplementedError
 
     def add_layernorm(self, x: torch.Tensor, delta: torch.Tensor | None, extra: torch.Tensor | None, weight: torch.Tensor,
-                      eps: float, h: torch.Tensor, rows: torch.Tensor | None = None) -> None:
+                      eps: float, h: torch.Tensor, rows: torch.Tensor | None = None, bias: torch.Tensor | None = None,
+                      post: tuple | None = None) -> None:
         """rows None: x = (x + delta) + extra (each if given), in place; h[n] = T(weight * (x[n] - m) / sqrt(mean((x[n] -
         m)^2) + eps)), m = mean(x[n]). rows (int32 (R,), -1 = none): h[r] is computed from x[rows[r]] + delta[rows[r]]; x is
-        not written and extra must be None. weight (D,) float32; delta, extra (N, D) float32."""
+        not written and extra must be None. weight (D,) float32; delta, extra (N, D) float32. bias (D,) float32: added to h
+        before it is rounded. post (weight, bias or None, eps): delta stands for its own layer norm, weight * (delta - mean) /
+        sqrt(mean((delta - mean)^2) + eps) + bias of its row, in everything above."""
         raise NotImplementedError
 
     def select_tokens(self, tokens: torch.Tensor, src: torch.Tensor, prev_ids: torch.Tensor, out: torch.Tensor) -> None:
@@ -134,9 +137,14 @@ class Ops:
         (alpha 1, an infinite limit and up_shift 0 give silu(g) * u.)"""
         raise NotImplementedError
 
+    def grouped_linear_act(self, h: torch.Tensor, w: torch.Tensor, route: Any, y: torch.Tensor, activation: str) -> None:
+        """w: (E, I, K). For every pair (row n, expert e) of the route: y[pair] = T(act(w[e] . h[n])), (N * top, I) T in the
+        route's own order of pairs; activation "relu2": max(z, 0)^2; float32."""
+        raise NotImplementedError
+
     def grouped_linear_scatter(self, y: torch.Tensor, w: torch.Tensor, route: Any, out: torch.Tensor) -> None:
         """w: (E, D, I). out[n * top + k] = w[e] . y[pair], float32 (N * top, D), for the pair of row n's k-th choice;
-        rows of padding are zero."""
+        rows of padding are zero. Choices without a pair (see `route_by_scores`) leave their rows as they are."""
         raise NotImplementedError
 
     # ---- recurrent mixers, windowed attention with a sink, routed experts
@@ -159,12 +167,23 @@ class Ops:
 
     def gated_delta_scan(self, qkv: torch.Tensor, heads: int, key_heads: int, key_dim: int, value_dim: int,
                          high: torch.Tensor, beta: torch.Tensor, a_log: torch.Tensor, dt_bias: torch.Tensor,
-                         unit_eps: float, query_scale: float, state: torch.Tensor, meta: Any, out: torch.Tensor) -> None:
-        """qkv: (N, 2 Hk dk + H dv) T = [q | k | v]; high: (N, >= H dk) float32 whose first H dk columns are the decay
-        inputs a; beta: (N, H) float32 (before the sigmoid); a_log (H,), dt_bias (H dk,) float32. Per portion, token by
+                         unit_eps: float, query_scale: float, state: torch.Tensor, meta: Any, out: torch.Tensor,
+                         head_decay: bool = False, high_offset: int = 0, beta_offset: int = 0) -> None:
+        """qkv: (N, 2 Hk dk + H dv) T = [q | k | v]; high: float32 (N, any width) whose H dk columns from high_offset on are
+        the decay inputs a; beta: float32 (N, any width), H columns from beta_offset on (before the sigmoid); head_decay: one
+        decay input (and dt_bias) per head instead of one per key channel. a_log (H,), dt_bias (H dk,) float32. Per portion, token by
         token, per head h (key head h // (H / Hk)): q^ = q / sqrt(sum q^2 + unit_eps) * query_scale, k^ likewise without
         the scale, b = sigmoid(beta), g = exp(-exp(a_log[h]) * softplus(a[h] + dt_bias[h])) per key channel;
         S = g * S (rows), u = b * (v - S^T k^), S = S + k^ u^T, out[n, h] = S^T q^. float32 throughout; out (N, H dv)."""
+        raise NotImplementedError
+
+    def channel_decay_scan(self, proj: torch.Tensor, heads: int, key_dim: int, value_dim: int, decay_in: torch.Tensor,
+                           decay_root: float, query_scale: float, state: torch.Tensor, meta: Any, out: torch.Tensor) -> None:
+        """proj: (N, >= H (2 dk + dv)) float32, a row = [q heads | k heads | v heads | ...]; decay_in (N, H dk) float32. Per
+        portion (meta.seg), token by token, per head, from the state of the portion's slot: S = diag(alpha) S + k v^T,
+        out[n, h] = S^T (q * query_scale) with alpha = sigmoid(decay_in)^(1 / decay_root) per key channel. float32 throughout;
+        out (N, H dv); the state (`recurrent_state_shape`) is that after the portion's last token. Rows of padding are left
+        as they are. A table may compute a long portion in blocks of tokens, in another order of the same sums."""
         raise NotImplementedError
 
     def head_norm_gate(self, o: torch.Tensor, heads: int, value_dim: int, weight: torch.Tensor | None, eps: float,
@@ -192,6 +211,18 @@ class Ops:
         blocks of tokens, in another order of the same sums."""
         raise NotImplementedError
 
+    def check_differential_attention(self, num_heads: int, num_kv_heads: int, map_dim: int, value_dim: int) -> None:
+        """Raise ValueError if `differential_attention` cannot take these sizes."""
+        raise NotImplementedError
+
+    def differential_attention(self, q: torch.Tensor, cache: Any, meta: Any, out: torch.Tensor, num_heads: int, num_kv_heads: int,
+                               map_dim: int, value_dim: int, scale: float, lam: torch.Tensor, eps: float, mult: float) -> None:
+        """q: (N, H, 2, d) T, cached keys (pages, G, page, 2 d), values (pages, G, page, dv). For map i of head h (kv head
+        h // (H / G)): a_i = sum_j softmax_j((q[n, h, i] . k_j[i d : (i + 1) d]) * scale) v_j over the keys j <= p of the row's
+        own request; with o = a_1 - lam[0] * a_2: out[n, h] = T(o / sqrt(mean(o^2) + eps) * mult), the mean over dv; float32
+        up to the one rounding. Padding rows give zeros."""
+        raise NotImplementedError
+
     def general_delta_scan(self, proj: torch.Tensor, heads: int, key_dim: int, value_dim: int, remove_offset: int,
                            decay_in: torch.Tensor, decay_bias: torch.Tensor, remove_bias: torch.Tensor, decay_rate: float,
                            unit_eps: float, state: torch.Tensor, meta: Any, out: torch.Tensor) -> None:
@@ -205,7 +236,7 @@ class Ops:
 
     def activate(self, src: torch.Tensor, offset: int, kind: str, out: torch.Tensor) -> None:
         """out[n, j] = T(act(src[n, offset + j])) for the columns of out; src float32 (N, any width); kind "tanh",
-        "sigmoid", "silu", "gelu_tanh", "identity", computed in float32 and rounded once. Padding rows need not be zero."""
+        "sigmoid", "silu", "gelu_tanh", "identity", "relu2" (max(z, 0)^2), computed in float32 and rounded once. Padding rows need not be zero."""
         raise NotImplementedError
 
     def gate_multiply(self, x: torch.Tensor, gate: torch.Tensor, gate_offset: int, kind: str, out: torch.Tensor) -> None:
@@ -282,6 +313,17 @@ class Ops:
         only if also floor(j / s) = floor(p / s) (keep_first must then be 0)."""
         raise NotImplementedError
 
+    def normed_sum(self, terms: list, norm_weights: list, weights: list, eps: float, out: torch.Tensor) -> None:
+        """out = sum_i weights[i] * (norm_weights[i] * terms[i] / sqrt(mean(terms[i]^2) + eps)), the mean over a row; all
+        float32, terms and out (N, D), norm_weights (D,), one to four terms added in the order given."""
+        raise NotImplementedError
+
+    def linear_act(self, a: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None, out: torch.Tensor, activation: str) -> bool:
+        """`linear` whose result passes an activation ("relu2": max(y, 0)^2) before its one rounding. Optional: returns
+        False, having done nothing, if this table has no such kernel for these sizes; the caller then runs `linear` into
+        float32 and `activate`."""
+        return False
+
     def weighted_sum(self, terms: list, weights: list, out: torch.Tensor) -> None:
         """out = sum_i weights[i] * terms[i], float32 (N, D), each product rounded, added in the order given."""
         raise NotImplementedError
@@ -289,7 +331,7 @@ class Ops:
     def route_by_scores(self, logits: torch.Tensor, num_experts: int, top: int, groups: int, keep_groups: int,
                         renormalize: bool, meta: Any, weights: torch.Tensor, align: int = 1, scoring: str = "softmax",
                         correction: torch.Tensor | None = None, group_top: int = 1, sum_eps: float = 0.0,
-                        scale: float = 1.0) -> Any:
+                        scale: float = 1.0, identity: int = 0) -> Any:
         """logits: (N, >= E) float32, the first E columns are router logits. s = softmax over them; the experts form
         `groups` equal groups of neighbours, a group's score is its largest s, only experts of the keep_groups best groups
         (lower index first among equals) can be chosen; of those the `top` with the largest s (lower index first among
@@ -297,16 +339,19 @@ class Ops:
         scoring "sigmoid": s = sigmoid(logit). correction (E,) float32: experts and groups are compared by s + correction,
         the weights stay s. group_top 2: a group's score is the sum of its two largest (of its one, if it has one).
         sum_eps: added to the sum that renormalize divides by; scale: multiplies the weights last.
+        identity i > 0: the last i of the num_experts are experts without products of their own (their output is their
+        input): they are scored and chosen like the others but have no pairs in the route.
         Returns the route of the (row, choice) pairs sorted by expert, as `route_by_table` does."""
         raise NotImplementedError
 
     def moe_combine(self, terms: torch.Tensor, weights: torch.Tensor, shared: torch.Tensor | None,
                     gate_logits: torch.Tensor | None, gate_column: int, out: torch.Tensor,
-                    add: torch.Tensor | None = None, scale: float = 1.0) -> None:
+                    add: torch.Tensor | None = None, scale: float = 1.0, handed_on: tuple | None = None) -> None:
         """out[n] = sum_k weights[n, k] * terms[n * top + k] (+ sigmoid(gate_logits[n, gate_column]) * shared[n]); all
         float32; terms (N top, D), weights (N, top), shared (N, D), the sum in rising k and the shared term last
         (gate_logits None: the shared term is added as it is). add (N, D) float32 and scale: out = scale * (add + the
-        sum). Padding rows give zeros."""
+        sum). Padding rows give zeros. handed_on (route of `route_by_scores`, first, h), h (N, D) T or float32: where the k-th
+        choice of row n is expert `first` or a later one, the term is h[n] and terms[n * top + k] is not read."""
         raise NotImplementedError
 
     def linear(self, a: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None, out: torch.Tensor) -> None:

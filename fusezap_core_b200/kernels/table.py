@@ -24,7 +24,7 @@ _DEVICE_ERRORS = {1: "a token id lies outside the embedding table", 2: "a positi
                   16: "a selected row lies outside the step"}
 
 
-_ACTIVATIONS = {"tanh": 0, "sigmoid": 1, "silu": 2, "gelu_tanh": 3, "identity": 4}
+_ACTIVATIONS = {"tanh": 0, "sigmoid": 1, "silu": 2, "gelu_tanh": 3, "identity": 4, "relu2": 5}
 RGLRU_COOK_ROWS = 4  # recurrent unit: steps whose longest portion is longer compute the recurrence's coefficients in a launch of their own
 SSD_CHUNK_ROWS = 16     # state space scan (bfloat16): portions of this many rows and more go to the tensor-core kernel where the sizes allow it
 SSD_SPREAD_ROWS = 16    # state space scan: in steps whose longest portion has this many rows a head's columns are spread over blocks of
@@ -126,7 +126,7 @@ class CudaOps(Ops):
         if self.dtype == torch.bfloat16:
             self.tc = load("fzb200_tc")      # tcgen05 / TMA kernels
         self.use_tensor_cores = self.tc is not None
-        self._attn_tc = self._mix = self._mix_tc = self._latent = self._latent_tc = self._seq = self._seq_tc = self._rows = self._ssd = self._ssd_tc = None   # libraries loaded (and built) when a part first asks for their kernels
+        self._attn_tc = self._mix = self._mix_tc = self._latent = self._latent_tc = self._seq = self._seq_tc = self._rows = self._ssd = self._ssd_tc = self._gla = None   # libraries loaded (and built) when a part first asks for their kernels
         self.prefill_tcgen05 = True        # False: long portions on the mma.sync flash-attention kernel
         self.fuse_swiglu = True            # gate/up product and SwiGLU in one kernel where the sizes allow it
         self.fuse_argmax = True            # lm_head product and argmax in one pass where no logits are asked for
@@ -206,6 +206,13 @@ class CudaOps(Ops):
         if self._ssd is None:
             self._ssd = load("fzb200_ssd")
         return self._ssd
+
+    @property
+    def gla(self):
+        """The scan of gated linear attention."""
+        if self._gla is None:
+            self._gla = load("fzb200_gla")
+        return self._gla
 
     @property
     def ssd_tc(self):
@@ -397,9 +404,17 @@ class CudaOps(Ops):
                                              c_float(eps), _p(self.err), self._stream()), "add_rmsnorm",
                     n_out * d * (4 + (8 if delta is not None and rows is None else 4 if delta is not None else 0) + h.element_size()))
 
-    def add_layernorm(self, x, delta, extra, weight, eps, h, rows=None) -> None:
+    def add_layernorm(self, x, delta, extra, weight, eps, h, rows=None, bias=None, post=None) -> None:
         self._want(x, "x", (torch.float32,), 2)
         self._want(weight, "norm weight", (torch.float32,), 1)
+        post_w, post_b, post_eps = post if post is not None else (None, None, 0.0)
+        if post_w is not None and delta is None:
+            raise KernelError("add_layernorm: a post norm without a term that it norms")
+        for t, name in ((bias, "norm bias"), (post_w, "post norm weight"), (post_b, "post norm bias")):
+            if t is not None:
+                self._want(t, name, (torch.float32,), 1)
+                if t.shape[0] != x.shape[1]:
+                    raise KernelError(f"add_layernorm: {name} {tuple(t.shape)} for rows of {x.shape[1]}")
         self._want(h, "h", (torch.float32, torch.bfloat16), 2)
         for t, name in ((delta, "delta"), (extra, "extra")):
             if t is not None:
@@ -416,9 +431,45 @@ class CudaOps(Ops):
         if h.shape != (n_out, d) or weight.shape[0] != d:
             raise KernelError(f"add_layernorm: h {tuple(h.shape)}, expected {(n_out, d)}; weight {tuple(weight.shape)}")
         adds = (delta is not None) + (extra is not None)
-        self._check(self.core.fz_add_layernorm(_p(x), _p(delta), _p(extra), _p(weight), _p(h), c_int(_CODE[h.dtype]), _p(rows),
-                                               c_int(n_out), c_int(n_src), c_int(d), c_float(eps), _p(self.err), self._stream()),
-                    "add_layernorm", n_out * d * (4 + 4 * adds + (4 if adds and rows is None else 0) + h.element_size()))
+        self._check(self.core.fz_add_layernorm(_p(x), _p(delta), _p(extra), _p(weight), _p(bias), _p(h), c_int(_CODE[h.dtype]), _p(rows),
+                                               c_int(n_out), c_int(n_src), c_int(d), c_float(eps), _p(post_w), _p(post_b),
+                                               c_float(post_eps), _p(self.err), self._stream()),
+                    "add_layernorm" if post_w is None else "add_layernorm (post norm)", n_out * d * (4 + 4 * adds + (4 if adds and rows is None else 0) + h.element_size()))
+
+    def normed_sum(self, terms, norm_weights, weights, eps, out) -> None:
+        if not 1 <= len(terms) <= 4 or len(weights) != len(terms) or len(norm_weights) != len(terms):
+            raise KernelError(f"normed_sum: {len(terms)} terms, {len(norm_weights)} norm weights and {len(weights)} weights (1 to 4 of each)")
+        self._want(out, "sum", (torch.float32,), 2)
+        for t, w in zip(terms, norm_weights):
+            self._want(t, "term", (torch.float32,), 2)
+            self._want(w, "norm weight", (torch.float32,), 1)
+            if t.shape != out.shape or w.shape[0] != out.shape[1]:
+                raise KernelError(f"normed_sum: term {tuple(t.shape)}, norm weight {tuple(w.shape)}, out {tuple(out.shape)}")
+        pad = [None] * (4 - len(terms))
+        n, d = out.shape
+        self._check(self.core.fz_normed_sum(*(_p(t) for t in [*terms, *pad]), *(_p(w) for w in [*norm_weights, *pad]),
+                                            *(c_float(w) for w in [*weights, *([0.0] * len(pad))]), c_int(len(terms)), _p(out),
+                                            c_int(n), c_int(d), c_float(eps), self._stream()), "normed_sum",
+                    n * d * 4 * (len(terms) + 1))
+
+    def linear_act(self, a, w, bias, out, activation: str) -> bool:
+        if activation != "relu2" or not (self.use_tensor_cores and self.fuse_swiglu and self.dtype == torch.bfloat16):
+            return False
+        m, k = a.shape
+        n = w.shape[0]
+        if self.tc.fz_gemm_tc_check(_p(a), _p(w), c_int(m), c_int(n), c_int(k)) != 0:
+            return False
+        self._want(a, "linear input", (self.dtype,), 2)
+        self._want(w, "linear weight", (self.dtype,), 2)
+        self._want(out, "linear output", (torch.float32, self.dtype), 2)
+        if bias is not None:
+            self._want(bias, "linear bias", (torch.float32,), 1)
+        if w.shape[1] != k or out.shape != (m, n) or (bias is not None and bias.shape[0] != n):
+            raise KernelError(f"linear_act: a {tuple(a.shape)}, w {tuple(w.shape)}, out {tuple(out.shape)}")
+        self._check(self.tc.fz_gemm_tc_relu2(_p(a), _p(w), _p(bias), _p(out), c_int(_CODE[out.dtype]), c_int(m), c_int(n), c_int(k),
+                                             _p(self.err), self._stream()), "linear_act (tensor cores)",
+                    ideal_linear_bytes(m, n, k, 2, 2, out.element_size()))
+        return True
 
     def linear(self, a, w, bias, out) -> None:
         self._want(a, "linear input", (self.dtype,), 2)
@@ -846,8 +897,9 @@ class CudaOps(Ops):
         self._want(table, "expert table", (torch.int32,), 2)
         return self._sort_pairs(token_ids, token_ids.shape[0], meta, table, num_experts, align)
 
-    def _sort_pairs(self, token_ids, n, meta, table, num_experts, align):
-        """The step's (row, choice) pairs sorted by expert table[id of the row, choice] (no ids: table[row, choice])."""
+    def _sort_pairs(self, token_ids, n, meta, table, num_experts, align, skip: int = 0):
+        """The step's (row, choice) pairs sorted by expert table[id of the row, choice] (no ids: table[row, choice]);
+        choices of the `skip` experts after the last have no pairs."""
         top = table.shape[1]
         # row tiles of 64 pairs; of 16 where an expert gets few rows (decoded tokens) and the tensor-core kernels run
         tile = int(self.mix.fz_grouped_tile_rows())
@@ -860,7 +912,7 @@ class CudaOps(Ops):
         idx = self._scratch("expert route", 2 * n * top + 3 * max_tiles, torch.int32)
         a_idx, c_idx, tiles = idx[:n * top], idx[n * top: 2 * n * top], idx[2 * n * top: 2 * n * top + 3 * max_tiles]
         self._check(self.mix.fz_route_by_table(_p(token_ids), _p(meta.seq_row), _p(table), c_int(n), c_int(table.shape[0]),
-                                               c_int(top), c_int(num_experts), _p(a_idx), _p(c_idx), _p(tiles),
+                                               c_int(top), c_int(num_experts), c_int(skip), _p(a_idx), _p(c_idx), _p(tiles),
                                                c_int(max_tiles), c_int(tile), _p(self.err), self._stream()), "route_by_table")
         return (a_idx, c_idx, tiles, max_tiles, n, top, meta.seq_row, tile)
 
@@ -870,7 +922,7 @@ class CudaOps(Ops):
                                                     c_longlong(0), c_int(n_out), c_int(k)) == 0)
 
     def grouped_linear_glu(self, h, w, route, y, alpha, limit, up_shift: float = 1.0) -> None:
-        a_idx, c_idx, tiles, max_tiles, n, top, seq_row, tile = route
+        a_idx, c_idx, tiles, max_tiles, n, top, seq_row, tile = route[:8]
         self._want(h, "expert input", (self.dtype,), 2)
         self._want(w, "expert gate/up weights", (self.dtype,), 3)
         self._want(y, "expert activation", (self.dtype,), 2)
@@ -890,8 +942,27 @@ class CudaOps(Ops):
                                                self._stream()),
                     "grouped_linear_glu", (min(w.shape[0], n * top) * 2 * inter * k + n * k + n * top * inter) * h.element_size())
 
+    def grouped_linear_act(self, h, w, route, y, activation: str) -> None:
+        a_idx, c_idx, tiles, max_tiles, n, top, seq_row, tile = route[:8]
+        if activation != "relu2":
+            raise KernelError(f"grouped_linear_act: activation {activation!r} is not 'relu2'")
+        self._want(h, "expert input", (self.dtype,), 2)
+        self._want(w, "expert up weights", (self.dtype,), 3)
+        self._want(y, "expert activation", (self.dtype,), 2)
+        k, inter = h.shape[1], w.shape[1]
+        if h.shape[0] != n or w.shape[2] != k or tuple(y.shape) != (n * top, inter):
+            raise KernelError(f"grouped_linear_act: h {tuple(h.shape)}, w {tuple(w.shape)}, y {tuple(y.shape)}")
+        nbytes = (min(w.shape[0], n * top) * inter * k + n * k + n * top * inter) * h.element_size()
+        tail = (c_int(inter), c_int(k), c_int(2), c_float(0.0), c_float(0.0), c_float(0.0), c_void_p(0), c_int(0), c_int(0), self._stream())
+        if self._grouped_tc(h, k, w, y, inter, inter, k):
+            self._check(self.mix_tc.fz_grouped_linear_tc(_p(h), _p(w), _p(y), _p(tiles), c_int(max_tiles), c_int(tile), _p(a_idx),
+                                                         c_void_p(0), c_int(_CODE[y.dtype]), *tail), "grouped_linear_act (tensor cores)", nbytes)
+            return
+        self._check(self.mix.fz_grouped_linear(_p(h), _p(w), _p(y), _p(tiles), c_int(max_tiles), c_int(tile), _p(a_idx), c_void_p(0),
+                                               c_int(_CODE[self.dtype]), c_int(_CODE[self.dtype]), *tail), "grouped_linear_act", nbytes)
+
     def grouped_linear_scatter(self, y, w, route, out) -> None:
-        a_idx, c_idx, tiles, max_tiles, n, top, seq_row, tile = route
+        a_idx, c_idx, tiles, max_tiles, n, top, seq_row, tile = route[:8]
         self._want(y, "expert activation", (self.dtype,), 2)
         self._want(w, "expert down weights", (self.dtype,), 3)
         self._want(out, "expert outputs", (torch.float32,), 2)
@@ -962,7 +1033,7 @@ class CudaOps(Ops):
             n * heads * (2 * key_dim + 2 * value_dim) * 4 + 2 * meta.n_segments * heads * value_dim * state.shape[3] * 4)
 
     def gated_delta_scan(self, qkv, heads, key_heads, key_dim, value_dim, high, beta, a_log, dt_bias, unit_eps, query_scale,
-                         state, meta, out) -> None:
+                         state, meta, out, head_decay: bool = False, high_offset: int = 0, beta_offset: int = 0) -> None:
         self._want(qkv, "q/k/v", (self.dtype,), 2)
         self._want(high, "decay inputs", (torch.float32,), 2)
         self._want(beta, "beta", (torch.float32,), 2)
@@ -970,19 +1041,38 @@ class CudaOps(Ops):
         self._want(dt_bias, "decay bias", (torch.float32,), 1)
         self._want(out, "delta-rule output", (torch.float32,), 2)
         n = qkv.shape[0]
-        if qkv.shape[1] != 2 * key_heads * key_dim + heads * value_dim or high.shape[0] != n or high.shape[1] < heads * key_dim \
-                or tuple(beta.shape) != (n, heads) or a_log.shape[0] != heads or dt_bias.shape[0] != heads * key_dim \
+        decays = heads if head_decay else heads * key_dim
+        if qkv.shape[1] != 2 * key_heads * key_dim + heads * value_dim or high.shape[0] != n or high_offset < 0 \
+                or high.shape[1] < high_offset + decays or beta.shape[0] != n or beta_offset < 0 \
+                or beta.shape[1] < beta_offset + heads or a_log.shape[0] != heads or dt_bias.shape[0] != decays \
                 or tuple(out.shape) != (n, heads * value_dim) or heads % key_heads:
             raise KernelError(f"gated_delta_scan: qkv {tuple(qkv.shape)}, high {tuple(high.shape)}, beta {tuple(beta.shape)}, "
                               f"out {tuple(out.shape)}")
         self._state(state, heads, key_dim, value_dim, "gated_delta_scan")
         self._meta_rows = meta.seq_row
         self._check(self.seq.fz_gated_delta_scan(
-            _p(qkv), c_int(_CODE[self.dtype]), c_int(heads), c_int(key_heads), c_int(key_dim), c_int(value_dim), _p(high),
-            c_int(high.shape[1]), _p(beta), _p(a_log), _p(dt_bias), c_float(unit_eps), c_float(query_scale), _p(state),
-            _p(meta.seg), c_int(meta.max_segments), _p(out), self._stream()), "gated_delta_scan",
-            n * (qkv.shape[1] * qkv.element_size() + heads * (key_dim + value_dim + 1) * 4)
+            _p(qkv), c_int(_CODE[self.dtype]), c_int(heads), c_int(key_heads), c_int(key_dim), c_int(value_dim),
+            c_void_p(high.data_ptr() + 4 * high_offset), c_int(high.shape[1]), c_void_p(beta.data_ptr() + 4 * beta_offset),
+            c_int(beta.shape[1]), _p(a_log), _p(dt_bias), c_float(unit_eps), c_float(query_scale), c_int(1 if head_decay else 0),
+            _p(state), _p(meta.seg), c_int(meta.max_segments), _p(out), self._stream()), "gated_delta_scan",
+            n * (qkv.shape[1] * qkv.element_size() + (decays + heads * (value_dim + 1)) * 4)
             + 2 * meta.n_segments * heads * value_dim * state.shape[3] * 4)
+
+    def channel_decay_scan(self, proj, heads, key_dim, value_dim, decay_in, decay_root, query_scale, state, meta, out) -> None:
+        self._want(proj, "linear attention projections", (torch.float32,), 2)
+        self._want(decay_in, "decay inputs", (torch.float32,), 2)
+        self._want(out, "linear attention output", (torch.float32,), 2)
+        n, ld = proj.shape
+        if ld < heads * (2 * key_dim + value_dim) or tuple(decay_in.shape) != (n, heads * key_dim) or \
+                tuple(out.shape) != (n, heads * value_dim) or not decay_root > 0:
+            raise KernelError(f"channel_decay_scan: proj {tuple(proj.shape)}, decay inputs {tuple(decay_in.shape)}, out {tuple(out.shape)}")
+        self._state(state, heads, key_dim, value_dim, "channel_decay_scan")
+        self._meta_rows = meta.seq_row
+        self._check(self.gla.fz_channel_decay_scan(
+            _p(proj), c_int(ld), c_int(heads), c_int(key_dim), c_int(value_dim), _p(decay_in), c_float(1.0 / decay_root),
+            c_float(query_scale), _p(state), _p(meta.seg), c_int(getattr(meta, "max_segments", meta.n_segments)), c_int(2 ** 31 - 1),
+            _p(out), self._stream()), "channel_decay_scan",
+            n * heads * (3 * key_dim + 2 * value_dim) * 4 + 2 * meta.n_segments * heads * value_dim * state.shape[3] * 4)
 
     def ssd_scan(self, xbc, heads, groups, state_dim, value_dim, dt, dt_offset, dt_bias, a_log, skip, state, meta, out) -> None:
         self._want(xbc, "x, B and C", (self.dtype,), 2)
@@ -1063,8 +1153,19 @@ class CudaOps(Ops):
         if self.seq.fz_sink_attention_check(c_int(num_heads), c_int(num_kv_heads), c_int(key_dim), c_int(value_dim)) != 0:
             raise ValueError(f"attention sizes not supported: {num_heads} heads, {num_kv_heads} kv heads, key size {key_dim}, "
                              f"value size {value_dim} (need heads % kv_heads == 0 and sizes of 1..512)")
-        if self.use_tensor_cores and self.sink_tensor_cores and key_dim == value_dim and key_dim in (64, 128):
+        if self._sink_mma_sizes(key_dim, value_dim, 1):
             self.seq_tc       # built and loaded with the model, not at its first step
+
+    def check_differential_attention(self, num_heads: int, num_kv_heads: int, map_dim: int, value_dim: int) -> None:
+        self.check_sink_attention(2 * num_heads, num_kv_heads, 2 * map_dim, value_dim)
+        if self._sink_mma_sizes(2 * map_dim, value_dim, 2):
+            self.seq_tc
+
+    def _sink_mma_sizes(self, key_dim: int, value_dim: int, maps: int) -> bool:
+        """Whether the tensor-core kernel takes these sizes of a cached key (all maps of a head) and value, leaving
+        alignment aside."""
+        return self.use_tensor_cores and self.sink_tensor_cores and self.dtype == torch.bfloat16 and key_dim in (64, 128) and \
+            (value_dim in (64, 128) or (maps == 1 and (key_dim, value_dim) == (64, 32)))
 
     def _kv_views(self, cache, hkv: int, dk: int, dv: int):
         k, v = cache.keys, cache.values
@@ -1127,30 +1228,59 @@ class CudaOps(Ops):
             if g.shape[0] != n or g_off < 0 or g_off + num_heads > g_ld:
                 raise KernelError(f"sink_attention: gates {tuple(g.shape)} from column {g_off} for {num_heads} heads")
         k, v = self._kv_views(cache, num_kv_heads, key_dim, value_dim)
-        table = meta.table(cache.group)
         nbytes = 0
         if self._profile is not None:
             seen = sum(min(sg.pos0 + i + 1, (window + keep_first) if window else sg.pos0 + i + 1, (sg.pos0 + i) % span + 1 if span else 1 << 62)
                        for sg in meta.segments for i in range(sg.n))
             nbytes = seen * num_kv_heads * (key_dim + value_dim) * k.element_size() + n * num_heads * (key_dim + value_dim) * q.element_size()
+        self._sink_launch(q, k, v, cache, meta, out, num_heads, num_kv_heads, key_dim, value_dim, scale, window, keep_first, sink,
+                          softcap, (g, g_ld, g_off), span, nbytes)
+
+    def differential_attention(self, q, cache, meta, out, num_heads, num_kv_heads, map_dim, value_dim, scale, lam, eps, mult) -> None:
+        self._want(q, "q", (self.dtype,), 2)
+        self._want(out, "attention output", (self.dtype,), 2)
+        self._want(lam, "lambda", (torch.float32,), 1)
+        n = q.shape[0]
+        if q.shape[1] != num_heads * 2 * map_dim or tuple(out.shape) != (n, num_heads * value_dim) or num_heads % num_kv_heads:
+            raise KernelError(f"differential_attention: q {tuple(q.shape)}, out {tuple(out.shape)}")
+        k, v = self._kv_views(cache, num_kv_heads, 2 * map_dim, value_dim)
+        nbytes = 0
+        if self._profile is not None:
+            nbytes = sum(sg.pos0 + i + 1 for sg in meta.segments for i in range(sg.n)) * num_kv_heads * (2 * map_dim + value_dim) * k.element_size() \
+                + n * num_heads * (2 * map_dim + value_dim) * q.element_size()
+        self._sink_launch(q, k, v, cache, meta, out, num_heads, num_kv_heads, 2 * map_dim, value_dim, scale, 0, 0, None, 0.0,
+                          (None, 0, 0), 0, nbytes, mix=(lam, eps, mult))
+
+    def _sink_launch(self, q, k, v, cache, meta, out, num_heads, num_kv_heads, key_dim, value_dim, scale, window, keep_first, sink,
+                     softcap, gate, span, nbytes, mix=None) -> None:
+        """mix (lambda, eps, mult): two softmax maps per head, halves of the cached key, combined (differential attention)."""
         # A step of single tokens (bfloat16): a row's keys are cut into runs of chunks, one block each, and merged by a
         # second kernel, so that a few rows fill the GPU. Other steps: blocks of consecutive rows of a portion that share
         # their key and value loads. (float32 keeps the one arithmetic for every step: a position's bits do not depend
         # on the cutting.)
+        n = q.shape[0]
+        g, g_ld, g_off = gate
+        table = meta.table(cache.group)
+        what = "sink_attention" if mix is None else "differential_attention"
+        maps = 1 if mix is None else 2
+        lam, mix_eps, mix_mult = mix if mix is not None else (None, 0.0, 0.0)
         max_portion = max(1, int(getattr(meta, "max_portion", 0)) or n)
         n_seg = getattr(meta, "max_segments", meta.n_segments)
         # prompt portions (bfloat16, keys and values of size 64 or 128): tiles of 64 rows on tensor cores
-        if self.use_tensor_cores and self.sink_tensor_cores and self.dtype == torch.bfloat16 and max_portion >= SINK_MMA_ROWS and \
-                key_dim == value_dim and key_dim in (64, 128) and self.seq_tc.fz_sink_attention_mma_check(
-                    c_int(num_heads), c_int(num_kv_heads), c_int(key_dim), c_int(value_dim), _p(k), _p(v), c_longlong(k.stride(0)),
+        if max_portion >= SINK_MMA_ROWS and self._sink_mma_sizes(key_dim, value_dim, maps) and self.seq_tc.fz_sink_attention_mma_check(
+                    c_int(num_heads), c_int(num_kv_heads), c_int(key_dim), c_int(value_dim), c_int(maps), _p(k), _p(v), c_longlong(k.stride(0)),
                     c_longlong(k.stride(1)), c_longlong(k.stride(2))) == 0:
             self._check(self.seq_tc.fz_sink_attention_mma(
                 _p(q), _p(k), _p(v), _p(meta.seg), _p(meta.seq_row), c_int(n_seg), c_int(max_portion), _p(table),
                 c_int(table.shape[1]), c_longlong(k.stride(0)), c_longlong(k.stride(1)), c_longlong(k.stride(2)),
                 c_int(cache.page_size), c_int(k.shape[0]), _p(out), c_int(n), c_int(num_heads), c_int(num_kv_heads),
-                c_int(key_dim), c_float(scale), c_int(window), c_int(keep_first), _p(sink), c_float(softcap), _p(g), c_int(g_ld),
-                c_int(g_off), c_int(span), _p(self.err), self._stream()), "sink_attention (tensor cores)", nbytes)
+                c_int(key_dim), c_int(value_dim), c_float(scale), c_int(window), c_int(keep_first), _p(sink), c_float(softcap), _p(g),
+                c_int(g_ld), c_int(g_off), c_int(span), c_int(maps), _p(lam), c_float(mix_eps), c_float(mix_mult), _p(self.err),
+                self._stream()), what + " (tensor cores)", nbytes)
             return
+        rows_out, heads = out, num_heads * maps
+        if maps > 1:      # both maps' results in float32, combined by a kernel of their own
+            rows_out = self._scratch("attention maps", n * heads * value_dim, torch.float32)
         unit_chunks = units = 0
         part = None
         if self.split_decode_keys and self.dtype == torch.bfloat16 and max_portion == 1:
@@ -1158,16 +1288,20 @@ class CudaOps(Ops):
             reach = min(window or ctx, span or ctx)      # the most keys a row sees, kept first tokens aside
             unit_chunks = 2 if window else max(2, -(-reach // (32 * self.sink_max_runs)))
             units = int(self.seq.fz_sink_attention_units(c_int(window), c_int(keep_first), c_int(ctx), c_int(unit_chunks), c_int(span)))
-            part = self._scratch("sink attention partials", n * num_heads * units * (value_dim + 2), torch.float32)
+            part = self._scratch("sink attention partials", n * heads * units * (value_dim + 2), torch.float32)
         self._check(self.seq.fz_sink_attention(
-            _p(q), _p(k), _p(v), _p(meta.pos), _p(meta.seq_row), _p(meta.seg), c_int(getattr(meta, "max_segments", meta.n_segments)),
+            _p(q), _p(k), _p(v), _p(meta.pos), _p(meta.seq_row), _p(meta.seg), c_int(n_seg),
             c_int(max_portion), _p(table), c_int(table.shape[1]), c_longlong(k.stride(0)),
-            c_longlong(k.stride(1)), c_longlong(k.stride(2)), c_int(cache.page_size), c_int(k.shape[0]), _p(out),
-            c_int(_CODE[self.dtype]), c_int(n), c_int(num_heads), c_int(num_kv_heads), c_int(key_dim), c_int(value_dim),
+            c_longlong(k.stride(1)), c_longlong(k.stride(2)), c_int(cache.page_size), c_int(k.shape[0]), _p(rows_out),
+            c_int(_CODE[self.dtype]), c_int(n), c_int(heads), c_int(num_kv_heads), c_int(key_dim), c_int(value_dim),
             c_float(scale), c_int(window), c_int(keep_first), _p(sink), c_int(unit_chunks), c_int(units), _p(part),
-            c_float(softcap), _p(g), c_int(g_ld), c_int(g_off), c_int(span), _p(self.err), self._stream()), "sink_attention", nbytes)
+            c_float(softcap), _p(g), c_int(g_ld), c_int(g_off), c_int(span), c_int(maps), _p(self.err), self._stream()), what, nbytes)
         if units:
             self.launches += 1      # the merge kernel
+        if maps > 1:
+            self._check(self.seq.fz_combine_maps(_p(rows_out), c_int(n), c_int(num_heads), c_int(value_dim), _p(lam), c_float(mix_eps),
+                                                 c_float(mix_mult), _p(meta.seq_row), _p(out), c_int(_CODE[out.dtype]), self._stream()),
+                        "combine_maps", n * num_heads * value_dim * (8 + out.element_size()))
 
     def general_delta_scan(self, proj, heads, key_dim, value_dim, remove_offset, decay_in, decay_bias, remove_bias, decay_rate,
                            unit_eps, state, meta, out) -> None:
@@ -1320,7 +1454,10 @@ class CudaOps(Ops):
                     out.numel() * 4 * (len(terms) + 1))
 
     def route_by_scores(self, logits, num_experts, top, groups, keep_groups, renormalize, meta, weights, align: int = 1,
-                        scoring: str = "softmax", correction=None, group_top: int = 1, sum_eps: float = 0.0, scale: float = 1.0):
+                        scoring: str = "softmax", correction=None, group_top: int = 1, sum_eps: float = 0.0, scale: float = 1.0,
+                        identity: int = 0):
+        if not 0 <= identity < num_experts:
+            raise KernelError(f"route_by_scores: {identity} of {num_experts} experts hand their input on")
         if scoring not in ("softmax", "sigmoid"):
             raise KernelError(f"route_by_scores: scoring {scoring!r} is not one of 'softmax', 'sigmoid'")
         if correction is not None:
@@ -1338,9 +1475,10 @@ class CudaOps(Ops):
                                             c_int(1 if scoring == "sigmoid" else 0), _p(correction), c_int(group_top),
                                             c_float(sum_eps), c_float(scale), _p(meta.seq_row), _p(choice), _p(weights), self._stream()), "router_topk")
         self._meta_rows = meta.seq_row
-        return self._sort_pairs(None, n, meta, choice, num_experts, align)
+        route = self._sort_pairs(None, n, meta, choice, num_experts - identity, align, identity)
+        return (*route, choice) if identity else route
 
-    def moe_combine(self, terms, weights, shared, gate_logits, gate_column, out, add=None, scale: float = 1.0) -> None:
+    def moe_combine(self, terms, weights, shared, gate_logits, gate_column, out, add=None, scale: float = 1.0, handed_on=None) -> None:
         self._want(terms, "expert terms", (torch.float32,), 2)
         self._want(weights, "router weights", (torch.float32,), 2)
         self._want(out, "feed-forward output", (torch.float32,), 2)
@@ -1364,7 +1502,14 @@ class CudaOps(Ops):
             self._want(add, "other term", (torch.float32,), 2)
             if add.shape != out.shape:
                 raise KernelError(f"moe_combine: other term {tuple(add.shape)}, out {tuple(out.shape)}")
+        choice, first, h = None, 0, None
+        if handed_on is not None:
+            route, first, h = handed_on
+            choice = route[8]
+            self._want(h, "feed-forward input", (torch.float32, torch.bfloat16), 2)
+            if tuple(choice.shape) != (n, top) or h.shape != out.shape:
+                raise KernelError(f"moe_combine: choices {tuple(choice.shape)}, input {tuple(h.shape)}, out {tuple(out.shape)}")
         self._check(self.seq.fz_moe_combine(_p(terms), _p(weights), c_int(top), _p(shared), _p(gate_logits), c_int(ldg),
                                             c_int(gate_column), _p(self._step_rows(n)), _p(out), c_int(n), c_int(d), _p(add), c_float(scale),
-                                            self._stream()),
+                                            _p(choice), c_int(first), _p(h), c_int(_CODE[h.dtype] if h is not None else F32), self._stream()),
                     "moe_combine", n * d * 4 * (top + 1 + (shared is not None) + (add is not None)))

@@ -95,6 +95,22 @@ class PendingSum:
         return self.extra
 
 
+@dataclass
+class PendingNorm:
+    """A pending residual term that passes a norm of its own before it is added to the stream. A norm part that can take
+    both in one pass does; any other consumer calls `resolve`, which hands back the normed term as the one still pending."""
+    delta: torch.Tensor
+    norm: "Norm"
+
+    def fold_into_norm(self, ctx, x, weight, eps, h, rows) -> bool:
+        return False
+
+    def resolve(self, ctx, x) -> torch.Tensor:
+        out = ctx.ws.get("normed_delta", tuple(x.shape), torch.float32)
+        self.norm.forward_into(ctx, self.delta, out)
+        return out
+
+
 class Part:
     # False for a part whose forward depends on the step's host-side metadata (for instance a Python loop over
     # `ctx.meta.segments`): such a step cannot be replayed from a captured CUDA graph, and the engine then runs every

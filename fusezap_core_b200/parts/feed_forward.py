@@ -4,6 +4,8 @@ One product with the rows [gate; up] stacked at load (fusezap/serve/models/llama
 exp(-g))` in 32-bit (fusezap/serve/cuda.py:284-303), then the down product (llama.py:752), whose result is the residual
 term. Optional biases are taken when the checkpoint has them (gate and up together; down). Where the kernel table has
 a fused kernel, the gate/up product and the activation run as one launch and the (N, 2 I) intermediate never exists.
+
+Ungated feed-forward: `down(act(up(h)))`, act = the square of relu, computed from the unrounded 32-bit sums.
 """
 from __future__ import annotations
 import torch
@@ -61,4 +63,35 @@ class SwiGLU(FeedForward):
             ops.swiglu(gu, a, **other)
         delta = ws.get(tag + "delta", (n, self.D), torch.float32)
         ops.linear(a, self.wd, self.bd, delta)
+        return delta
+
+
+@register_feed_forward("ungated")
+class Ungated(FeedForward):
+    def __init__(self, hidden_size: int, intermediate_size: int, names: tuple[str, str] = ("up_proj", "down_proj"),
+                 suffix: str = ".weight", activation: str = "relu2"):
+        """suffix: what follows a matrix's name in the checkpoint. activation: "relu2", max(z, 0)^2."""
+        if activation != "relu2":
+            raise ValueError(f"activation {activation!r} is not 'relu2'")
+        self.D, self.I, self.names, self.suffix, self.activation = hidden_size, intermediate_size, tuple(names), suffix, activation
+        self.wu = self.wd = None
+
+    def tensors(self) -> dict[str, ParamSpec]:
+        u, d = self.names
+        return {f"{u}{self.suffix}": ParamSpec((self.I, self.D)), f"{d}{self.suffix}": ParamSpec((self.D, self.I))}
+
+    def bind(self, tensors, ops) -> None:
+        u, d = self.names
+        self.wu, self.wd = tensors[f"{u}{self.suffix}"], tensors[f"{d}{self.suffix}"]
+
+    def forward(self, ctx, h: torch.Tensor, tag: str = "") -> torch.Tensor:
+        """tag: a prefix for the names of its scratch buffers (a feed-forward that runs inside another one)."""
+        n, ops, ws = h.shape[0], ctx.ops, ctx.ws
+        a = ws.get(tag + "act", (n, self.I), ops.dtype)
+        if not ops.linear_act(h, self.wu, None, a, self.activation):
+            up = ws.get(tag + "up", (n, self.I), torch.float32)
+            ops.linear(h, self.wu, None, up)
+            ops.activate(up, 0, self.activation, a)
+        delta = ws.get(tag + "delta", (n, self.D), torch.float32)
+        ops.linear(a, self.wd, None, delta)
         return delta

@@ -7,14 +7,15 @@ computed in 32-bit and h is rounded once to the activation dtype. With `groups` 
 equal consecutive parts, each by its own mean square; the weight still spans the whole vector. With `offset` the
 multiplier is `offset + w` (a weight stored as its distance from one has offset 1), added in float32 once at load.
 
-LayerNorm: `h = w * (x - mean(x)) / sqrt(mean((x - mean(x))^2) + eps)`, no bias; the same residual add, and where the
-pending term is a `PendingSum` its other stream is added in the same pass.
+LayerNorm: `h = w * (x - mean(x)) / sqrt(mean((x - mean(x))^2) + eps)`, plus a bias where it has one; the same residual
+add, and where the pending term is a `PendingSum` its other stream is added, where it is a `PendingNorm` with a layer norm
+the term is normed, in the same pass.
 """
 from __future__ import annotations
 import torch
 
 from ..weights import ParamSpec
-from .base import Norm, PendingSum, register_norm
+from .base import Norm, PendingNorm, PendingSum, register_norm
 
 
 @register_norm("rmsnorm")
@@ -66,26 +67,46 @@ class RMSNorm(Norm):
 
 @register_norm("layernorm")
 class LayerNorm(Norm):
-    def __init__(self, size: int, eps: float, name: str = "weight"):
-        """name: the weight's tensor name relative to the part ("" when the part's prefix is the whole name)."""
+    def __init__(self, size: int, eps: float, name: str = "weight", bias: str | None = None):
+        """name: the weight's tensor name relative to the part ("" when the part's prefix is the whole name). bias: the
+        name (after the weight's) of a bias added last; None: the norm has none."""
         self.size, self.eps, self.name = size, float(eps), name
+        self.bias_name = None if bias is None else (f"{name}.{bias}" if name else bias)
         self.weight: torch.Tensor | None = None
+        self.bias: torch.Tensor | None = None
 
     def tensors(self) -> dict[str, ParamSpec]:
-        return {self.name: ParamSpec((self.size,), role="vector", init="ones")}
+        out = {self.name: ParamSpec((self.size,), role="vector", init="ones")}
+        if self.bias_name is not None:
+            out[self.bias_name] = ParamSpec((self.size,), role="vector")
+        return out
 
     def bind(self, tensors, ops) -> None:
         self.weight = tensors[self.name].float().contiguous()
+        if self.bias_name is not None:
+            self.bias = tensors[self.bias_name].float().contiguous()
 
     def forward(self, ctx, x, delta, rows=None, n_rows=None):
         n = x.shape[0] if rows is None else (n_rows if n_rows is not None else rows.shape[0])
         h = ctx.ws.get("norm_h" if rows is None else "norm_h_rows", (n, self.size), ctx.ops.dtype)
-        extra = None
-        if isinstance(delta, PendingSum) and rows is None:
+        extra, options = None, {}
+        if isinstance(delta, PendingNorm) and isinstance(delta.norm, LayerNorm):
+            post = delta.norm
+            delta, options["post"] = delta.delta, (post.weight, post.bias, post.eps)
+        elif isinstance(delta, PendingSum) and rows is None:
             delta, extra = delta.delta, delta.extra
+            if hasattr(delta, "resolve"):
+                delta = delta.resolve(ctx, x)
         elif hasattr(delta, "resolve"):
             if rows is not None:
                 raise NotImplementedError("a pending operation on the stream cannot be resolved for selected rows only")
             delta = delta.resolve(ctx, x)
-        ctx.ops.add_layernorm(x, delta, extra, self.weight, self.eps, h, rows)
+        if self.bias is not None:
+            options["bias"] = self.bias
+        ctx.ops.add_layernorm(x, delta, extra, self.weight, self.eps, h, rows, **options)
         return h
+
+    def forward_into(self, ctx, x, h) -> None:
+        """h = norm(x), into a buffer of the caller's."""
+        options = {} if self.bias is None else {"bias": self.bias}
+        ctx.ops.add_layernorm(x, None, None, self.weight, self.eps, h, None, **options)

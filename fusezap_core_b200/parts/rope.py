@@ -51,12 +51,14 @@ class RotaryEncoding(PositionEncoding):
         if head_dim % 2:
             raise ValueError(f"rope needs an even head_dim, got {head_dim}")
         self.head_dim, self.precise = head_dim, bool(precise)
-        if precise and kind not in ("default", "llama3", "yarn"):
-            raise NotImplementedError("precise angles are computed for unscaled, llama3-scaled and yarn-scaled frequencies only")
+        if precise and kind not in ("default", "linear", "llama3", "yarn"):
+            raise NotImplementedError("precise angles are computed for unscaled, linearly, llama3- and yarn-scaled frequencies only")
         if kind == "yarn" and not precise:
             raise NotImplementedError("yarn-scaled frequencies are computed in 64-bit only (precise=True)")
         self.magnitude = float(magnitude)
         self.inv_freq64 = np.float64(theta) ** (-np.arange(0, head_dim, 2, dtype=np.float64) / np.float64(head_dim))
+        if precise and kind == "linear":
+            self.inv_freq64 = self.inv_freq64 / float(factor)
         if precise and kind == "llama3":
             # by wavelength l = 2 pi / f: short ones (l < old / high) stay, long ones (l > old / low) are divided by
             # `factor`, those between are blended with s = (old / l - low) / (high - low); all in 64-bit

@@ -767,3 +767,121 @@ class PlainOpsSpace(PlainOpsGated):
             w = w / (w.sum(-1, keepdim=True) + sum_eps)
         weights.copy_(w * scale)
         return order, meta.seq_row >= 0
+
+
+class PlainOpsSandwich(PlainOpsSpace):
+    """The operations of layers with a norm after each sublayer, of parallel mixers whose results are normed, of the delta
+    rule with one decay per head, of gated linear and differential attention, and of ungated experts beside experts that hand
+    their input on."""
+
+    def add_layernorm(self, x, delta, extra, weight, eps, h, rows=None, bias=None, post=None) -> None:
+        if post is not None:
+            w, b, e = post
+            d = delta - delta.mean(-1, keepdim=True)
+            delta = w.float() * (d * torch.rsqrt((d * d).mean(-1, keepdim=True) + e))
+            if b is not None:
+                delta = delta + b.float()
+        if bias is None:
+            return super().add_layernorm(x, delta, extra, weight, eps, h, rows)
+        y = torch.empty(h.shape, dtype=torch.float32)
+        super().add_layernorm(x, delta, extra, weight, eps, y, rows)
+        y = y + bias.float()
+        if rows is not None:
+            y = torch.where((rows < 0)[:, None], torch.zeros_like(y), y)
+        h.copy_(y.to(h.dtype))
+
+    def normed_sum(self, terms, norm_weights, weights, eps, out) -> None:
+        acc = torch.zeros_like(out)
+        for t, w, s in zip(terms, norm_weights, weights):
+            acc = acc + s * (w.float() * (t * torch.rsqrt((t * t).mean(-1, keepdim=True) + eps)))
+        out.copy_(acc)
+
+    def linear_act(self, a, w, bias, out, activation) -> bool:
+        return False
+
+    def activate(self, src, offset, kind, out) -> None:
+        if kind != "relu2":
+            return super().activate(src, offset, kind, out)
+        out.copy_((torch.relu(src[:, offset: offset + out.shape[1]].float()) ** 2).to(out.dtype))
+
+    def gated_delta_scan(self, qkv, heads, key_heads, key_dim, value_dim, high, beta, a_log, dt_bias, unit_eps, query_scale,
+                         state, meta, out, head_decay=False, high_offset=0, beta_offset=0) -> None:
+        H, dk = heads, key_dim
+        n_in = H if head_decay else H * dk
+        a = high[:, high_offset: high_offset + n_in]
+        if head_decay:      # one number per head, for every key channel of the head
+            a, dt_bias = a.repeat_interleave(dk, 1), dt_bias.repeat_interleave(dk)
+        super().gated_delta_scan(qkv, heads, key_heads, key_dim, value_dim, a.contiguous(), beta[:, beta_offset: beta_offset + H].contiguous(),
+                                 a_log, dt_bias, unit_eps, query_scale, state, meta, out)
+
+    def channel_decay_scan(self, proj, heads, key_dim, value_dim, decay_in, decay_root, query_scale, state, meta, out) -> None:
+        H, dk, dv = heads, key_dim, value_dim
+        for sg in meta.segments:
+            r = slice(sg.row0, sg.row0 + sg.n)
+            x = proj[r].double()
+            q = x[:, :H * dk].reshape(-1, H, dk) * query_scale
+            k = x[:, H * dk: 2 * H * dk].reshape(-1, H, dk)
+            v = x[:, 2 * H * dk: 2 * H * dk + H * dv].reshape(-1, H, dv)
+            a = torch.exp(torch.nn.functional.logsigmoid(decay_in[r].double()) / decay_root).reshape(-1, H, dk)
+            S = state[sg.state_slot].double()
+            for t in range(sg.n):
+                S = a[t][:, :, None] * S + k[t][:, :, None] * v[t][:, None, :]
+                out[sg.row0 + t] = torch.einsum("hkv,hk->hv", S, q[t]).reshape(-1).float()
+            state[sg.state_slot] = S.float()
+
+    def check_differential_attention(self, num_heads, num_kv_heads, map_dim, value_dim) -> None:
+        if num_heads % num_kv_heads:
+            raise ValueError("bad head counts")
+
+    def differential_attention(self, q, cache, meta, out, num_heads, num_kv_heads, map_dim, value_dim, scale, lam, eps, mult) -> None:
+        H, G, d, dv = num_heads, num_kv_heads, map_dim, value_dim
+        pos, row = meta.pos.long(), meta.seq_row.long()
+        table, bs = meta.table(cache.group), cache.page_size
+        out.zero_()
+        for i in range(q.shape[0]):
+            if row[i] < 0:
+                continue
+            js = torch.arange(int(pos[i]) + 1)
+            pages = table[row[i], js // bs].long()
+            assert (pages >= 0).all(), "a visible key has no page"
+            K = cache.keys[pages, :, js % bs].float().view(-1, G, 2, d)
+            V = cache.values[pages, :, js % bs].float()
+            s = torch.einsum("gamd,jgmd->gamj", q[i].float().view(G, H // G, 2, d), K) * scale
+            a = torch.einsum("gamj,jgv->gamv", torch.softmax(s, -1), V).reshape(H, 2, dv)
+            o = a[:, 0] - lam.float() * a[:, 1]
+            out[i] = (o * torch.rsqrt((o * o).mean(-1, keepdim=True) + eps) * mult).reshape(-1).to(out.dtype)
+
+    def grouped_linear_act(self, h, w, route, y, activation) -> None:
+        assert activation == "relu2"
+        order, live = route
+        n, top = order.shape
+        for i in range(n):
+            for k in range(top):
+                e = int(order[i, k])
+                if live[i] and e < w.shape[0]:
+                    y[i * top + k] = (torch.relu(h[i].float() @ w[e].float().T) ** 2).to(y.dtype)
+
+    def grouped_linear_scatter(self, y, w, route, out) -> None:
+        order, live = route
+        n, top = order.shape
+        out.fill_(float("nan"))      # rows without a product must not be read
+        for i in range(n):
+            for k in range(top):
+                e = int(order[i, k])
+                if not live[i]:
+                    out[i * top + k] = 0
+                elif e < w.shape[0]:
+                    out[i * top + k] = y[i * top + k].float() @ w[e].float().T
+
+    def route_by_scores(self, logits, num_experts, top, groups, keep_groups, renormalize, meta, weights, align=1,
+                        scoring="softmax", correction=None, group_top=1, sum_eps=0.0, scale=1.0, identity=0):
+        return super().route_by_scores(logits, num_experts, top, groups, keep_groups, renormalize, meta, weights, align, scoring,
+                                       correction, group_top, sum_eps, scale)
+
+    def moe_combine(self, terms, weights, shared, gate_logits, gate_column, out, add=None, scale=1.0, handed_on=None) -> None:
+        if handed_on is None:
+            return super().moe_combine(terms, weights, shared, gate_logits, gate_column, out, add, scale)
+        (order, live), first, h = handed_on
+        n, top = weights.shape
+        t = torch.where((order >= first)[:, :, None], h.float()[:, None, :], terms.view(n, top, -1))
+        super().moe_combine(t.reshape(n * top, -1), weights, shared, gate_logits, gate_column, out, add, scale)
