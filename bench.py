@@ -1,7 +1,7 @@
 """Benchmark: decode tokens per second of the Llama-3.1-8B-sized model (random bf16 weights) on one B200.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--batch 8] [--context 4096] [--layers L] [--impl ours|reference]
-                    [--preset NAME] [--workload decode|stream|pepilix|gizulorn|nepudra|gimotar|gimupel]
+                    [--preset NAME] [--workload decode|stream|pepilix|gizulorn|nepudra|gimotar|gimupel|muretar]
 
 A "step" is one decode step of `--batch` requests whose contexts end at `--context` tokens. Prints ONE JSON line:
   value      decoded tokens per second, timed on the device (CUDA events around K steps: metadata copy + graph replay)
@@ -166,7 +166,8 @@ def main() -> int:
     ap.add_argument("--no-points", action="store_true", help="skip the batch 1 and 64 points")
     ap.add_argument("--no-e2e", action="store_true")
     ap.add_argument("--reference-device", default="CUDA", help="the reference's device name for --impl reference")
-    ap.add_argument("--workload", default="decode", choices=["decode", "stream", "pepilix", "gizulorn", "nepudra", "gimotar", "gimupel"],
+    ap.add_argument("--workload", default="decode", choices=["decode", "stream", "pepilix", "gizulorn", "nepudra", "gimotar", "gimupel",
+                                                                    "muretar"],
                     help="pepilix: prefill and decode of the Pepilix design at a few layer sizes, beside the dense decoder "
                          "at equal width, layers, heads and active feed-forward size")
     ap.add_argument("--sizes", default="w1024,w2048", help="pepilix workload: which of its sizes to run")
@@ -204,6 +205,8 @@ def main() -> int:
         return design_workload(a, "gimotar")
     if a.workload == "gimupel":
         return design_workload(a, "gimupel")
+    if a.workload == "muretar":
+        return design_workload(a, "muretar")
 
     import numpy as np
     import torch
@@ -554,6 +557,34 @@ def gimupel_configs(name: str, L: int, ctx: int):
     return gip, giz
 
 
+# Layer sizes for the Muretar workload: (width, heads, kv heads and size of one map of the differential attention, heads, kv heads
+# and head size of the attention beside the delta rule, heads, key heads, key and value size of the delta rule, heads, key and
+# value size of the gated linear attention, experts, experts that hand the input on, top, expert ff, shared ff, vocab). Layers
+# cycle through gated linear attention, parallel, differential attention, gated linear attention; every layer has routed
+# experts and a shared expert. Gizulorn beside it (`GIZULORN_SIZES` of the same width) has the same width, layers, heads, head
+# sizes, state sizes, experts, expert and shared sizes and vocabulary: each of Muretar's kernels has a like kernel there (the
+# attention has no window here, and a window there).
+MURETAR_SIZES = {
+    "r1024": (1024, 8, 2, 32, 8, 2, 64, 8, 4, 64, 128, 8, 64, 128, 16, 2, 2, 512, 512, 32768),
+    "r2048": (2048, 16, 4, 64, 16, 4, 128, 16, 8, 128, 128, 16, 128, 128, 32, 4, 4, 512, 1024, 32768),
+}
+
+
+def muretar_configs(name: str, L: int, ctx: int):
+    D, Hd, kvd, map_dim, H, kv, hd, Hr, kr, dk, dv, Hg, gk, gv, E, ident, top, ff, shared, V = MURETAR_SIZES[name]
+    mlp = {"kind": "moe", "router": {"experts": E, "identity": ident, "top": top}, "expert": {"ff": ff}, "shared": {"ff": shared}}
+    par = {"left": {"heads": H, "kv_heads": kv, "dim": hd, "vdim": hd, "scale": hd ** -0.5,
+                    "rot": {"base": 5e5, "dims": hd, "scaling": {"factor": 8.0}}},
+           "right": {"heads": Hr, "kv_heads": kr, "dim": dk, "vdim": dv, "conv": 4}}
+    gla = {"heads": Hg, "dim": gk, "vdim": gv, "tau": 16.0}
+    att = {"heads": Hd, "kv_heads": kvd, "dim": map_dim, "vdim": 2 * map_dim, "scale": map_dim ** -0.5, "diff": 0.5}
+    kinds = [("gla", gla), ("parallel", par), ("attention", att), ("gla", gla)]
+    mur = {"architecture": "Muretar", "vocab": V, "width": D, "norm": {"eps": 1e-6},
+           "layers": [{"type": kinds[i % 4][0], "mixer": kinds[i % 4][1], "mlp": mlp} for i in range(L)]}
+    giz, _ = gizulorn_configs("g" + name[1:], L, ctx)
+    return mur, giz
+
+
 def pepilix_workload(a) -> int:
     return design_workload(a, "pepilix")
 
@@ -575,8 +606,8 @@ def design_workload(a, design: str) -> int:
     rng = np.random.default_rng(5)
 
     SIZES = {"pepilix": PEPILIX_SIZES, "gizulorn": GIZULORN_SIZES, "nepudra": NEPUDRA_SIZES, "gimotar": GIMOTAR_SIZES,
-             "gimupel": GIMUPEL_SIZES}[design]
-    twin = "gizulorn" if design in ("nepudra", "gimotar", "gimupel") else "dense"        # the model timed beside the design
+             "gimupel": GIMUPEL_SIZES, "muretar": MURETAR_SIZES}[design]
+    twin = "gizulorn" if design in ("nepudra", "gimotar", "gimupel", "muretar") else "dense"        # the model timed beside the design
 
     def configs(name):
         if design == "gizulorn":
@@ -587,6 +618,8 @@ def design_workload(a, design: str) -> int:
             return gimotar_configs(name, L, ctx)
         if design == "gimupel":
             return gimupel_configs(name, L, ctx)
+        if design == "muretar":
+            return muretar_configs(name, L, ctx)
         D, H, dn, dr, dv, r, E, top, ff, V = PEPILIX_SIZES[name]
         mixer = {"heads": H, "dim": dn, "rot_dim": dr, "vdim": dv, "kv_rank": r, "scale": (dn + dr) ** -0.5,
                  "rot": {"base": 10000.0, "dims": dr}}
@@ -694,6 +727,10 @@ def design_workload(a, design: str) -> int:
                                          ("width", "ssm_heads", "ssm_vdim", "state", "groups", "norm_groups", "heads", "kv_heads", "head_dim",
                                           "window", "experts", "top", "expert_groups", "keep", "ff", "dense_ff", "vocab")
                                          if design == "gimupel" else
+                                         ("width", "diff_heads", "diff_kv_heads", "map_dim", "heads", "kv_heads", "head_dim", "delta_heads",
+                                          "delta_key_heads", "delta_dim", "delta_vdim", "gla_heads", "gla_dim", "gla_vdim", "experts",
+                                          "identity", "top", "ff", "shared_ff", "vocab")
+                                         if design == "muretar" else
                                          ("width", "heads", "dim", "vdim", "kv_heads", "window", "key_heads", "experts", "top", "groups",
                                           "keep", "ff", "shared_ff", "vocab"), SIZES[n])) for n in sizes},
                    "beside": twin,

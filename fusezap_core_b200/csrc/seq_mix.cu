@@ -655,18 +655,18 @@ __device__ __forceinline__ float decay_of(float a, float rate) {
 }
 // S = g * S (rows); u = beta (v - S^T k^); S += k^ u^T; o = S^T q^. qkv rows: [q (Hk dk) | k (Hk dk) | v (H dv)] of T.
 // HEAD: one decay per head (high holds one input per head), else one per head and key channel. high and beta point at
-// their first column; their rows are ldh and ldb floats long.
+// their first column; their rows are ldh and ldb floats long. Portions of more than max_rows rows are left to another kernel.
 template <typename T, int R, bool HEAD>
 __global__ void __launch_bounds__(SCAN_MAX_THREADS)
 gated_delta_scan_kernel(const T* __restrict__ qkv, int H, int Hk, int dk, int dv, int tch,
                         const float* __restrict__ high, int ldh, const float* __restrict__ beta, int ldb,
                         const float* __restrict__ a_log, const float* __restrict__ dt_bias, float unit_eps, float q_scale,
-                        float* __restrict__ state, const int* __restrict__ seg, float* __restrict__ out) {
+                        float* __restrict__ state, const int* __restrict__ seg, int max_rows, float* __restrict__ out) {
   fz_grid_launch_dependents();
   const int s = blockIdx.x, h = blockIdx.y;
   const int row0 = seg[4 * s], cnt = seg[4 * s + 1], slot = seg[4 * s + 3];
   fz_grid_wait();
-  if (cnt <= 0 || slot < 0) return;
+  if (cnt <= 0 || cnt > max_rows || slot < 0) return;
   extern __shared__ __align__(16) float smem[];
   const int NT = blockDim.x;
   const int dkp = R * DPT, COLS = NT / R * DC;
@@ -1566,7 +1566,7 @@ FZ_API int fz_retention_scan(const float* proj, int ld, int H, int dk, int dv, c
 template <typename T, int R, bool HEAD>
 static int launch_delta(const void* qkv, int H, int Hk, int dk, int dv, const float* high, int ldh, const float* beta, int ldb,
                         const float* a_log, const float* dt_bias, float unit_eps, float q_scale, float* state, const int* seg,
-                        int n_seg, float* out, cudaStream_t stream) {
+                        int n_seg, int max_rows, float* out, cudaStream_t stream) {
   const int threads = scan_threads(dv, R), cols = threads / R * DC;
   const int tch = delta_smem(dk, R, cols, 16, sizeof(T), HEAD) <= 48 * 1024 ? 16 : 8;
   const size_t smem = delta_smem(dk, R, cols, tch, sizeof(T), HEAD);
@@ -1574,7 +1574,7 @@ static int launch_delta(const void* qkv, int H, int Hk, int dk, int dv, const fl
   int st = allow_smem(gated_delta_scan_kernel<T, R, HEAD>, smem, allowed);
   if (st != FZ_OK) return st;
   fz_launch(gated_delta_scan_kernel<T, R, HEAD>, dim3(n_seg, H, (dv + cols - 1) / cols), dim3(threads), smem, stream, (const T*)qkv,
-            H, Hk, dk, dv, tch, high, ldh, beta, ldb, a_log, dt_bias, unit_eps, q_scale, state, seg, out);
+            H, Hk, dk, dv, tch, high, ldh, beta, ldb, a_log, dt_bias, unit_eps, q_scale, state, seg, max_rows, out);
   FZ_LAUNCH_CHECK();
   return FZ_OK;
 }
@@ -1582,10 +1582,11 @@ static int launch_delta(const void* qkv, int H, int Hk, int dk, int dv, const fl
 // high: the first decay input of row 0 (head_decay: one per head, else H dk of them), rows ldh floats apart; beta likewise.
 FZ_API int fz_gated_delta_scan(const void* qkv, int dtype, int H, int Hk, int dk, int dv, const float* high, int ldh,
                                const float* beta, int ldb, const float* a_log, const float* dt_bias, float unit_eps, float q_scale,
-                               int head_decay, float* state, const int* seg, int n_seg, float* out, cudaStream_t stream) {
+                               int head_decay, float* state, const int* seg, int n_seg, int max_rows, float* out,
+                               cudaStream_t stream) {
   if (n_seg <= 0) return FZ_OK;
   if (H <= 0 || H > 65535 || Hk <= 0 || H % Hk || dv <= 0 || fz_recurrent_key_pad(dk) < 0) return FZ_BAD_SHAPE;
-#define FZ_ARGS qkv, H, Hk, dk, dv, high, ldh, beta, ldb, a_log, dt_bias, unit_eps, q_scale, state, seg, n_seg, out, stream
+#define FZ_ARGS qkv, H, Hk, dk, dv, high, ldh, beta, ldb, a_log, dt_bias, unit_eps, q_scale, state, seg, n_seg, max_rows, out, stream
 #define FZ_CALL_F(R) (head_decay ? launch_delta<float, R, true>(FZ_ARGS) : launch_delta<float, R, false>(FZ_ARGS))
 #define FZ_CALL_B(R) (head_decay ? launch_delta<__nv_bfloat16, R, true>(FZ_ARGS) : launch_delta<__nv_bfloat16, R, false>(FZ_ARGS))
   if (dtype == FZ_F32) { FZ_BY_LANES(lanes_per_column(dk), FZ_CALL_F) }

@@ -35,6 +35,8 @@ LIBRARIES: dict[str, list[str]] = {
     "fzb200_ssd_tc": ["ssd_chunk.cu"],                                       # bfloat16 only: long portions of that scan on tensor cores
     # the scan of gated linear attention, token by token (both dtypes)
     "fzb200_gla": ["gla.cu"],
+    # bfloat16 only: long portions of that scan and of the delta rule with one decay per head on tensor cores
+    "fzb200_scan_tc": ["scan_chunk.cu"],
     # depth-averaged layers, the hashed pair embedding, a columnwise activation (both dtypes)
     "fzb200_rows": ["stream_rows.cu"],
     "fzb200_seq_tc": ["attn_sink_mma.cu"],                                   # bfloat16 only: that attention on tensor cores

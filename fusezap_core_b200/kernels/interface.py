@@ -177,6 +177,10 @@ class Ops:
         S = g * S (rows), u = b * (v - S^T k^), S = S + k^ u^T, out[n, h] = S^T q^. float32 throughout; out (N, H dv)."""
         raise NotImplementedError
 
+    def check_chunked_scan(self, heads: int, key_dim: int, value_dim: int) -> None:
+        """Builds and loads, with the model and not at its first step, what `channel_decay_scan` or `gated_delta_scan` with
+        head_decay need for long portions of these sizes."""
+
     def channel_decay_scan(self, proj: torch.Tensor, heads: int, key_dim: int, value_dim: int, decay_in: torch.Tensor,
                            decay_root: float, query_scale: float, state: torch.Tensor, meta: Any, out: torch.Tensor) -> None:
         """proj: (N, >= H (2 dk + dv)) float32, a row = [q heads | k heads | v heads | ...]; decay_in (N, H dk) float32. Per

@@ -29,6 +29,7 @@ RGLRU_COOK_ROWS = 4  # recurrent unit: steps whose longest portion is longer com
 SSD_CHUNK_ROWS = 16     # state space scan (bfloat16): portions of this many rows and more go to the tensor-core kernel where the sizes allow it
 SSD_SPREAD_ROWS = 16    # state space scan: in steps whose longest portion has this many rows a head's columns are spread over blocks of
 SSD_SPREAD_THREADS = 64  # this many threads (few blocks otherwise); shorter portions take blocks of up to 512 threads
+SCAN_CHUNK_ROWS = 16  # linear attention and the delta rule with one decay per head (bfloat16): portions of this many rows (16 at least) and more go to the tensor-core kernels
 SINK_MMA_ROWS = 16  # windowed attention with a sink: steps whose longest portion has this many rows go to the tensor-core kernel
 LONG_PORTION = 8    # attention: portions of at least this many tokens go to the tile (prefill) kernels
 TILE_ROWS = 128     # token rows per tile of those kernels
@@ -126,7 +127,7 @@ class CudaOps(Ops):
         if self.dtype == torch.bfloat16:
             self.tc = load("fzb200_tc")      # tcgen05 / TMA kernels
         self.use_tensor_cores = self.tc is not None
-        self._attn_tc = self._mix = self._mix_tc = self._latent = self._latent_tc = self._seq = self._seq_tc = self._rows = self._ssd = self._ssd_tc = self._gla = None   # libraries loaded (and built) when a part first asks for their kernels
+        self._attn_tc = self._mix = self._mix_tc = self._latent = self._latent_tc = self._seq = self._seq_tc = self._rows = self._ssd = self._ssd_tc = self._gla = self._scan_tc = None   # libraries loaded (and built) when a part first asks for their kernels
         self.prefill_tcgen05 = True        # False: long portions on the mma.sync flash-attention kernel
         self.fuse_swiglu = True            # gate/up product and SwiGLU in one kernel where the sizes allow it
         self.fuse_argmax = True            # lm_head product and argmax in one pass where no logits are asked for
@@ -142,6 +143,7 @@ class CudaOps(Ops):
         self.cut_prefill_keys = True       # few query tiles with many keys behind them are cut along the keys
         self._profile = None               # a StepProfile while the engine profiles its steps
         self._meta_rows = None             # meta.seq_row of the step being run, for ops that take no `meta`
+        self.scan_tensor_cores = True      # linear attention and delta-rule scans of long portions on tensor cores (bfloat16)
         self.ssd_tensor_cores = True       # state space scan of long portions on tensor cores (bfloat16)
         self.split_decode_keys = True      # windowed attention with a sink: steps of single tokens cut a row's keys into runs
         self.sink_tensor_cores = True      # that attention on tensor cores for portions of SINK_MMA_ROWS rows and more (bfloat16)
@@ -213,6 +215,13 @@ class CudaOps(Ops):
         if self._gla is None:
             self._gla = load("fzb200_gla")
         return self._gla
+
+    @property
+    def scan_tc(self):
+        """That scan, and the delta rule's with one decay per head, for long portions on tensor cores (bfloat16)."""
+        if self._scan_tc is None:
+            self._scan_tc = load("fzb200_scan_tc")
+        return self._scan_tc
 
     @property
     def ssd_tc(self):
@@ -997,6 +1006,19 @@ class CudaOps(Ops):
         if self._ssd_chunked(None, heads, groups, state_dim, value_dim):
             self.ssd_tc
 
+    def check_chunked_scan(self, heads: int, key_dim: int, value_dim: int) -> None:
+        self._scan_chunked(heads, key_dim, value_dim)
+
+    def _scan_chunked(self, heads: int, key_dim: int, value_dim: int) -> bool:
+        return bool(self.use_tensor_cores and self.scan_tensor_cores and self.dtype == torch.bfloat16 and
+                    self.scan_tc.fz_scan_chunk_check(c_int(heads), c_int(key_dim), c_int(value_dim)) == 0)
+
+    def _chunk_scratch(self, n: int, heads: int, key_dim: int, value_dim: int, delta: bool) -> torch.Tensor:
+        """Where the first of the two kernels leaves a chunk's operands for the second."""
+        self.scan_tc.fz_scan_chunk_scratch.restype = c_longlong
+        size = self.scan_tc.fz_scan_chunk_scratch(c_int(n), c_int(heads), c_int(key_dim), c_int(value_dim), c_int(1 if delta else 0))
+        return self._scratch("scan operands", int(size), torch.uint8)
+
     def _ssd_chunked(self, xbc, heads: int, groups: int, state_dim: int, value_dim: int) -> bool:
         return bool(self.use_tensor_cores and self.ssd_tensor_cores and self.dtype == torch.bfloat16 and state_dim % 16 == 0 and
                     value_dim % 16 == 0 and self.ssd_tc.fz_ssd_chunk_check(_p(xbc), c_int(heads), c_int(groups), c_int(state_dim), c_int(value_dim)) == 0)
@@ -1050,13 +1072,27 @@ class CudaOps(Ops):
                               f"out {tuple(out.shape)}")
         self._state(state, heads, key_dim, value_dim, "gated_delta_scan")
         self._meta_rows = meta.seq_row
+        nbytes = n * (qkv.shape[1] * qkv.element_size() + (decays + heads * (value_dim + 1)) * 4) \
+            + 2 * meta.n_segments * heads * value_dim * state.shape[3] * 4
+        inputs = (c_void_p(high.data_ptr() + 4 * high_offset), c_int(high.shape[1]), c_void_p(beta.data_ptr() + 4 * beta_offset),
+                  c_int(beta.shape[1]), _p(a_log), _p(dt_bias), c_float(unit_eps), c_float(query_scale))
+        max_portion = max(1, int(getattr(meta, "max_portion", 0)) or n)
+        max_rows = 2 ** 31 - 1
+        if head_decay and max_portion >= SCAN_CHUNK_ROWS and self._scan_chunked(heads, key_dim, value_dim):
+            # long portions 16 tokens at a time on tensor cores, the step's short ones (if it can have any) token by token
+            scratch = self._chunk_scratch(n, heads, key_dim, value_dim, True)
+            self._check(self.scan_tc.fz_delta_chunk(
+                _p(qkv), c_int(heads), c_int(key_heads), c_int(key_dim), c_int(value_dim), *inputs, _p(state), _p(meta.seg),
+                c_int(meta.max_segments), c_int(SCAN_CHUNK_ROWS), c_int(max_portion), _p(scratch), _p(out), self._stream()),
+                "gated_delta_scan (tensor cores)", nbytes)
+            self.launches += 1
+            if max_portion == n:
+                return
+            max_rows, nbytes = SCAN_CHUNK_ROWS - 1, 0
         self._check(self.seq.fz_gated_delta_scan(
-            _p(qkv), c_int(_CODE[self.dtype]), c_int(heads), c_int(key_heads), c_int(key_dim), c_int(value_dim),
-            c_void_p(high.data_ptr() + 4 * high_offset), c_int(high.shape[1]), c_void_p(beta.data_ptr() + 4 * beta_offset),
-            c_int(beta.shape[1]), _p(a_log), _p(dt_bias), c_float(unit_eps), c_float(query_scale), c_int(1 if head_decay else 0),
-            _p(state), _p(meta.seg), c_int(meta.max_segments), _p(out), self._stream()), "gated_delta_scan",
-            n * (qkv.shape[1] * qkv.element_size() + (decays + heads * (value_dim + 1)) * 4)
-            + 2 * meta.n_segments * heads * value_dim * state.shape[3] * 4)
+            _p(qkv), c_int(_CODE[self.dtype]), c_int(heads), c_int(key_heads), c_int(key_dim), c_int(value_dim), *inputs,
+            c_int(1 if head_decay else 0), _p(state), _p(meta.seg), c_int(meta.max_segments), c_int(max_rows), _p(out), self._stream()),
+            "gated_delta_scan", nbytes)
 
     def channel_decay_scan(self, proj, heads, key_dim, value_dim, decay_in, decay_root, query_scale, state, meta, out) -> None:
         self._want(proj, "linear attention projections", (torch.float32,), 2)
@@ -1068,11 +1104,21 @@ class CudaOps(Ops):
             raise KernelError(f"channel_decay_scan: proj {tuple(proj.shape)}, decay inputs {tuple(decay_in.shape)}, out {tuple(out.shape)}")
         self._state(state, heads, key_dim, value_dim, "channel_decay_scan")
         self._meta_rows = meta.seq_row
-        self._check(self.gla.fz_channel_decay_scan(
-            _p(proj), c_int(ld), c_int(heads), c_int(key_dim), c_int(value_dim), _p(decay_in), c_float(1.0 / decay_root),
-            c_float(query_scale), _p(state), _p(meta.seg), c_int(getattr(meta, "max_segments", meta.n_segments)), c_int(2 ** 31 - 1),
-            _p(out), self._stream()), "channel_decay_scan",
-            n * heads * (3 * key_dim + 2 * value_dim) * 4 + 2 * meta.n_segments * heads * value_dim * state.shape[3] * 4)
+        nbytes = n * heads * (3 * key_dim + 2 * value_dim) * 4 + 2 * meta.n_segments * heads * value_dim * state.shape[3] * 4
+        inputs = (_p(proj), c_int(ld), c_int(heads), c_int(key_dim), c_int(value_dim), _p(decay_in), c_float(1.0 / decay_root),
+                  c_float(query_scale), _p(state), _p(meta.seg), c_int(meta.max_segments))
+        max_portion = max(1, int(getattr(meta, "max_portion", 0)) or n)
+        max_rows = 2 ** 31 - 1
+        if max_portion >= SCAN_CHUNK_ROWS and self._scan_chunked(heads, key_dim, value_dim):
+            # long portions 16 tokens at a time on tensor cores, the step's short ones (if it can have any) token by token
+            scratch = self._chunk_scratch(n, heads, key_dim, value_dim, False)
+            self._check(self.scan_tc.fz_gla_chunk(*inputs, c_int(SCAN_CHUNK_ROWS), c_int(max_portion), _p(scratch), _p(out), self._stream()),
+                        "channel_decay_scan (tensor cores)", nbytes)
+            self.launches += 1
+            if max_portion == n:
+                return
+            max_rows, nbytes = SCAN_CHUNK_ROWS - 1, 0
+        self._check(self.gla.fz_channel_decay_scan(*inputs, c_int(max_rows), _p(out), self._stream()), "channel_decay_scan", nbytes)
 
     def ssd_scan(self, xbc, heads, groups, state_dim, value_dim, dt, dt_offset, dt_bias, a_log, skip, state, meta, out) -> None:
         self._want(xbc, "x, B and C", (self.dtype,), 2)

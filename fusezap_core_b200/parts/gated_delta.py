@@ -91,6 +91,8 @@ class GatedDelta(Mixer):
         self.norm_w = tensors[n["norm"]].float().contiguous()
         self.wo = tensors[n["out"]]
         self.state_shape = ops.recurrent_state_shape(H, dk, dv)
+        if self.head_decay:
+            ops.check_chunked_scan(H, dk, dv)
 
     def _bind_two_steps(self, tensors) -> None:
         n, H, dk, dv = self.names, self.H, self.dk, self.dv
@@ -113,6 +115,10 @@ class GatedDelta(Mixer):
 
     def state_need(self) -> dict:
         return {"S": self.state_shape, **self.conv.state_need()}
+
+    def step_needs(self) -> tuple[str, ...]:
+        # with one decay per head, which scan runs depends on the longest portion, which is then part of a step's shape
+        return ("portions",) if self.head_decay else ()
 
     def forward(self, ctx, h: torch.Tensor, cache: LayerCache) -> torch.Tensor:
         n, ops, ws = h.shape[0], ctx.ops, ctx.ws

@@ -60,6 +60,7 @@ class GatedLinearAttention(Mixer):
         self.norm_w = tensors[n["norm"]].float().contiguous()
         self.wo = tensors[n["out"]]
         self.state_shape = ops.recurrent_state_shape(H, dk, dv)
+        ops.check_chunked_scan(H, dk, dv)
 
     def state_need(self) -> dict:
         return {"S": self.state_shape}

@@ -814,6 +814,9 @@ class PlainOpsSandwich(PlainOpsSpace):
         super().gated_delta_scan(qkv, heads, key_heads, key_dim, value_dim, a.contiguous(), beta[:, beta_offset: beta_offset + H].contiguous(),
                                  a_log, dt_bias, unit_eps, query_scale, state, meta, out)
 
+    def check_chunked_scan(self, heads, key_dim, value_dim) -> None:
+        pass
+
     def channel_decay_scan(self, proj, heads, key_dim, value_dim, decay_in, decay_root, query_scale, state, meta, out) -> None:
         H, dk, dv = heads, key_dim, value_dim
         for sg in meta.segments:
