@@ -9,6 +9,10 @@
 // kernel merges a row's pieces in rising order and normalises. Rows of portions with at least `long_from` tokens are
 // left to the prefill kernel.
 //
+// Two maps per head (maps = 2, differential attention): Hq counts maps, neighbouring pairs of which share a stored query row
+// of HD values [map 1 | map 2] and the head's values; a map scores its own half of the key, so its row of the tile is the stored
+// row with the other half zero. Results then go out as float32, (rows, Hq, HD), for the kernel that combines the maps.
+//
 // Two variants. `attn_decode_units_kernel` (page sizes 8, 16 and multiples of 16; see there): a persistent grid whose
 // warps each take an equal share of the step's 64-key units and fetch them with TMA tile loads through rings of their
 // own; this is what keeps HBM3e busy at small and large batches alike. `attn_decode_kernel` (any page size): grid
@@ -185,13 +189,17 @@ __device__ __forceinline__ void merge_and_store(float* scratch, const float (&o)
   }
 }
 
+// Whether dimension d of a stored query row belongs to row r of the tile (maps = 1: always).
+template <int HD>
+__device__ __forceinline__ bool own_half(int r, int d, int maps) { return maps == 1 || (d >= HD / 2) == (r & 1); }
+
 template <int HD>
 __global__ void __launch_bounds__(THREADS)
 attn_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ k_pool,
                    const __nv_bfloat16* __restrict__ v_pool, const int* __restrict__ pos,
                    const int* __restrict__ seq_row, const int* __restrict__ seg, const int* __restrict__ table, int mb,
                    long long page_stride, int page_size, float* __restrict__ part_o, float* __restrict__ part_ml,
-                   int Hq, int Hkv, float scale_log2, int window, int long_from) {
+                   int Hq, int Hkv, float scale_log2, int window, int long_from, int maps) {
   fz_grid_launch_dependents();
   fz_grid_wait();
   constexpr int KSTEPS = HD / 16;      // k-steps of Q K^T
@@ -221,10 +229,10 @@ attn_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __r
 
   // Q: G rows of HD, zero rows up to 16, swizzled
   {
-    const __nv_bfloat16* qrow = q + (size_t)n * Hq * HD + (size_t)kvh * G * HD;
+    const __nv_bfloat16* qrow = q + ((size_t)n * Hq + (size_t)kvh * G) / maps * HD;
     for (int e = tid; e < 16 * (HD / 8); e += THREADS) {
       const int r = e / (HD / 8), c = e - r * (HD / 8);
-      cp_async16(s_q + swz<HD>(r, c), qrow + (size_t)r * HD + c * 8, r < G);
+      cp_async16(s_q + swz<HD>(r, c), qrow + (size_t)(r / maps) * HD + c * 8, r < G && own_half<HD>(r, c * 8, maps));
     }
   }
   const int ntiles = (k_end - k_begin + TILE - 1) / TILE;
@@ -321,7 +329,7 @@ attn_decode_units_kernel(const __grid_constant__ CUtensorMap kv_map, const __nv_
                          const int* __restrict__ pos, const int* __restrict__ seq_row, const int* __restrict__ seg,
                          const int* __restrict__ table, int mb, int page_size, float* __restrict__ part_o,
                          float* __restrict__ part_ml, int N, int Hq, int Hkv, int NPU, float scale_log2, int window,
-                         int long_from, int single, int* err) {
+                         int long_from, int single, int maps, int* err) {
   // SMALLG (at most 8 query heads per kv head): the transposed products of `attend16_small`
   constexpr int KSTEPS = HD / 16, OB = SMALLG ? HD / 16 : HD / 8, QW = SMALLG ? 2 : 4, HALVES = HD / 64;
   constexpr int HALF_BYTES = 16 * 128;                 // one column half of a 16-key group
@@ -502,23 +510,26 @@ attn_decode_units_kernel(const __grid_constant__ CUtensorMap kv_map, const __nv_
     if (cc.n != q_n || cc.kvh != q_kvh) {
       // another row or kv head: its G query heads, read from global memory straight into the MMA fragments
       q_n = cc.n; q_kvh = cc.kvh;
-      const uint32_t* qw = (const uint32_t*)(q + ((size_t)q_n * Hq + (size_t)q_kvh * G) * HD);
+      const uint32_t* qw = (const uint32_t*)(q + ((size_t)q_n * Hq + (size_t)q_kvh * G) / maps * HD);
       const int r0 = lane >> 2, cw = lane & 3;
+      const int ra = r0 / maps * HD, rb = (r0 + 8) / maps * HD;      // the stored rows of tile rows r0 and r0 + 8
       if constexpr (SMALLG) {
         // B operand (Q^T): head lane / 4, dimensions 2 (lane % 4) + {0, 1} and + 8 of every 16; zero past the group
 #pragma unroll
         for (int ks = 0; ks < KSTEPS; ++ks) {
-          qf[ks][0] = r0 < G ? qw[(r0 * HD + 16 * ks) / 2 + cw] : 0u;
-          qf[ks][1] = r0 < G ? qw[(r0 * HD + 16 * ks + 8) / 2 + cw] : 0u;
+          const bool own = r0 < G && own_half<HD>(r0, 16 * ks, maps);
+          qf[ks][0] = own ? qw[(ra + 16 * ks) / 2 + cw] : 0u;
+          qf[ks][1] = own ? qw[(ra + 16 * ks + 8) / 2 + cw] : 0u;
         }
       } else {
         // A operand: lane l holds rows (heads) l / 4 and l / 4 + 8, columns 2 (l % 4) + {0, 1} and + 8 of every 16
 #pragma unroll
         for (int ks = 0; ks < KSTEPS; ++ks) {
-          qf[ks][0] = r0 < G ? qw[(r0 * HD + 16 * ks) / 2 + cw] : 0u;
-          qf[ks][1] = r0 + 8 < G ? qw[((r0 + 8) * HD + 16 * ks) / 2 + cw] : 0u;
-          qf[ks][2] = r0 < G ? qw[(r0 * HD + 16 * ks + 8) / 2 + cw] : 0u;
-          qf[ks][3] = r0 + 8 < G ? qw[((r0 + 8) * HD + 16 * ks + 8) / 2 + cw] : 0u;
+          const bool half = own_half<HD>(r0, 16 * ks, maps);      // (r0 and r0 + 8 are rows of the same map)
+          qf[ks][0] = half && r0 < G ? qw[(ra + 16 * ks) / 2 + cw] : 0u;
+          qf[ks][1] = half && r0 + 8 < G ? qw[(rb + 16 * ks) / 2 + cw] : 0u;
+          qf[ks][2] = half && r0 < G ? qw[(ra + 16 * ks + 8) / 2 + cw] : 0u;
+          qf[ks][3] = half && r0 + 8 < G ? qw[(rb + 16 * ks + 8) / 2 + cw] : 0u;
         }
       }
     }
@@ -634,7 +645,8 @@ attn_decode_units_kernel(const __grid_constant__ CUtensorMap kv_map, const __nv_
 __global__ void __launch_bounds__(256)
 attn_combine_units_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                           const int* __restrict__ pos, const int* __restrict__ seq_row, const int* __restrict__ seg,
-                          __nv_bfloat16* __restrict__ out, int Hq, int HD, int NPU, int window, int long_from) {
+                          __nv_bfloat16* __restrict__ out, float* __restrict__ out32, int Hq, int HD, int NPU, int window,
+                          int long_from) {
   extern __shared__ float2 s_ml[];             // [units of the row], then the groups' results
   fz_grid_launch_dependents();
   const int n = blockIdx.y, h = blockIdx.x, tid = threadIdx.x;
@@ -646,8 +658,10 @@ attn_combine_units_kernel(const float* __restrict__ part_o, const float* __restr
   const int p = pos[n];
   fz_grid_wait();
   __nv_bfloat16* orow = out + ((size_t)n * Hq + h) * HD;
+  float* orow32 = out32 + ((size_t)n * Hq + h) * HD;
   if (row < 0) {
-    if (grp == 0) *(uint2*)(orow + d4) = make_uint2(0u, 0u);
+    if (grp == 0 && out32 != nullptr) *(float4*)(orow32 + d4) = make_float4(0.f, 0.f, 0.f, 0.f);
+    else if (grp == 0) *(uint2*)(orow + d4) = make_uint2(0u, 0u);
     return;
   }
   if (skip) return;
@@ -724,6 +738,10 @@ attn_combine_units_kernel(const float* __restrict__ part_o, const float* __restr
     merge4(O, s_o[k * per_row + tid], fa, fb);
   }
   const float inv = 1.0f / L;
+  if (out32 != nullptr) {
+    *(float4*)(orow32 + d4) = make_float4(O.x * inv, O.y * inv, O.z * inv, O.w * inv);
+    return;
+  }
   const __nv_bfloat162 a = __floats2bfloat162_rn(O.x * inv, O.y * inv), c = __floats2bfloat162_rn(O.z * inv, O.w * inv);
   *(uint2*)(orow + d4) = make_uint2(*(const uint32_t*)&a, *(const uint32_t*)&c);
 }
@@ -731,14 +749,19 @@ attn_combine_units_kernel(const float* __restrict__ part_o, const float* __restr
 // One block per (token row, query head): merges the partitions in rising order, normalises, rounds to bf16.
 __global__ void attn_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                     const int* __restrict__ seq_row, const int* __restrict__ seg,
-                                    __nv_bfloat16* __restrict__ out, int Hq, int HD, int NP, int long_from) {
+                                    __nv_bfloat16* __restrict__ out, float* __restrict__ out32, int Hq, int HD, int NP,
+                                    int long_from) {
   fz_grid_launch_dependents();
   fz_grid_wait();
   const int n = blockIdx.y, h = blockIdx.x;
   __nv_bfloat16* orow = out + ((size_t)n * Hq + h) * HD;
+  float* orow32 = out32 + ((size_t)n * Hq + h) * HD;
   const int row = seq_row[n];
   if (row < 0) {
-    for (int d = threadIdx.x; d < HD; d += blockDim.x) orow[d] = __float2bfloat16_rn(0.f);
+    for (int d = threadIdx.x; d < HD; d += blockDim.x) {
+      if (out32 != nullptr) orow32[d] = 0.f;
+      else orow[d] = __float2bfloat16_rn(0.f);
+    }
     return;
   }
   if (seg[row * 4 + 1] >= long_from) return;
@@ -755,14 +778,15 @@ __global__ void attn_combine_kernel(const float* __restrict__ part_o, const floa
       const float f = exp2f(ml[2 * i] - M);
       if (f != 0.f) acc += po[(size_t)i * HD + d] * f;     // an empty partition's O was never written
     }
-    orow[d] = __float2bfloat16_rn(acc * inv);
+    if (out32 != nullptr) orow32[d] = acc * inv;
+    else orow[d] = __float2bfloat16_rn(acc * inv);
   }
 }
 
 template <int HD, int BOX, int NSTAGE, int MINB, bool SMALLG>
 int launch_units(const void* q, const void* k_pool, long long pool_rows, const int* pos, const int* seq_row, const int* seg,
                  const int* table, int mb, int page_size, void* out, float* part_o, float* part_ml, int N, int Hq, int Hkv,
-                 float scale, int window, int NPU, int long_from, int single, int* err, cudaStream_t stream) {
+                 float scale, int window, int NPU, int long_from, int single, int maps, float* out32, int* err, cudaStream_t stream) {
   CUtensorMap map;
   int st = fztma::get_map_bf16(k_pool, pool_rows, HD, BOX, &map);
   if (st != FZ_OK) return st;
@@ -788,7 +812,7 @@ int launch_units(const void* q, const void* k_pool, long long pool_rows, const i
   if (ctas > (long long)sms * MINB) ctas = (long long)sms * MINB;
   fz_launch(attn_decode_units_kernel<HD, BOX, NSTAGE, MINB, SMALLG>, dim3((unsigned)ctas), dim3(THREADS), smem, stream, map,
             (const __nv_bfloat16*)q, pos, seq_row, seg, table, mb, page_size, part_o, part_ml, N, Hq, Hkv, NPU,
-            scale * 1.4426950408889634f, window, long_from, single, err);
+            scale * 1.4426950408889634f, window, long_from, single, maps, err);
   FZ_LAUNCH_CHECK();
   dim3 cgrid(Hq, N);
   // shared memory: the row's (max, sum) pairs, then 256 float4 and up to 16 float2 of the chains' results
@@ -797,7 +821,7 @@ int launch_units(const void* q, const void* k_pool, long long pool_rows, const i
   // 3.161, batch 4 3.369 -> 3.348; at batch 8 (256 blocks) 3.780 -> 3.789 and at batch 64 1.3 % slower
   const int ct = (long long)N * Hq <= sms ? 256 : 128;
   fz_launch(attn_combine_units_kernel, cgrid, dim3(ct), (size_t)(NPU + 2) * 8 + 256 * 16 + 16 * 8, stream, (const float*)part_o,
-            (const float*)part_ml, pos, seq_row, seg, (__nv_bfloat16*)out, Hq, HD, NPU, window, long_from);
+            (const float*)part_ml, pos, seq_row, seg, (__nv_bfloat16*)out, out32, Hq, HD, NPU, window, long_from);
   FZ_LAUNCH_CHECK();
   return FZ_OK;
 }
@@ -814,8 +838,8 @@ inline int units_sms() {
 template <int HD, int BOX>
 int launch_tma(const void* q, const void* k_pool, long long pool_rows, const int* pos, const int* seq_row, const int* seg,
                const int* table, int mb, int page_size, void* out, float* part_o, float* part_ml, int N, int Hq, int Hkv,
-               float scale, int window, int NPU, int long_from, int single, int* err, cudaStream_t stream) {
-#define FZ_U(NS_, MB_, SG_) return launch_units<HD, BOX, NS_, MB_, SG_>(q, k_pool, pool_rows, pos, seq_row, seg, table, mb, page_size, out, part_o, part_ml, N, Hq, Hkv, scale, window, NPU, long_from, single, err, stream)
+               float scale, int window, int NPU, int long_from, int single, int maps, float* out32, int* err, cudaStream_t stream) {
+#define FZ_U(NS_, MB_, SG_) return launch_units<HD, BOX, NS_, MB_, SG_>(q, k_pool, pool_rows, pos, seq_row, seg, table, mb, page_size, out, part_o, part_ml, N, Hq, Hkv, scale, window, NPU, long_from, single, maps, out32, err, stream)
   // three stages of 16 keys per warp and two CTAs per SM (eight warps with 24 KB in flight each) measured best
   if (Hq / Hkv > 8) FZ_U(3, 2, false);
   // So few units that every warp of one CTA per SM gets at most one (a single row at 4,096 keys): four stages, so that
@@ -829,7 +853,7 @@ int launch_tma(const void* q, const void* k_pool, long long pool_rows, const int
 template <int HD>
 int launch(const void* q, const void* k_pool, const void* v_pool, const int* pos, const int* seq_row, const int* seg,
            const int* table, int mb, long long page_stride, int page_size, void* out, float* part_o, float* part_ml,
-           int N, int Hq, int Hkv, float scale, int window, int NP, int long_from, cudaStream_t stream) {
+           int N, int Hq, int Hkv, float scale, int window, int NP, int long_from, int maps, float* out32, cudaStream_t stream) {
   constexpr int TILE_BYTES = TILE * HD * 2;
   constexpr size_t smem_pipe = 2 * STAGES * TILE_BYTES + 16 * HD * 2;
   constexpr size_t smem_merge = (size_t)4 * 16 * (HD + 4) * 4 + 4 * 16 * 2 * 4;
@@ -843,11 +867,11 @@ int launch(const void* q, const void* k_pool, const void* v_pool, const int* pos
   dim3 grid(NP, Hkv, N);
   fz_launch(attn_decode_kernel<HD>, grid, dim3(THREADS), smem, stream, (const __nv_bfloat16*)q, (const __nv_bfloat16*)k_pool,
             (const __nv_bfloat16*)v_pool, pos, seq_row, seg, table, mb, page_stride, page_size, part_o, part_ml, Hq, Hkv,
-            scale * 1.4426950408889634f, window, long_from);
+            scale * 1.4426950408889634f, window, long_from, maps);
   FZ_LAUNCH_CHECK();
   dim3 cgrid(Hq, N);
   fz_launch(attn_combine_kernel, cgrid, dim3(HD < 128 ? 64 : 128), 0, stream, (const float*)part_o, (const float*)part_ml,
-            seq_row, seg, (__nv_bfloat16*)out, Hq, HD, NP, long_from);
+            seq_row, seg, (__nv_bfloat16*)out, out32, Hq, HD, NP, long_from);
   FZ_LAUNCH_CHECK();
   return FZ_OK;
 }
@@ -865,14 +889,18 @@ FZ_API int fz_attn_decode_check(int Hq, int Hkv, int hd) {
 FZ_API int fz_attn_partitions(int max_context) { return max_context <= 0 ? 1 : unit_of(max_context - 1) + 1; }
 
 // Float32 scratch the call needs: part_o N * Hq * NP * hd floats, part_ml N * Hq * NP * 2 floats.
+// maps 2: see the head of this file; out is not written, out32 (N * Hq * hd floats) is. maps 1: out32 null, or where the results
+// go as float32 instead of out.
 // single_tokens != 0: every portion of the step is one token (the caller knows; the kernel then reads no portion records).
 // num_pages > 0 and a pool laid out as (pages, 2, Hkv, page_size, hd) with v_pool = k_pool + Hkv * page_size * hd select
 // the TMA variant where the page size allows it (8, 16 or a multiple of 16); otherwise the cp.async variant runs.
 FZ_API int fz_attn_decode(const void* q, const void* k_pool, const void* v_pool, const int* pos, const int* seq_row,
                           const int* seg, const int* table, int mb, long long page_stride, int page_size, void* out,
                           float* part_o, float* part_ml, int N, int Hq, int Hkv, int hd, float scale, int window,
-                          int max_context, int long_from, int single_tokens, int num_pages, int* err, cudaStream_t stream) {
+                          int max_context, int long_from, int single_tokens, int num_pages, int maps, float* out32, int* err,
+                          cudaStream_t stream) {
   if (N <= 0) return FZ_OK;
+  if ((maps != 1 && maps != 2) || (maps == 2 && (out32 == nullptr || (Hq / Hkv) % 2))) return FZ_BAD_SHAPE;
   const int single = single_tokens ? 1 : 0;
   if (fz_attn_decode_check(Hq, Hkv, hd) != FZ_OK || page_size <= 0) return FZ_BAD_SHAPE;
   if (N > 65535 || Hkv > 65535) return FZ_TOO_LARGE;
@@ -885,7 +913,7 @@ FZ_API int fz_attn_decode(const void* q, const void* k_pool, const void* v_pool,
                       (long long)N * Hkv * NPU < (1LL << 30) && (size_t)NPU * 8 < 40 * 1024 && !getenv("FZB200_NO_TMA_ATTN");
   if (tma_ok) {
     const long long pool_rows = (long long)num_pages * 2 * Hkv * page_size;
-#define FZ_T(HD_, BOX_) return launch_tma<HD_, BOX_>(q, k_pool, pool_rows, pos, seq_row, seg, table, mb, page_size, out, part_o, part_ml, N, Hq, Hkv, scale, window, NPU, long_from, single, err, stream)
+#define FZ_T(HD_, BOX_) return launch_tma<HD_, BOX_>(q, k_pool, pool_rows, pos, seq_row, seg, table, mb, page_size, out, part_o, part_ml, N, Hq, Hkv, scale, window, NPU, long_from, single, maps, out32, err, stream)
     if (hd == 64 && page_size == 8) FZ_T(64, 8);
     if (hd == 64) FZ_T(64, 16);
     if (page_size == 8) FZ_T(128, 8);
@@ -893,8 +921,8 @@ FZ_API int fz_attn_decode(const void* q, const void* k_pool, const void* v_pool,
 #undef FZ_T
   }
   if (hd == 64)
-    return launch<64>(q, k_pool, v_pool, pos, seq_row, seg, table, mb, page_stride, page_size, out, part_o, part_ml, N, Hq, Hkv, scale, window, NP, long_from, stream);
-  return launch<128>(q, k_pool, v_pool, pos, seq_row, seg, table, mb, page_stride, page_size, out, part_o, part_ml, N, Hq, Hkv, scale, window, NP, long_from, stream);
+    return launch<64>(q, k_pool, v_pool, pos, seq_row, seg, table, mb, page_stride, page_size, out, part_o, part_ml, N, Hq, Hkv, scale, window, NP, long_from, maps, out32, stream);
+  return launch<128>(q, k_pool, v_pool, pos, seq_row, seg, table, mb, page_stride, page_size, out, part_o, part_ml, N, Hq, Hkv, scale, window, NP, long_from, maps, out32, stream);
 }
 
 #ifdef FZ_TIMELINE

@@ -215,6 +215,10 @@ class Ops:
         blocks of tokens, in another order of the same sums."""
         raise NotImplementedError
 
+    def paged_attention_sizes(self, num_heads: int, num_kv_heads: int, head_dim: int) -> bool:
+        """Whether `paged_attention` has kernels for these sizes that a mixer should prefer to the general ones."""
+        return False
+
     def check_differential_attention(self, num_heads: int, num_kv_heads: int, map_dim: int, value_dim: int) -> None:
         """Raise ValueError if `differential_attention` cannot take these sizes."""
         raise NotImplementedError

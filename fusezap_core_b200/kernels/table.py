@@ -641,7 +641,8 @@ class CudaOps(Ops):
                     _p(q), _p(k), _p(v), _p(meta.pos), _p(meta.seq_row), _p(meta.seg), _p(table), c_int(table.shape[1]),
                     c_longlong(page_stride), c_int(cache.page_size), _p(out), _p(part_o), _p(part_ml), c_int(n),
                     c_int(hq), c_int(hkv), c_int(hd), c_float(scale), c_int(window), c_int(meta.max_context),
-                    c_int(LONG_PORTION), c_int(1 if plan.single_tokens else 0), c_int(k.shape[0]), _p(self.err), self._stream()),
+                    c_int(LONG_PORTION), c_int(1 if plan.single_tokens else 0), c_int(k.shape[0]), c_int(1), c_void_p(0), _p(self.err),
+                    self._stream()),
                     "paged_attention (decode)", kv)
                 self.launches += 1    # the combine kernel
             if plan.n_tiles > 0 and self.prefill_tcgen05 and \
@@ -1202,10 +1203,18 @@ class CudaOps(Ops):
         if self._sink_mma_sizes(key_dim, value_dim, 1):
             self.seq_tc       # built and loaded with the model, not at its first step
 
+    def paged_attention_sizes(self, num_heads: int, num_kv_heads: int, head_dim: int) -> bool:
+        return bool(self.use_tensor_cores and self.attn_tc.fz_attn_decode_check(c_int(num_heads), c_int(num_kv_heads), c_int(head_dim)) == 0)
+
     def check_differential_attention(self, num_heads: int, num_kv_heads: int, map_dim: int, value_dim: int) -> None:
         self.check_sink_attention(2 * num_heads, num_kv_heads, 2 * map_dim, value_dim)
         if self._sink_mma_sizes(2 * map_dim, value_dim, 2):
             self.seq_tc
+        self._diff_decode(num_heads, num_kv_heads, map_dim, value_dim)
+
+    def _diff_decode(self, num_heads: int, num_kv_heads: int, map_dim: int, value_dim: int) -> bool:
+        """Whether single tokens go to the split-key kernel of the paged attention, a map as a query head of its own."""
+        return self.split_decode_keys and value_dim == 2 * map_dim and self.paged_attention_sizes(2 * num_heads, num_kv_heads, value_dim)
 
     def _sink_mma_sizes(self, key_dim: int, value_dim: int, maps: int) -> bool:
         """Whether the tensor-core kernel takes these sizes of a cached key (all maps of a head) and value, leaving
@@ -1294,8 +1303,28 @@ class CudaOps(Ops):
         if self._profile is not None:
             nbytes = sum(sg.pos0 + i + 1 for sg in meta.segments for i in range(sg.n)) * num_kv_heads * (2 * map_dim + value_dim) * k.element_size() \
                 + n * num_heads * (2 * map_dim + value_dim) * q.element_size()
+        one_token = max(1, int(getattr(meta, "max_portion", 0)) or n) == 1
+        if one_token and k.stride(2) == value_dim and self._diff_decode(num_heads, num_kv_heads, map_dim, value_dim):
+            k, v, page_stride = self._pool(cache, num_kv_heads, value_dim)
+            table, heads = meta.table(cache.group), 2 * num_heads
+            parts = self.attn_tc.fz_attn_partitions(c_int(meta.max_context))
+            part_o = self._scratch("attention partials", n * heads * parts * (value_dim + 2), torch.float32)
+            rows_out = self._scratch("attention maps", n * heads * value_dim, torch.float32)
+            self._check(self.attn_tc.fz_attn_decode(
+                _p(q), _p(k), _p(v), _p(meta.pos), _p(meta.seq_row), _p(meta.seg), _p(table), c_int(table.shape[1]),
+                c_longlong(page_stride), c_int(cache.page_size), c_void_p(0), _p(part_o), _p(part_o[n * heads * parts * value_dim:]), c_int(n),
+                c_int(heads), c_int(num_kv_heads), c_int(value_dim), c_float(scale), c_int(0), c_int(meta.max_context), c_int(LONG_PORTION),
+                c_int(1), c_int(k.shape[0]), c_int(2), _p(rows_out), _p(self.err), self._stream()), "differential_attention (decode)", nbytes)
+            self.launches += 1    # the kernel that merges the partial results
+            self._combine_maps(rows_out, n, num_heads, value_dim, lam, eps, mult, meta, out)
+            return
         self._sink_launch(q, k, v, cache, meta, out, num_heads, num_kv_heads, 2 * map_dim, value_dim, scale, 0, 0, None, 0.0,
                           (None, 0, 0), 0, nbytes, mix=(lam, eps, mult))
+
+    def _combine_maps(self, maps, n, num_heads, value_dim, lam, eps, mult, meta, out) -> None:
+        self._check(self.seq.fz_combine_maps(_p(maps), c_int(n), c_int(num_heads), c_int(value_dim), _p(lam), c_float(eps), c_float(mult),
+                                             _p(meta.seq_row), _p(out), c_int(_CODE[out.dtype]), self._stream()),
+                    "combine_maps", n * num_heads * value_dim * (8 + out.element_size()))
 
     def _sink_launch(self, q, k, v, cache, meta, out, num_heads, num_kv_heads, key_dim, value_dim, scale, window, keep_first, sink,
                      softcap, gate, span, nbytes, mix=None) -> None:
@@ -1345,9 +1374,7 @@ class CudaOps(Ops):
         if units:
             self.launches += 1      # the merge kernel
         if maps > 1:
-            self._check(self.seq.fz_combine_maps(_p(rows_out), c_int(n), c_int(num_heads), c_int(value_dim), _p(lam), c_float(mix_eps),
-                                                 c_float(mix_mult), _p(meta.seq_row), _p(out), c_int(_CODE[out.dtype]), self._stream()),
-                        "combine_maps", n * num_heads * value_dim * (8 + out.element_size()))
+            self._combine_maps(rows_out, n, num_heads, value_dim, lam, mix_eps, mix_mult, meta, out)
 
     def general_delta_scan(self, proj, heads, key_dim, value_dim, remove_offset, decay_in, decay_bias, remove_bias, decay_rate,
                            unit_eps, state, meta, out) -> None:

@@ -59,7 +59,8 @@ class DifferentialAttention(Mixer):
         ops.check_differential_attention(self.H, self.G, self.d, self.dv)
 
     def cache_need(self) -> KVNeed:
-        return KVNeed(self.G, 2 * self.d, 0, value_dim=self.dv)
+        # (keys and values of one size lie in halves of a page, as the paged attention's kernels want them)
+        return KVNeed(self.G, 2 * self.d, 0, value_dim=0 if self.dv == 2 * self.d else self.dv)
 
     def step_needs(self) -> tuple[str, ...]:
         return ("portions",)      # its kernels tile the rows of portions: the longest portion is part of a step's shape

@@ -76,6 +76,7 @@ class SinkAttention(Mixer):
         if value_mix not in (None, "source", "blend") or (value_mix and not own_kv):
             raise ValueError(f"value_mix {value_mix!r} is not one of None, 'source', 'blend', or the layer has no values of its own")
         self.value_mix, self.value_mix_key = value_mix, value_mix_key
+        self.paged = False
         self.wqkv = self.bqkv = self.wo = self.bo = self.sink = self.q_norm_w = self.k_norm_w = self.mix_w = None
 
     def tensors(self) -> dict[str, ParamSpec]:
@@ -125,15 +126,26 @@ class SinkAttention(Mixer):
         if self.value_mix == "blend":
             self.mix_w = tensors[n["value_mix"]].float().reshape(1).contiguous()
         ops.check_sink_attention(self.Hq, self.Hkv, self.dk, self.dv)
+        # attention over all earlier keys without any of the extras is what the paged attention's kernels compute, where
+        # this table has some for the sizes
+        self.paged = self.plain_causal() and ops.paged_attention_sizes(self.Hq, self.Hkv, self.dk)
+        if self.paged:
+            ops.check_attention(self.Hq, self.Hkv, self.dk)
+
+    def plain_causal(self) -> bool:
+        return not (self.window or self.keep_first or self.has_sink or self.softcap or self.head_gate or self.span) and \
+            self.own_kv and self.dk == self.dv and not self.cache_window
 
     def cache_need(self) -> KVNeed:
-        return KVNeed(self.Hkv, self.dk, self.cache_window, value_dim=self.dv,
+        return KVNeed(self.Hkv, self.dk, self.cache_window, value_dim=0 if self.paged else self.dv,
                       keep_first=self.keep_first if self.cache_window else 0)
 
     def position_name(self) -> str | None:
         return self.position
 
     def step_needs(self) -> tuple[str, ...]:
+        if self.paged:
+            return ("attention", "portions")
         return ("portions",)      # its kernels tile the rows of portions: the longest portion is part of a step's shape
 
     def forward(self, ctx, h: torch.Tensor, cache: LayerCache) -> torch.Tensor:
@@ -167,7 +179,9 @@ class SinkAttention(Mixer):
                                 ctx.meta, cache, q, Hq, Hkv, dk, dv, q_norm=self.q_norm_w, k_norm=self.k_norm_w,
                                 norm_eps=self.norm_eps, query_temperature=self.q_temp)
         o = ws.get("sink_out", (n, Hq * dv), ops.dtype)
-        if self.span:
+        if self.paged:
+            ops.paged_attention(q, cache, ctx.meta, o, Hq, Hkv, dk, self.scale, 0)
+        elif self.span:
             ops.sink_attention(q, cache, ctx.meta, o, Hq, Hkv, dk, dv, self.scale, self.window, self.keep_first, self.sink,
                                softcap=self.softcap, gate=(qkv, self.off_gate) if self.head_gate else None, span=self.span)
         elif self.softcap or self.head_gate:

@@ -266,6 +266,9 @@ class PlainOpsWide(PlainOps):
 class PlainOpsSeq(PlainOpsWide):
     """The operations of the recurrent mixers, the windowed attention with a sink and the routed experts."""
 
+    def paged_attention_sizes(self, num_heads, num_kv_heads, head_dim) -> bool:
+        return False
+
     def recurrent_state_shape(self, heads, key_dim, value_dim):
         return (heads, key_dim, value_dim)
 
