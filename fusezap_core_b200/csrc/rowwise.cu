@@ -430,8 +430,14 @@ static int launch_layernorm(float* x, const float* delta, const float* extra, co
     if (p.w != nullptr) fz_launch(add_layernorm_vec_kernel<TH, NT, V, true>, dim3(n_out), dim3(NT), 0, stream, x, delta, extra, w, b, (TH*)h, rows, n_src, D, eps, p, err); \
     else fz_launch(add_layernorm_vec_kernel<TH, NT, V, false>, dim3(n_out), dim3(NT), 0, stream, x, delta, extra, w, b, (TH*)h, rows, n_src, D, eps, p, err); \
   } while (0)
+  // (a post norm has four sums over the block: with many rows, blocks of four warps with more values per thread wait less for
+  // one another; bfloat16 only, since the order of a sum follows from the shape of the block)
+  const bool narrow = p.w != nullptr && sizeof(TH) == 2 && n_out >= 256;
   if (!vec) fz_launch(add_layernorm_kernel<TH>, dim3(n_out), dim3(256), 0, stream, x, delta, extra, w, b, (TH*)h, rows, n_src, D, eps, p, err);
   else if (D <= 4 * 128) FZ_LN(128, 1);
+  else if (narrow && D <= 4 * 256) FZ_LN(128, 2);
+  else if (narrow && D <= 4 * 512) FZ_LN(128, 4);
+  else if (narrow && D <= 8 * 512) FZ_LN(256, 4);
   else if (D <= 4 * 256) FZ_LN(256, 1);
   else if (D <= 4 * 512) FZ_LN(512, 1);
   else if (D <= 8 * 512) FZ_LN(512, 2);

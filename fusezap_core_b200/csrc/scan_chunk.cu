@@ -17,19 +17,22 @@
 // Two kernels. The first has a block per (chunk, head), all independent: decays, unit vectors, P, T, W and V' in 32-bit, left in
 // a record of scratch memory as operands of matrix products, each 32-bit number as the sum of two bfloat16 numbers (its
 // rounding and the rounding of what is left; the products of two rests are dropped: a relative error of 2^-17 per term). The
-// second walks a portion's chunks in order: a warp keeps 16 value columns of S^T in its accumulators from the portion's first
-// chunk to its last; as the first operand of the products with Q and W, and with U^T as the first operand of the products with
-// P and K, the accumulators' own layout is that of the operand, so the state never leaves the registers. The next two
-// chunks' records travel to shared memory meanwhile (cp.async).
+// second walks a portion's chunks in order: a block owns 32 value columns of a head of a portion, and each of its four warps
+// keeps 16 of them x half of the key channels of S^T in its accumulators from the portion's first chunk to its last. As the
+// first operand of the products with Q and W, and with U^T as the first operand of the products with P and K, the accumulators'
+// own layout is that of the operand, so the state never leaves the registers. What the two halves of the key channels add up
+// to (o, and for the delta rule W S) passes through shared memory. A chunk's record, and the block's columns of V, travel to
+// shared memory in one bulk copy each, two chunks ahead; the first kernel writes them in the layout they are used in.
 #include "attn_mma.cuh"
+#include "tma.cuh"
 #include <math.h>
 
 namespace {
 using namespace fzattn;
 constexpr int C = 16;                       // tokens per chunk
 constexpr int COOK_THREADS = 256;
-constexpr int WARPS = 4;                    // warps of the second kernel: 16 value columns each
-constexpr int STAGES = 3;
+constexpr int SLICE = 32;                   // value columns per block of the second kernel
+constexpr int STAGES = 6;                  // chunks in shared memory at a time
 constexpr float LOG2E = 1.4426950408889634f;
 
 // 2^x for x <= 0 (results below the normal range are zero)
@@ -47,38 +50,50 @@ __device__ __forceinline__ void split2(float a, float b, uint32_t& hi, uint32_t&
   lo = pack_bf16(a - f.x, b - f.y);
 }
 
-// The record of a (chunk, head), in bytes: MATS matrices [16][dkp] of bf16 (Q, K and for the delta rule W; rounding, then
-// rest), P [16][16] (rounding, rest), the decays of the chunk (dkp floats), V: rounding and rest [16][dvp] bf16 (linear
-// attention) or V' [16][dvp] float (delta rule).
-struct Record {
-  int dkp, dvp, mats;
-  __host__ __device__ Record(int dkp_, int dv, bool delta) : dkp(dkp_), dvp((dv + 15) / 16 * 16), mats(delta ? 6 : 4) {}
-  __host__ __device__ int mat() const { return C * dkp * 2; }
-  __host__ __device__ int p() const { return mats * mat(); }
-  __host__ __device__ int decay() const { return p() + 2 * C * C * 2; }
-  __host__ __device__ int v() const { return decay() + dkp * 4; }
-  __host__ __device__ long long bytes() const { return v() + C * dvp * 4; }
+// The record of a (chunk, head), in bytes. Main part: MATS matrices [16][DKP] of bf16 (Q, K and for the delta rule W; rounding,
+// then rest), P [16][16] (rounding, rest), the chunk's decays (DKP floats). Then V in slices of 32 columns: rounding and rest
+// [16][32] bf16 (linear attention) or V' [16][32] float (delta rule). Every row is 16 bytes longer than its values (an odd
+// number of 16-byte units: the rows that are read together from shared memory fall into different banks).
+template <int DKP, bool DELTA> struct Record {
+  static constexpr int MATS = DELTA ? 6 : 4, ROW = DKP * 2 + 16, MAT = C * ROW, P_ROW = C * 2 + 16, P_MAT = C * P_ROW;
+  static constexpr int P = MATS * MAT, DECAY = P + 2 * P_MAT, MAIN = DECAY + DKP * 4;
+  static constexpr int V_ROW = SLICE * (DELTA ? 4 : 2) + 16, V_MAT = C * V_ROW, V = (DELTA ? 1 : 2) * V_MAT;
+  static constexpr int STAGE = MAIN + V;
 };
+__host__ __device__ inline int slices_of(int dv) { return (dv + SLICE - 1) / SLICE; }
+template <int DKP, bool DELTA> __host__ __device__ inline long long record_bytes(int dv) {
+  return Record<DKP, DELTA>::MAIN + (long long)slices_of(dv) * Record<DKP, DELTA>::V;
+}
 // The records of a portion that begins at row r stand from place ceil(r / 8) on. A portion of n >= 16 rows has ceil(n / 16) of
 // them, and ceil((r + n) / 8) >= ceil(r / 8) + ceil((n - 7) / 8) >= ceil(r / 8) + ceil(n / 16): no two portions of 16 rows and
 // more share a place, and a step of N rows needs ceil(N / 8) places, whatever portions it holds.
 __device__ __forceinline__ long long record_place(int row0, int chunk) { return (row0 + 7) / 8 + chunk; }
 
-// A [16][cols] matrix of shared memory (ld floats per row) times row factors, as rounding and rest.
-template <typename Fn>
-__device__ __forceinline__ void leave_matrix(unsigned char* hi, unsigned char* lo, int cols, Fn value) {
-  for (int e = threadIdx.x; e < C * cols / 2; e += COOK_THREADS) {
-    const int t = e / (cols / 2), c = 2 * (e - t * (cols / 2));
+// A [16][DKP] matrix as rounding (matrix `m` of the record) and rest (the one after it); value2(t, c): elements c and c + 1.
+template <int DKP, bool DELTA, typename Fn>
+__device__ __forceinline__ void leave_matrix(unsigned char* rec, int m, Fn value2) {
+  using R = Record<DKP, DELTA>;
+  const int c = 2 * (threadIdx.x % (DKP / 2));
+#pragma unroll
+  for (int t = threadIdx.x / (DKP / 2); t < C; t += 2 * COOK_THREADS / DKP) {
+    const float2 v = value2(t, c);
     uint32_t h, l;
-    split2(value(t, c), value(t, c + 1), h, l);
-    ((uint32_t*)hi)[e] = h;
-    ((uint32_t*)lo)[e] = l;
+    split2(v.x, v.y, h, l);
+    *(uint32_t*)(rec + m * R::MAT + t * R::ROW + 2 * c) = h;
+    *(uint32_t*)(rec + (m + 1) * R::MAT + t * R::ROW + 2 * c) = l;
   }
+}
+// Row t of P, whose element `lane` is v: rounding and rest.
+template <typename R>
+__device__ __forceinline__ void leave_p(unsigned char* rec, int t, int lane, float v) {
+  const __nv_bfloat16 hi = __float2bfloat16_rn(v);
+  *(__nv_bfloat16*)(rec + R::P + t * R::P_ROW + 2 * lane) = hi;
+  *(__nv_bfloat16*)(rec + R::P + R::P_MAT + t * R::P_ROW + 2 * lane) = __float2bfloat16_rn(v - __bfloat162float(hi));
 }
 
 struct CookArgs {
   const int* seg;
-  int H, Hk, dk, dv, dkp, min_rows;
+  int H, Hk, dk, dv, min_rows;
   unsigned char* scratch;
   // linear attention: proj rows of ld floats [q heads | k heads | v heads | ...], z rows of H dk decay inputs
   const float* proj;
@@ -97,112 +112,113 @@ struct CookArgs {
 };
 
 // grid (portions, chunks of the longest portion, heads)
+template <int DKP>
 __global__ void __launch_bounds__(COOK_THREADS)
 gla_cook_kernel(const CookArgs a) {
+  using R = Record<DKP, false>;
   fz_grid_launch_dependents();
   const int s = blockIdx.x, c0 = blockIdx.y * C, h = blockIdx.z;
   const int row0 = a.seg[4 * s], cnt = a.seg[4 * s + 1], slot = a.seg[4 * s + 3];
   fz_grid_wait();
   if (cnt < a.min_rows || c0 >= cnt || slot < 0) return;
-  extern __shared__ __align__(16) float sm[];
-  const int dk = a.dk, dkp = a.dkp, LD = dkp + 1, valid = min(C, cnt - c0);
-  float* q = sm;                 // [16][LD]
-  float* k = q + C * LD;
-  float* L = k + C * LD;         // logarithms (base 2) of the decays, then their running sums
-  const Record rec(dkp, a.dv, false);
-  unsigned char* out = a.scratch + (record_place(row0, blockIdx.y) * a.H + h) * rec.bytes();
+  constexpr int LD = DKP + 4;
+  __shared__ __align__(16) float q[C * LD], k[C * LD], L[C * LD];      // L: logarithms (base 2) of the decays, then their running sums
+  const int dk = a.dk, valid = min(C, cnt - c0), tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  unsigned char* rec = a.scratch + (record_place(row0, blockIdx.y) * a.H + h) * record_bytes<DKP, false>(a.dv);
   const size_t n0 = (size_t)(row0 + c0);
-  for (int e = threadIdx.x; e < C * dkp; e += COOK_THREADS) {
-    const int t = e / dkp, c = e - t * dkp;
-    float qv = 0.f, kv = 0.f, lv = 0.f;
-    if (c < dk && t < valid) {
-      const float* in = a.proj + (n0 + t) * a.ld;
-      qv = __fmul_rn(in[(size_t)h * dk + c], a.q_scale);
-      kv = in[(size_t)(a.H + h) * dk + c];
-      lv = -a.inv_root * softplus32(-a.z[(n0 + t) * a.H * dk + (size_t)h * dk + c]) * LOG2E;
+  {
+    const int c = tid % DKP;
+#pragma unroll
+    for (int t = tid / DKP; t < C; t += COOK_THREADS / DKP) {
+      float qv = 0.f, kv = 0.f, lv = 0.f;
+      if (c < dk && t < valid) {
+        const float* in = a.proj + (n0 + t) * a.ld;
+        qv = __fmul_rn(in[(size_t)h * dk + c], a.q_scale);
+        kv = in[(size_t)(a.H + h) * dk + c];
+        lv = -a.inv_root * softplus32(-a.z[(n0 + t) * a.H * dk + (size_t)h * dk + c]) * LOG2E;
+      }
+      q[t * LD + c] = qv;
+      k[t * LD + c] = kv;
+      L[t * LD + c] = lv;
     }
-    q[t * LD + c] = qv;
-    k[t * LD + c] = kv;
-    L[t * LD + c] = lv;
   }
-  {                              // V needs nothing of the above
-    unsigned char* v = out + rec.v();
-    leave_matrix(v, v + C * rec.dvp * 2, rec.dvp, [&](int t, int c) {
-      return t < valid && c < a.dv ? a.proj[(n0 + t) * a.ld + (size_t)2 * a.H * dk + (size_t)h * a.dv + c] : 0.f;
-    });
+#pragma unroll
+  for (int half = 0; half < 2; ++half) {         // V needs nothing of the above
+    const int t = warp + 8 * half;
+    const float* in = a.proj + (n0 + t) * a.ld + (size_t)2 * a.H * dk + (size_t)h * a.dv;
+    for (int c = 2 * lane; c < slices_of(a.dv) * SLICE; c += 64) {
+      uint32_t hi, lo;
+      split2(t < valid && c < a.dv ? in[c] : 0.f, t < valid && c + 1 < a.dv ? in[c + 1] : 0.f, hi, lo);
+      unsigned char* v = rec + R::MAIN + (c / SLICE) * R::V + t * R::V_ROW + (c % SLICE) * 2;
+      *(uint32_t*)v = hi;
+      *(uint32_t*)(v + R::V_MAT) = lo;
+    }
   }
   __syncthreads();
-  if (threadIdx.x < dkp) {
+  if (tid < DKP) {
     float run = 0.f;
 #pragma unroll
-    for (int t = 0; t < C; ++t) { run += L[t * LD + threadIdx.x]; L[t * LD + threadIdx.x] = run; }
-    ((float*)(out + rec.decay()))[threadIdx.x] = ex2(run);
+    for (int t = 0; t < C; ++t) { run += L[t * LD + tid]; L[t * LD + tid] = run; }
+    ((float*)(rec + R::DECAY))[tid] = ex2(run);
   }
   __syncthreads();
-  leave_matrix(out, out + rec.mat(), dkp, [&](int t, int c) { return q[t * LD + c] * ex2(L[t * LD + c]); });
-  leave_matrix(out + 2 * rec.mat(), out + 3 * rec.mat(), dkp, [&](int t, int c) { return k[t * LD + c] * ex2(L[(C - 1) * LD + c] - L[t * LD + c]); });
-  __nv_bfloat16* P = (__nv_bfloat16*)(out + rec.p());
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  auto at = [&](const float* m, int t, int c) { return *(const float2*)(m + t * LD + c); };
+  leave_matrix<DKP, false>(rec, 0, [&](int t, int c) {
+    const float2 x = at(q, t, c), l = at(L, t, c);
+    return make_float2(x.x * ex2(l.x), x.y * ex2(l.y));
+  });
+  leave_matrix<DKP, false>(rec, 2, [&](int t, int c) {
+    const float2 x = at(k, t, c), l = at(L, t, c), e = at(L, C - 1, c);
+    return make_float2(x.x * ex2(e.x - l.x), x.y * ex2(e.y - l.y));
+  });
+  const int c = 4 * lane;                        // this lane's four key channels
+  const bool in = c < DKP;
+  const float4 none = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
   for (int half = 0; half < 2; ++half) {         // a warp takes token `warp` and token 15 - `warp`: 17 pairs
     const int t = half == 0 ? warp : C - 1 - warp;
-    float qt[4], Lt[4];
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      const int c = lane + 32 * i;
-      qt[i] = c < dkp ? q[t * LD + c] : 0.f;
-      Lt[i] = c < dkp ? L[t * LD + c] : 0.f;
-    }
+    const float4 qt = in ? *(const float4*)(q + t * LD + c) : none, Lt = in ? *(const float4*)(L + t * LD + c) : none;
     float mine = 0.f;                            // lane s keeps P_ts
     for (int x = 0; x <= t; ++x) {
-      float acc = 0.f;
-#pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        const int c = lane + 32 * i;
-        if (c < dkp) acc = fmaf(qt[i] * k[x * LD + c], ex2(Lt[i] - L[x * LD + c]), acc);
-      }
+      const float4 kx = in ? *(const float4*)(k + x * LD + c) : none, Lx = in ? *(const float4*)(L + x * LD + c) : none;
+      float acc = qt.x * kx.x * ex2(Lt.x - Lx.x);
+      acc = fmaf(qt.y * kx.y, ex2(Lt.y - Lx.y), acc);
+      acc = fmaf(qt.z * kx.z, ex2(Lt.z - Lx.z), acc);
+      acc = fmaf(qt.w * kx.w, ex2(Lt.w - Lx.w), acc);
       acc = warp_sum(acc);
       if (lane == x) mine = acc;
     }
-    if (lane < C) {
-      const __nv_bfloat16 hi = __float2bfloat16_rn(mine);
-      P[t * C + lane] = hi;
-      P[C * C + t * C + lane] = __float2bfloat16_rn(mine - __bfloat162float(hi));
-    }
+    if (lane < C) leave_p<R>(rec, t, lane, mine);
   }
 }
 
+template <int DKP>
 __global__ void __launch_bounds__(COOK_THREADS)
 delta_cook_kernel(const CookArgs a) {
+  using R = Record<DKP, true>;
   fz_grid_launch_dependents();
   const int s = blockIdx.x, c0 = blockIdx.y * C, h = blockIdx.z;
   const int row0 = a.seg[4 * s], cnt = a.seg[4 * s + 1], slot = a.seg[4 * s + 3];
   const float rate2 = expf(a.a_log[h]) * LOG2E, bias = a.dt_bias[h];
   fz_grid_wait();
   if (cnt < a.min_rows || c0 >= cnt || slot < 0) return;
-  extern __shared__ __align__(16) float sm[];
-  const int dk = a.dk, dkp = a.dkp, LD = dkp + 1, valid = min(C, cnt - c0);
-  const Record rec(dkp, a.dv, true);
-  const int dvp = rec.dvp;
-  float* q = sm;                 // [16][LD]
-  float* k = q + C * LD;
-  float* v = k + C * LD;         // [16][dvp]
-  float* M = v + C * dvp;        // [16][17]: beta_t e^{L_t - L_s} k_t . k_s below the diagonal
-  float* T1 = M + C * 17;        // [16][17]: T diag(beta)
-  float* T2 = T1 + C * 17;       // [16][17]: T diag(beta e^L)
-  float* L = T2 + C * 17;        // [16]
-  float* b = L + C;              // [16]
-  unsigned char* out = a.scratch + (record_place(row0, blockIdx.y) * a.H + h) * rec.bytes();
+  constexpr int LD = DKP + 4, TP = 17;
+  __shared__ __align__(16) float q[C * LD], k[C * LD];
+  __shared__ float M[C * TP], T1[C * TP], T2[C * TP], L[C], b[C];      // M: beta_t e^{L_t - L_s} k_t . k_s below the diagonal; T1: T diag(beta), T2: T diag(beta e^L)
+  extern __shared__ __align__(16) float v[];     // [16][columns of V, to a multiple of 32]
+  const int dk = a.dk, valid = min(C, cnt - c0), tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int dvp = slices_of(a.dv) * SLICE;
+  unsigned char* rec = a.scratch + (record_place(row0, blockIdx.y) * a.H + h) * record_bytes<DKP, true>(a.dv);
   const size_t n0 = (size_t)(row0 + c0);
   const int kh = h / (a.H / a.Hk), W = 2 * a.Hk * dk + a.H * a.dv;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  constexpr int PER = (DKP + 31) / 32;           // key channels per lane
 #pragma unroll
-  for (int half = 0; half < 2; ++half) {         // a warp brings two tokens in: unit vectors
+  for (int half = 0; half < 2; ++half) {         // a warp brings two tokens in: unit vectors, values
     const int t = warp + 8 * half;
     const __nv_bfloat16* in = a.qkv + (n0 + t) * W;
-    float qv[4], kv[4], sq = 0.f, sk = 0.f;
+    float qv[PER], kv[PER], sq = 0.f, sk = 0.f;
 #pragma unroll
-    for (int i = 0; i < 4; ++i) {
+    for (int i = 0; i < PER; ++i) {
       const int c = lane + 32 * i;
       const bool ok = c < dk && t < valid;
       qv[i] = ok ? __bfloat162float(in[(size_t)kh * dk + c]) : 0.f;
@@ -212,17 +228,15 @@ delta_cook_kernel(const CookArgs a) {
     }
     const float nq = sqrtf(warp_sum(sq) + a.unit_eps), nk = sqrtf(warp_sum(sk) + a.unit_eps);
 #pragma unroll
-    for (int i = 0; i < 4; ++i) {
+    for (int i = 0; i < PER; ++i) {
       const int c = lane + 32 * i;
-      if (c < dkp) {
+      if (c < DKP) {
         q[t * LD + c] = __fmul_rn(__fdiv_rn(qv[i], nq), a.q_scale);
         k[t * LD + c] = __fdiv_rn(kv[i], nk);
       }
     }
-  }
-  for (int e = threadIdx.x; e < C * dvp; e += COOK_THREADS) {
-    const int t = e / dvp, c = e - t * dvp;
-    v[e] = t < valid && c < a.dv ? __bfloat162float(a.qkv[(n0 + t) * W + (size_t)2 * a.Hk * dk + (size_t)h * a.dv + c]) : 0.f;
+    const __nv_bfloat16* vin = in + (size_t)2 * a.Hk * dk + (size_t)h * a.dv;
+    for (int c = lane; c < dvp; c += 32) v[t * dvp + c] = t < valid && c < a.dv ? __bfloat162float(vin[c]) : 0.f;
   }
   if (warp == 0) {
     float l = 0.f, be = 0.f;
@@ -238,126 +252,125 @@ delta_cook_kernel(const CookArgs a) {
     if (lane < C) { L[lane] = l; b[lane] = be; }
   }
   __syncthreads();
-  __nv_bfloat16* P = (__nv_bfloat16*)(out + rec.p());
+  const int c = 4 * lane;                        // this lane's four key channels
+  const bool in = c < DKP;
+  const float4 none = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
   for (int half = 0; half < 2; ++half) {
     const int t = half == 0 ? warp : C - 1 - warp;
-    float qt[4], kt[4];
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      const int c = lane + 32 * i;
-      qt[i] = c < dkp ? q[t * LD + c] : 0.f;
-      kt[i] = c < dkp ? k[t * LD + c] : 0.f;
-    }
+    const float4 qt = in ? *(const float4*)(q + t * LD + c) : none, kt = in ? *(const float4*)(k + t * LD + c) : none;
     float qk = 0.f, kk = 0.f;                    // lane s keeps the products with k_s
     for (int x = 0; x <= t; ++x) {
-      float p = 0.f, m = 0.f;
-#pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        const int c = lane + 32 * i;
-        const float kx = c < dkp ? k[x * LD + c] : 0.f;
-        p = fmaf(qt[i], kx, p);
-        m = fmaf(kt[i], kx, m);
-      }
-      p = warp_sum(p);
-      m = warp_sum(m);
+      const float4 kx = in ? *(const float4*)(k + x * LD + c) : none;
+      const float p = warp_sum(fmaf(qt.x, kx.x, fmaf(qt.y, kx.y, fmaf(qt.z, kx.z, qt.w * kx.w))));
+      const float m = warp_sum(fmaf(kt.x, kx.x, fmaf(kt.y, kx.y, fmaf(kt.z, kx.z, kt.w * kx.w))));
       if (lane == x) { qk = p; kk = m; }
     }
     if (lane < C) {
       const float f = lane <= t ? ex2(L[t] - L[lane]) : 0.f;
-      qk *= f;
-      const __nv_bfloat16 hi = __float2bfloat16_rn(qk);
-      P[t * C + lane] = hi;
-      P[C * C + t * C + lane] = __float2bfloat16_rn(qk - __bfloat162float(hi));
-      M[t * 17 + lane] = lane < t ? b[t] * f * kk : 0.f;
+      leave_p<R>(rec, t, lane, qk * f);
+      M[t * TP + lane] = lane < t ? b[t] * f * kk : 0.f;
     }
   }
   __syncthreads();
-  if (threadIdx.x < C) {                         // column j of T by substitution: T_tj = [t = j] - sum_{s < t} M_ts T_sj
-    const int j = threadIdx.x;
+  if (tid < C) {                                 // column j of T by substitution: T_tj = [t = j] - sum_{s < t} M_ts T_sj
+    const int j = tid;
     float x[C];
 #pragma unroll
     for (int t = 0; t < C; ++t) {
       float acc = t == j ? 1.f : 0.f;
 #pragma unroll
-      for (int y = 0; y < t; ++y) acc = fmaf(-M[t * 17 + y], x[y], acc);
+      for (int y = 0; y < t; ++y) acc = fmaf(-M[t * TP + y], x[y], acc);
       x[t] = acc;
     }
     const float b1 = b[j], b2 = b1 * ex2(L[j]);
 #pragma unroll
-    for (int t = 0; t < C; ++t) { T1[t * 17 + j] = x[t] * b1; T2[t * 17 + j] = x[t] * b2; }
+    for (int t = 0; t < C; ++t) { T1[t * TP + j] = x[t] * b1; T2[t * TP + j] = x[t] * b2; }
   }
   const float last = L[C - 1];
-  leave_matrix(out, out + rec.mat(), dkp, [&](int t, int c) { return q[t * LD + c] * ex2(L[t]); });
-  leave_matrix(out + 2 * rec.mat(), out + 3 * rec.mat(), dkp, [&](int t, int c) { return k[t * LD + c] * ex2(last - L[t]); });
-  if (threadIdx.x < dkp) ((float*)(out + rec.decay()))[threadIdx.x] = ex2(last);
+  auto at = [&](const float* m, int t, int c) { return *(const float2*)(m + t * LD + c); };
+  leave_matrix<DKP, true>(rec, 0, [&](int t, int c) {
+    const float2 x = at(q, t, c);
+    const float f = ex2(L[t]);
+    return make_float2(x.x * f, x.y * f);
+  });
+  leave_matrix<DKP, true>(rec, 2, [&](int t, int c) {
+    const float2 x = at(k, t, c);
+    const float f = ex2(last - L[t]);
+    return make_float2(x.x * f, x.y * f);
+  });
+  if (tid < DKP) ((float*)(rec + R::DECAY))[tid] = ex2(last);
   __syncthreads();
-  leave_matrix(out + 4 * rec.mat(), out + 5 * rec.mat(), dkp, [&](int t, int c) {
-    float acc = 0.f;
-    for (int y = 0; y <= t; ++y) acc = fmaf(T2[t * 17 + y], k[y * LD + c], acc);
+  leave_matrix<DKP, true>(rec, 4, [&](int t, int c) {
+    float2 acc = make_float2(0.f, 0.f);
+    for (int y = 0; y <= t; ++y) {
+      const float2 x = at(k, y, c);
+      const float f = T2[t * TP + y];
+      acc.x = fmaf(f, x.x, acc.x);
+      acc.y = fmaf(f, x.y, acc.y);
+    }
     return acc;
   });
-  float* vout = (float*)(out + rec.v());
-  for (int e = threadIdx.x; e < C * dvp; e += COOK_THREADS) {
-    const int t = e / dvp, c = e - t * dvp;
-    float acc = 0.f;
-    for (int y = 0; y <= t; ++y) acc = fmaf(T1[t * 17 + y], v[y * dvp + c], acc);
-    vout[e] = acc;
+#pragma unroll
+  for (int half = 0; half < 2; ++half) {         // a warp takes token `warp` and token 15 - `warp`: 17 terms in all
+    const int t = half == 0 ? warp : C - 1 - warp;
+    for (int c = lane; c < dvp; c += 32) {
+      float acc = 0.f;
+      for (int y = 0; y <= t; ++y) acc = fmaf(T1[t * TP + y], v[y * dvp + c], acc);
+      *(float*)(rec + R::MAIN + (c / SLICE) * R::V + t * R::V_ROW + (c % SLICE) * 4) = acc;
+    }
   }
 }
 
-// ---- the second kernel: grid (portions, heads, blocks of 64 value columns)
-// A stage of shared memory: the record's matrices with rows of dkp + 8 values, P with rows of 24, the decays, this block's 64
-// columns of V with rows of 72 bf16 (rounding, rest) or 68 floats (an odd number of 16-byte units per row: no bank conflicts).
-template <int DKP, bool DELTA> struct Stage {
-  static constexpr int MATS = DELTA ? 6 : 4, ROW = DKP * 2 + 16, MAT = C * ROW, P_ROW = 48, P_MAT = C * P_ROW;
-  static constexpr int P = MATS * MAT, DECAY = P + 2 * P_MAT, V = DECAY + DKP * 4;
-  static constexpr int V_ROW = DELTA ? 272 : 144, V_MAT = C * V_ROW, BYTES = V + (DELTA ? 1 : 2) * V_MAT;
-};
+__device__ __forceinline__ void bulk_load(uint32_t dst, const void* src, uint32_t bytes, uint64_t* bar) {
+  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];"
+               ::"r"(dst), "l"(src), "r"(bytes), "r"(smem_u32(bar)) : "memory");
+}
+__device__ __forceinline__ void pair_barrier(int id) { asm volatile("bar.sync %0, 64;" ::"r"(id) : "memory"); }
 
-template <int DKP, bool DELTA>
-__global__ void __launch_bounds__(32 * WARPS)
+// ---- the second kernel: grid (portions, heads, slices of 32 value columns), 64 KS threads: warp w owns columns 16 (w % 2) ..
+// + 15 of the slice and part w / 2 of the KS parts of the key channels.
+template <int DKP, bool DELTA, int KS>
+__global__ void __launch_bounds__(64 * KS)
 scan_chunk_kernel(const unsigned char* __restrict__ scratch, int H, int dv, float* __restrict__ state, const int* __restrict__ seg,
-                  int min_rows, float* __restrict__ out) {
-  using St = Stage<DKP, DELTA>;
+                  int min_rows, float* __restrict__ out, int* err) {
+  using R = Record<DKP, DELTA>;
   fz_grid_launch_dependents();
-  const int s = blockIdx.x, h = blockIdx.y, col0 = blockIdx.z * 16 * WARPS;
+  const int s = blockIdx.x, h = blockIdx.y, slice = blockIdx.z;
   const int row0 = seg[4 * s], cnt = seg[4 * s + 1], slot = seg[4 * s + 3];
   fz_grid_wait();
   if (cnt < min_rows || cnt <= 0 || slot < 0) return;
   extern __shared__ __align__(128) unsigned char smem[];
+  __shared__ uint64_t full[STAGES];
+  __shared__ float xo[KS > 1 ? 2 : 1][2][8][32];                 // results of the second half of the key channels, by chunk parity
+  __shared__ float xd[DELTA && KS > 1 ? 2 * KS : 1][8][32];      // a warp's part of W S
   const uint32_t s0 = smem_u32(smem);
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, cg = warp & 1, kh = warp >> 1;
   const int g = lane >> 2, q2 = 2 * (lane & 3);            // an accumulator's row (and row + 8) and first column
-  const Record rec(DKP, dv, DELTA);
   const int nc = (cnt + C - 1) / C;
-  const unsigned char* base = scratch + (record_place(row0, 0) * H + h) * rec.bytes();
-  const long long step = (long long)H * rec.bytes();
-  const int vcols = min(16 * WARPS, rec.dvp - col0);       // this block's columns of V (a multiple of 16)
+  const long long bytes = record_bytes<DKP, DELTA>(dv), step = (long long)H * bytes;
+  const unsigned char* base = scratch + (record_place(row0, 0) * H + h) * bytes;
 
-  auto issue = [&](int c) {
-    if (c < nc) {
-      const unsigned char* r = base + c * step;
-      const uint32_t st = s0 + (c % STAGES) * St::BYTES;
-      constexpr int PER = DKP / 8;                         // 16-byte pieces per row
-      for (int e = tid; e < St::MATS * C * PER; e += 32 * WARPS) cp_async16(st + (e / PER) * St::ROW + (e % PER) * 16, r + e * 16, true);
-      for (int e = tid; e < 2 * C * 2; e += 32 * WARPS) cp_async16(st + St::P + (e >> 1) * St::P_ROW + (e & 1) * 16, r + rec.p() + e * 16, true);
-      if (tid < DKP / 4) cp_async16(st + St::DECAY + tid * 16, r + rec.decay() + tid * 16, true);
-      const int rows = DELTA ? C : 2 * C, per = DELTA ? vcols / 4 : vcols / 8, src = rec.dvp * (DELTA ? 4 : 2), at = col0 * (DELTA ? 4 : 2);
-      for (int e = tid; e < rows * per; e += 32 * WARPS) {
-        const int t = e / per, i = e - t * per;
-        cp_async16(st + St::V + t * St::V_ROW + i * 16, r + rec.v() + (long long)t * src + at + i * 16, true);
-      }
-    }
-    cp_async_commit();                                     // (an empty group past the last chunk keeps the count)
+  if (tid == 0) {
+    for (int i = 0; i < STAGES; ++i) fztma::mbar_init(&full[i], 1);
+    fztma::mbar_init_fence();
+  }
+  auto issue = [&](int c) {                                // one thread
+    const unsigned char* r = base + c * step;
+    const uint32_t st = s0 + (c % STAGES) * R::STAGE;
+    uint64_t* bar = &full[c % STAGES];
+    fztma::mbar_expect_tx(bar, R::STAGE);
+    bulk_load(st, r, R::MAIN, bar);
+    bulk_load(st + R::MAIN, r + R::MAIN + (long long)slice * R::V, R::V, bar);
   };
-#pragma unroll
-  for (int c = 0; c < STAGES - 1; ++c) issue(c);
+  if (tid == 0)
+    for (int c = 0; c < STAGES - 1 && c < nc; ++c) issue(c);
 
-  constexpr int KN = DKP / 16;
+  constexpr int KN = DKP / 16 / KS;                        // 16-channel steps of this warp
+  const int k0 = kh * KN;
   float S[2 * KN][4];                                      // S^T: rows are value columns, columns are key channels
-  const int ca = col0 + 16 * warp + g, cb = ca + 8;        // this thread's two value columns
-  float* sa = state + (((size_t)slot * H + h) * dv + ca) * DKP + q2;
+  const int ca = slice * SLICE + 16 * cg + g, cb = ca + 8; // this thread's two value columns
+  float* sa = state + (((size_t)slot * H + h) * dv + ca) * DKP + 16 * k0 + q2;
   float* sb = sa + (size_t)8 * DKP;
 #pragma unroll
   for (int n = 0; n < 2 * KN; ++n) {
@@ -368,88 +381,106 @@ scan_chunk_kernel(const unsigned char* __restrict__ scratch, int H, int dv, floa
   const int mi = lane >> 3, l7 = lane & 7;
   // rows of operands whose 16 rows are the product's columns (Q, W, P), and of those whose rows are summed over (K, V)
   const uint32_t off_n = ((mi >> 1) * 8 + l7), off_k = ((mi & 1) * 8 + l7);
-  const bool mine = 16 * warp < vcols;
+  float O[2][4];                                           // results of the chunk in hand (columns x tokens)
+  auto leave_results = [&](int c) {                        // by the warps of the first part: theirs and the second part's
+    const int valid = min(C, cnt - c * C);
+    float* dst = out + ((size_t)(row0 + c * C) * H + h) * dv;
+#pragma unroll
+    for (int n = 0; n < 2; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int t = 8 * n + q2 + (e & 1), col = e < 2 ? ca : cb;
+        const float y = KS > 1 ? O[n][e] + xo[c & 1][cg][4 * n + e][lane] : O[n][e];
+        if (t < valid && col < dv) dst[(size_t)t * H * dv + col] = y;
+      }
+  };
+  __syncthreads();                                         // the barriers are ready
 
   for (int c = 0; c < nc; ++c) {
-    cp_async_wait<STAGES - 2>();
-    __syncthreads();
-    issue(c + STAGES - 1);                                 // into the place of chunk c - 1
-    if (!mine) continue;
-    const uint32_t st = s0 + (c % STAGES) * St::BYTES;
-    const unsigned char* sp = smem + (c % STAGES) * St::BYTES;
-    float O[3][2][4], D[DELTA ? 3 : 1][2][4];              // hi . hi, rest . hi, hi . rest
+    const bool ok = fztma::mbar_wait(&full[c % STAGES], (c / STAGES) & 1);
+    if (!__syncthreads_and(ok)) {                          // (also: everyone is done with chunk c - 1)
+      if (tid == 0) atomicOr(err, FZ_ERR_WAIT_TIMEOUT);
+      return;
+    }
+    if (tid == 0 && c + STAGES - 1 < nc) issue(c + STAGES - 1);      // into the place of chunk c - 1
+    if (c > 0 && kh == 0) leave_results(c - 1);
+    const uint32_t st = s0 + (c % STAGES) * R::STAGE;
+    const unsigned char* sp = smem + (c % STAGES) * R::STAGE;
+    uint32_t hi[KN][4], lo[KN][4];                         // the state as a first operand
 #pragma unroll
-    for (int x = 0; x < 3; ++x)
+    for (int k = 0; k < KN; ++k) {
+      split2(S[2 * k][0], S[2 * k][1], hi[k][0], lo[k][0]);
+      split2(S[2 * k][2], S[2 * k][3], hi[k][1], lo[k][1]);
+      split2(S[2 * k + 1][0], S[2 * k + 1][1], hi[k][2], lo[k][2]);
+      split2(S[2 * k + 1][2], S[2 * k + 1][3], hi[k][3], lo[k][3]);
+    }
+    float acc[3][2][4];                                    // hi . hi, rest . hi, hi . rest
+    auto clear = [&]() {
+#pragma unroll
+      for (int x = 0; x < 3; ++x)
+#pragma unroll
+        for (int n = 0; n < 2; ++n)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) acc[x][n][e] = 0.f;
+    };
+    auto times = [&](const uint32_t (&ah)[4], const uint32_t (&al)[4], uint32_t at_hi, uint32_t at_lo) {
+      uint32_t bh[4], bl[4];
+      ldmatrix_x4(bh, at_hi);
+      ldmatrix_x4(bl, at_lo);
+#pragma unroll
+      for (int n = 0; n < 2; ++n) {
+        mma_bf16(acc[0][n], ah, bh[2 * n], bh[2 * n + 1]);
+        mma_bf16(acc[1][n], al, bh[2 * n], bh[2 * n + 1]);
+        mma_bf16(acc[2][n], ah, bl[2 * n], bl[2 * n + 1]);
+      }
+    };
+    const uint32_t a_q = st + off_n * R::ROW + (mi & 1) * 16 + 32 * k0;
+    float D[2][4];
+    if constexpr (DELTA) {                                 // this part of W S
+      clear();
+#pragma unroll
+      for (int k = 0; k < KN; ++k) times(hi[k], lo[k], a_q + 4 * R::MAT + 32 * k, a_q + 5 * R::MAT + 32 * k);
 #pragma unroll
       for (int n = 0; n < 2; ++n)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) { O[x][n][e] = 0.f; if (DELTA) D[DELTA ? x : 0][n][e] = 0.f; }
-    const uint32_t a_q = st + off_n * St::ROW + (mi & 1) * 16;
-#pragma unroll
-    for (int k = 0; k < KN; ++k) {
-      uint32_t hi[4], lo[4];
-      split2(S[2 * k][0], S[2 * k][1], hi[0], lo[0]);
-      split2(S[2 * k][2], S[2 * k][3], hi[1], lo[1]);
-      split2(S[2 * k + 1][0], S[2 * k + 1][1], hi[2], lo[2]);
-      split2(S[2 * k + 1][2], S[2 * k + 1][3], hi[3], lo[3]);
-      uint32_t bh[4], bl[4];
-      ldmatrix_x4(bh, a_q + 32 * k);
-      ldmatrix_x4(bl, a_q + St::MAT + 32 * k);
-#pragma unroll
-      for (int n = 0; n < 2; ++n) {
-        mma_bf16(O[0][n], hi, bh[2 * n], bh[2 * n + 1]);
-        mma_bf16(O[1][n], lo, bh[2 * n], bh[2 * n + 1]);
-        mma_bf16(O[2][n], hi, bl[2 * n], bl[2 * n + 1]);
-      }
-      if constexpr (DELTA) {
-        ldmatrix_x4(bh, a_q + 4 * St::MAT + 32 * k);
-        ldmatrix_x4(bl, a_q + 5 * St::MAT + 32 * k);
-#pragma unroll
-        for (int n = 0; n < 2; ++n) {
-          mma_bf16(D[0][n], hi, bh[2 * n], bh[2 * n + 1]);
-          mma_bf16(D[1][n], lo, bh[2 * n], bh[2 * n + 1]);
-          mma_bf16(D[2][n], hi, bl[2 * n], bl[2 * n + 1]);
+        for (int e = 0; e < 4; ++e) {
+          D[n][e] = acc[0][n][e] + (acc[1][n][e] + acc[2][n][e]);
+          if (KS > 1) xd[warp][4 * n + e][lane] = D[n][e];
         }
-      }
     }
+    clear();
+#pragma unroll
+    for (int k = 0; k < KN; ++k) times(hi[k], lo[k], a_q + 32 * k, a_q + R::MAT + 32 * k);
     uint32_t uh[4], ul[4];                                 // U^T (value columns x tokens) as a first operand
     if constexpr (DELTA) {
-      const float* v = (const float*)(sp + St::V) + 16 * warp + g;
-      constexpr int VR = St::V_ROW / 4;
+      if (KS > 1) {
+        pair_barrier(1 + cg);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) D[i >> 2][i & 3] = xd[cg][i][lane] + xd[cg + 2][i][lane];      // (the same order in both warps)
+      }
+      const float* v = (const float*)(sp + R::MAIN) + 16 * cg + g;
+      constexpr int VR = R::V_ROW / 4;
       float U[2][4];
 #pragma unroll
       for (int n = 0; n < 2; ++n)
 #pragma unroll
-        for (int e = 0; e < 4; ++e)
-          U[n][e] = v[(8 * n + q2 + (e & 1)) * VR + (e >> 1) * 8] - (D[0][n][e] + (D[1][n][e] + D[2][n][e]));
+        for (int e = 0; e < 4; ++e) U[n][e] = v[(8 * n + q2 + (e & 1)) * VR + (e >> 1) * 8] - D[n][e];
       split2(U[0][0], U[0][1], uh[0], ul[0]);
       split2(U[0][2], U[0][3], uh[1], ul[1]);
       split2(U[1][0], U[1][1], uh[2], ul[2]);
       split2(U[1][2], U[1][3], uh[3], ul[3]);
     } else {
-      const uint32_t a_v = st + St::V + off_n * St::V_ROW + (16 * warp + (mi & 1) * 8) * 2;
+      const uint32_t a_v = st + R::MAIN + off_n * R::V_ROW + (16 * cg + (mi & 1) * 8) * 2;
       ldmatrix_x4_trans(uh, a_v);
-      ldmatrix_x4_trans(ul, a_v + St::V_MAT);
+      ldmatrix_x4_trans(ul, a_v + R::V_MAT);
     }
-    {
-      const uint32_t a_p = st + St::P + off_n * St::P_ROW + (mi & 1) * 16;
-      uint32_t bh[4], bl[4];
-      ldmatrix_x4(bh, a_p);
-      ldmatrix_x4(bl, a_p + St::P_MAT);
-#pragma unroll
-      for (int n = 0; n < 2; ++n) {
-        mma_bf16(O[0][n], uh, bh[2 * n], bh[2 * n + 1]);
-        mma_bf16(O[1][n], ul, bh[2 * n], bh[2 * n + 1]);
-        mma_bf16(O[2][n], uh, bl[2 * n], bl[2 * n + 1]);
-      }
-    }
-    const uint32_t a_k = st + 2 * St::MAT + off_k * St::ROW + (mi >> 1) * 16;
-    const float* dec = (const float*)(sp + St::DECAY) + q2;
+    const uint32_t a_k = st + 2 * R::MAT + off_k * R::ROW + (mi >> 1) * 16 + 32 * k0;
+    const float* dec = (const float*)(sp + R::DECAY) + 16 * k0 + q2;
 #pragma unroll
     for (int k = 0; k < KN; ++k) {
       uint32_t bh[4], bl[4];
       ldmatrix_x4_trans(bh, a_k + 32 * k);
-      ldmatrix_x4_trans(bl, a_k + St::MAT + 32 * k);
+      ldmatrix_x4_trans(bl, a_k + R::MAT + 32 * k);
 #pragma unroll
       for (int n = 0; n < 2; ++n) {
         float* x = S[2 * k + n];
@@ -460,18 +491,20 @@ scan_chunk_kernel(const unsigned char* __restrict__ scratch, int H, int dv, floa
         mma_bf16(x, uh, bl[2 * n], bl[2 * n + 1]);
       }
     }
-    const int valid = min(C, cnt - c * C);
-    float* dst = out + ((size_t)(row0 + c * C) * H + h) * dv;
+    if (kh == KS - 1) {
+      const uint32_t a_p = st + R::P + off_n * R::P_ROW + (mi & 1) * 16;
+      times(uh, ul, a_p, a_p + R::P_MAT);
+    }
 #pragma unroll
     for (int n = 0; n < 2; ++n)
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        const int t = 8 * n + q2 + (e & 1), col = e < 2 ? ca : cb;
-        if (t < valid && col < dv) dst[(size_t)t * H * dv + col] = O[0][n][e] + (O[1][n][e] + O[2][n][e]);
+        O[n][e] = acc[0][n][e] + (acc[1][n][e] + acc[2][n][e]);
+        if (KS > 1 && kh == 1) xo[c & 1][cg][4 * n + e][lane] = O[n][e];
       }
   }
-  cp_async_wait<0>();
-  if (!mine) return;
+  __syncthreads();
+  if (kh == 0) leave_results(nc - 1);
 #pragma unroll
   for (int n = 0; n < 2 * KN; ++n) {
     if (ca < dv) *(float2*)(sa + 8 * n) = make_float2(S[n][0], S[n][1]);
@@ -496,36 +529,36 @@ int allow_smem(K kern, size_t smem, size_t& allowed) {
 }
 
 template <int DKP, bool DELTA>
-int launch_scan(const CookArgs& a, float* state, int n_seg, float* out, cudaStream_t stream) {
-  constexpr size_t smem = (size_t)STAGES * Stage<DKP, DELTA>::BYTES;
-  static size_t allowed = 48 * 1024;
-  int st = allow_smem(scan_chunk_kernel<DKP, DELTA>, smem, allowed);
-  if (st != FZ_OK) return st;
-  fz_launch(scan_chunk_kernel<DKP, DELTA>, dim3(n_seg, a.H, (a.dv + 16 * WARPS - 1) / (16 * WARPS)), dim3(32 * WARPS), smem, stream,
-            (const unsigned char*)a.scratch, a.H, a.dv, state, a.seg, a.min_rows, out);
+int launch_both(const CookArgs& a, float* state, int n_seg, int max_rows, float* out, int* err, cudaStream_t stream) {
+  constexpr int KS = DKP >= 32 ? 2 : 1;
+  const int chunks = (max_rows + C - 1) / C;
+  if (chunks > 65535) return FZ_TOO_LARGE;
+  const size_t cook_smem = DELTA ? sizeof(float) * C * slices_of(a.dv) * SLICE : 0;
+  constexpr size_t smem = (size_t)STAGES * Record<DKP, DELTA>::STAGE;
+  static size_t allowed_c = 16 * 1024, allowed = 32 * 1024;      // (beside their static shared memory)
+  auto cook = DELTA ? delta_cook_kernel<DKP> : gla_cook_kernel<DKP>;
+  auto scan = scan_chunk_kernel<DKP, DELTA, KS>;
+  int st = allow_smem(cook, cook_smem, allowed_c);
+  if (st != FZ_OK || (st = allow_smem(scan, smem, allowed)) != FZ_OK) return st;
+  fz_launch(cook, dim3(n_seg, chunks, a.H), dim3(COOK_THREADS), cook_smem, stream, a);
+  FZ_LAUNCH_CHECK();
+  fz_launch(scan, dim3(n_seg, a.H, slices_of(a.dv)), dim3(64 * KS), smem, stream, (const unsigned char*)a.scratch, a.H, a.dv, state, a.seg,
+            a.min_rows, out, err);
   FZ_LAUNCH_CHECK();
   return FZ_OK;
 }
 
 template <bool DELTA>
-int run(CookArgs a, float* state, int n_seg, int max_rows, float* out, cudaStream_t stream) {
-  a.dkp = padded_keys(a.dk);
-  const int chunks = (max_rows + C - 1) / C, LD = a.dkp + 1;
-  if (chunks > 65535) return FZ_TOO_LARGE;
-  const Record rec(a.dkp, a.dv, DELTA);
-  const size_t smem = sizeof(float) * (DELTA ? 2 * (size_t)C * LD + (size_t)C * rec.dvp + 3 * C * 17 + 2 * C : 3 * (size_t)C * LD);
-  static size_t allowed = 48 * 1024;
-  auto cook = DELTA ? delta_cook_kernel : gla_cook_kernel;
-  int st = allow_smem(cook, smem, allowed);
-  if (st != FZ_OK) return st;
-  fz_launch(cook, dim3(n_seg, chunks, a.H), dim3(COOK_THREADS), smem, stream, a);
-  FZ_LAUNCH_CHECK();
-  switch (a.dkp) {
-    case 16: return launch_scan<16, DELTA>(a, state, n_seg, out, stream);
-    case 32: return launch_scan<32, DELTA>(a, state, n_seg, out, stream);
-    case 64: return launch_scan<64, DELTA>(a, state, n_seg, out, stream);
-    default: return launch_scan<128, DELTA>(a, state, n_seg, out, stream);
+int run(const CookArgs& a, float* state, int n_seg, int max_rows, float* out, int* err, cudaStream_t stream) {
+  switch (padded_keys(a.dk)) {
+    case 16: return launch_both<16, DELTA>(a, state, n_seg, max_rows, out, err, stream);
+    case 32: return launch_both<32, DELTA>(a, state, n_seg, max_rows, out, err, stream);
+    case 64: return launch_both<64, DELTA>(a, state, n_seg, max_rows, out, err, stream);
+    default: return launch_both<128, DELTA>(a, state, n_seg, max_rows, out, err, stream);
   }
+}
+template <bool DELTA> long long bytes_of(int dkp, int dv) {
+  return dkp == 16 ? record_bytes<16, DELTA>(dv) : dkp == 32 ? record_bytes<32, DELTA>(dv) : dkp == 64 ? record_bytes<64, DELTA>(dv) : record_bytes<128, DELTA>(dv);
 }
 }  // namespace
 
@@ -536,31 +569,32 @@ FZ_API int fz_scan_chunk_check(int H, int dk, int dv) {
 
 // Bytes of scratch for a step of N rows (see record_place).
 FZ_API long long fz_scan_chunk_scratch(int N, int H, int dk, int dv, int delta) {
-  return ((long long)N / 8 + 1) * H * Record(padded_keys(dk), dv, delta != 0).bytes();
+  const int dkp = padded_keys(dk);
+  return ((long long)N / 8 + 1) * H * (delta ? bytes_of<true>(dkp, dv) : bytes_of<false>(dkp, dv));
 }
 
 // Portions of min_rows rows and more (max_rows at most); the state is (slots, H, dv, padded keys). See fz_channel_decay_scan.
 FZ_API int fz_gla_chunk(const float* proj, int ld, int H, int dk, int dv, const float* z, float inv_root, float q_scale, float* state,
-                        const int* seg, int n_seg, int min_rows, int max_rows, void* scratch, float* out, cudaStream_t stream) {
+                        const int* seg, int n_seg, int min_rows, int max_rows, void* scratch, float* out, int* err, cudaStream_t stream) {
   if (n_seg <= 0) return FZ_OK;
   if (fz_scan_chunk_check(H, dk, dv) != FZ_OK || ld < H * (2 * dk + dv) || scratch == nullptr || ((uintptr_t)scratch & 15) || min_rows < C) return FZ_BAD_SHAPE;
   CookArgs a = {};
   a.seg = seg; a.H = a.Hk = H; a.dk = dk; a.dv = dv; a.min_rows = min_rows; a.scratch = (unsigned char*)scratch;
   a.proj = proj; a.ld = ld; a.z = z; a.inv_root = inv_root; a.q_scale = q_scale;
-  return run<false>(a, state, n_seg, max_rows, out, stream);
+  return run<false>(a, state, n_seg, max_rows, out, err, stream);
 }
 
 // See fz_gated_delta_scan (one decay per head).
 FZ_API int fz_delta_chunk(const void* qkv, int H, int Hk, int dk, int dv, const float* high, int ldh, const float* beta, int ldb,
                           const float* a_log, const float* dt_bias, float unit_eps, float q_scale, float* state, const int* seg,
-                          int n_seg, int min_rows, int max_rows, void* scratch, float* out, cudaStream_t stream) {
+                          int n_seg, int min_rows, int max_rows, void* scratch, float* out, int* err, cudaStream_t stream) {
   if (n_seg <= 0) return FZ_OK;
   if (fz_scan_chunk_check(H, dk, dv) != FZ_OK || Hk <= 0 || H % Hk || scratch == nullptr || ((uintptr_t)scratch & 15) || min_rows < C) return FZ_BAD_SHAPE;
   CookArgs a = {};
   a.seg = seg; a.H = H; a.Hk = Hk; a.dk = dk; a.dv = dv; a.min_rows = min_rows; a.scratch = (unsigned char*)scratch;
   a.qkv = (const __nv_bfloat16*)qkv; a.high = high; a.ldh = ldh; a.beta = beta; a.ldb = ldb; a.a_log = a_log; a.dt_bias = dt_bias;
   a.unit_eps = unit_eps; a.q_scale = q_scale;
-  return run<true>(a, state, n_seg, max_rows, out, stream);
+  return run<true>(a, state, n_seg, max_rows, out, err, stream);
 }
 
 #ifdef FZ_TIMELINE

@@ -1084,7 +1084,7 @@ class CudaOps(Ops):
             scratch = self._chunk_scratch(n, heads, key_dim, value_dim, True)
             self._check(self.scan_tc.fz_delta_chunk(
                 _p(qkv), c_int(heads), c_int(key_heads), c_int(key_dim), c_int(value_dim), *inputs, _p(state), _p(meta.seg),
-                c_int(meta.max_segments), c_int(SCAN_CHUNK_ROWS), c_int(max_portion), _p(scratch), _p(out), self._stream()),
+                c_int(meta.max_segments), c_int(SCAN_CHUNK_ROWS), c_int(max_portion), _p(scratch), _p(out), _p(self.err), self._stream()),
                 "gated_delta_scan (tensor cores)", nbytes)
             self.launches += 1
             if max_portion == n:
@@ -1113,7 +1113,7 @@ class CudaOps(Ops):
         if max_portion >= SCAN_CHUNK_ROWS and self._scan_chunked(heads, key_dim, value_dim):
             # long portions 16 tokens at a time on tensor cores, the step's short ones (if it can have any) token by token
             scratch = self._chunk_scratch(n, heads, key_dim, value_dim, False)
-            self._check(self.scan_tc.fz_gla_chunk(*inputs, c_int(SCAN_CHUNK_ROWS), c_int(max_portion), _p(scratch), _p(out), self._stream()),
+            self._check(self.scan_tc.fz_gla_chunk(*inputs, c_int(SCAN_CHUNK_ROWS), c_int(max_portion), _p(scratch), _p(out), _p(self.err), self._stream()),
                         "channel_decay_scan (tensor cores)", nbytes)
             self.launches += 1
             if max_portion == n:

@@ -95,7 +95,7 @@ MUR_TC = model(96, 64, 1e-5, [               # sizes that the tensor-core kernel
     1,
     layer(par(left(2, 1, 128, 128, 0.1, 1e4, 64), right(2, 1, 64, 64, 2)), dense(64)),
 ])
-CONFIGS = {"mix": (MUR_MIX, 3), "odd": (MUR_ODD, 5), "one": (MUR_ONE, 9), "tc": (MUR_TC, 4)}
+CONFIGS = {"mix": (MUR_MIX, 3), "odd": (MUR_ODD, 5), "one": (MUR_ONE, 9), "tc": (MUR_TC, 13)}
 STD_SCALE = 5.0
 
 
