@@ -35,6 +35,9 @@ shared expert in a parallel block), beside Gizulorn at equal sizes.
 `--workload gimupel` (`--sizes p1024,p2048`, `--layers 4`) does the same for the Gimupel design (selective state space
 layers with a convolution and a gated norm in parts, windowed attention with normed heads, experts chosen by corrected
 sigmoid scores in groups, layers run twice with the embedding added again), beside Gizulorn at equal sizes.
+`--workload muretar` (`--sizes r1024,r2048`, `--layers 4`) does the same for the Muretar design (a norm before and after each
+sublayer, gated linear attention, attention beside the delta rule with one decay per head, differential attention, ungated
+experts beside ones that hand their input on), beside Gizulorn at equal sizes.
 `--workload pepilix` (`--sizes w1024,w2048`, `--layers 4`) times the Pepilix design beside the dense decoder at equal
 width, layers, heads, vocabulary and active feed-forward size: a 2,048-token prompt and decode steps at `--batch`
 requests through `LLMEngine.step()`, and (unless `--no-points`) a kernel-by-kernel profile of both; its line's `sizes`

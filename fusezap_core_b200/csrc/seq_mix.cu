@@ -1207,6 +1207,47 @@ moe_combine_kernel(const float* __restrict__ terms, const float* __restrict__ w,
   }
 }
 
+// The same for D % 4 == 0 and 16-byte aligned rows, four values per thread: every value's sum is the scalar kernel's.
+__device__ __forceinline__ float4 input4(const float* p) { return *(const float4*)p; }
+__device__ __forceinline__ float4 input4(const __nv_bfloat16* p) {
+  const uint2 v = *(const uint2*)p;
+  const float2 a = __bfloat1622float2(*(const __nv_bfloat162*)&v.x), b = __bfloat1622float2(*(const __nv_bfloat162*)&v.y);
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+template <typename TH>
+__global__ void __launch_bounds__(256)
+moe_combine_vec_kernel(const float* __restrict__ terms, const float* __restrict__ w, int top, const float* __restrict__ shared,
+                       const float* __restrict__ gl, int ldg, int col, const int* __restrict__ seq_row, float* __restrict__ out,
+                       int N, int D, const float* __restrict__ add, float scale, const int* __restrict__ choice, int n_experts,
+                       const TH* __restrict__ hin) {
+  fz_grid_launch_dependents();
+  fz_grid_wait();
+  const int n = blockIdx.x, d = 4 * (blockIdx.y * blockDim.x + threadIdx.x);
+  if (d >= D) return;
+  const bool pad = seq_row[n] < 0;
+  float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+  auto take = [&](float f, float4 t) {
+    acc.x = __fmaf_rn(f, t.x, acc.x); acc.y = __fmaf_rn(f, t.y, acc.y); acc.z = __fmaf_rn(f, t.z, acc.z); acc.w = __fmaf_rn(f, t.w, acc.w);
+  };
+  if (!pad) {
+    float sg = 1.f;
+    if (shared != nullptr && gl != nullptr) sg = 1.0f / (1.0f + expf(-gl[(size_t)n * ldg + col]));
+    const size_t at0 = (size_t)n * top;
+#pragma unroll 4
+    for (int k = 0; k < top; ++k) {
+      const bool hand_on = choice != nullptr && choice[at0 + k] >= n_experts;
+      take(w[at0 + k], hand_on ? input4(hin + (size_t)n * D + d) : *(const float4*)(terms + (at0 + k) * D + d));
+    }
+    if (shared != nullptr) take(sg, *(const float4*)(shared + (size_t)n * D + d));
+    if (add != nullptr) {
+      const float4 t = *(const float4*)(add + (size_t)n * D + d);
+      acc.x = __fadd_rn(acc.x, t.x); acc.y = __fadd_rn(acc.y, t.y); acc.z = __fadd_rn(acc.z, t.z); acc.w = __fadd_rn(acc.w, t.w);
+    }
+    if (scale != 1.f) { acc.x = __fmul_rn(acc.x, scale); acc.y = __fmul_rn(acc.y, scale); acc.z = __fmul_rn(acc.z, scale); acc.w = __fmul_rn(acc.w, scale); }
+  }
+  *(float4*)(out + (size_t)n * D + d) = acc;
+}
+
 // ------------------------------------------------------------------------------ real-gated linear recurrent unit
 // Per channel c of part b (W / B channels each): r = sigmoid(g_r + bias), i = sigmoid(g_i + bias),
 // a = exp(-k_c r) with k_c = sharpness * softplus(lam_c), S <- a S + sqrt(1 - a^2) (i u), out = S y. Everything in
@@ -1696,13 +1737,13 @@ FZ_API int fz_moe_combine(const float* terms, const float* w, int top, const flo
                           int n_experts, const void* hin, int hin_dtype, cudaStream_t stream) {
   if (N <= 0 || D <= 0) return FZ_OK;
   if (choice != nullptr && hin == nullptr) return FZ_BAD_SHAPE;
-  const int by = (D + 1023) / 1024 > 0 ? (D + 1023) / 1024 : 1;
-  if (hin_dtype == FZ_BF16)
-    fz_launch(moe_combine_kernel<__nv_bfloat16>, dim3(N, by), dim3(256), 0, stream, terms, w, top, shared, gl, ldg, col, seq_row, out, N,
-              D, add, scale, choice, n_experts, (const __nv_bfloat16*)hin);
-  else
-    fz_launch(moe_combine_kernel<float>, dim3(N, by), dim3(256), 0, stream, terms, w, top, shared, gl, ldg, col, seq_row, out, N, D, add,
-              scale, choice, n_experts, (const float*)hin);
+  const bool vec = D % 4 == 0 && (((uintptr_t)terms | (uintptr_t)shared | (uintptr_t)out | (uintptr_t)add | (uintptr_t)hin) & 15) == 0;
+  const int threads = !vec ? 256 : D >= 1024 ? 256 : (D / 4 + 31) / 32 * 32;
+  const dim3 grid(N, vec ? (D / 4 + threads - 1) / threads : (D + 1023) / 1024);
+#define FZ_COMBINE(KERNEL, TH) fz_launch(KERNEL<TH>, grid, dim3(threads), 0, stream, terms, w, top, shared, gl, ldg, col, seq_row, out, N, D, add, scale, choice, n_experts, (const TH*)hin)
+  if (hin_dtype == FZ_BF16) { if (vec) FZ_COMBINE(moe_combine_vec_kernel, __nv_bfloat16); else FZ_COMBINE(moe_combine_kernel, __nv_bfloat16); }
+  else { if (vec) FZ_COMBINE(moe_combine_vec_kernel, float); else FZ_COMBINE(moe_combine_kernel, float); }
+#undef FZ_COMBINE
   FZ_LAUNCH_CHECK();
   return FZ_OK;
 }

@@ -147,6 +147,22 @@ def make_dir(name: str, tmp, cfg: dict | None = None, seed: int | None = None, c
     return d, cfg, read_model_dir(d)
 
 
+def corrections_apart(w: dict) -> None:
+    """Router corrections further apart than any two scores, so that no choice hangs on rounding."""
+    for k in [k for k in w if k.endswith("correction")]:
+        n = w[k].shape[0]
+        w[k] = torch.randperm(n, generator=torch.Generator().manual_seed(n)).float() * 1.5 - 4.0
+
+
+def other_rank(w: dict, rank: int) -> None:
+    """Gives every two-step decay projection this inner size."""
+    g = torch.Generator().manual_seed(rank)
+    for k in [k for k in w if k.endswith("mix.a1")]:
+        k2 = k[:-1] + "2"
+        w[k] = torch.randn(rank, w[k].shape[1], generator=g) * 0.1
+        w[k2] = torch.randn(w[k2].shape[0], rank, generator=g) * 0.5
+
+
 def drawn_config(seed: int, small: bool = True) -> dict:
     """A configuration drawn from a seed: the layer types in any order, odd and even sizes (the tensor-core kernels' among
     them), with and without feed-forward, layers that share weights."""

@@ -8,7 +8,7 @@ import pytest
 import torch
 
 import plain_muretar as plain
-from muretar_util import CONFIGS, MUR_MIX, MUR_ODD, MUR_ONE, MUR_TC, Oracle, drawn_config, make_dir, plain_logits, tokens_for
+from muretar_util import CONFIGS, MUR_MIX, MUR_ODD, MUR_ONE, MUR_TC, Oracle, drawn_config, make_dir, other_rank, plain_logits, tokens_for
 from pepilix_util import rel_rms, run_cut, run_mixed
 from plain_ops import PlainOpsSandwich
 from fusezap_core_b200 import LLMEngine, SamplingParams
@@ -242,6 +242,16 @@ def test_greedy_generation_through_the_entry_point(dirs):
         for i, t in enumerate(new):
             row = lg[len(prompt) - 1 + i]
             assert int(row.argmax()) == t or row.max() - row[t] < 1e-3
+
+
+def test_the_decay_projections_inner_size_is_the_checkpoints(tmp_path):
+    """Whatever it is: five, which no product's tile divides, and more than the width."""
+    for rank in (5, 80):
+        d, cfg, w = make_dir(f"rank{rank}", tmp_path, MUR_MIX, 3, change=lambda t: other_rank(t, rank))
+        assert w["l1.mix.a1"].shape[0] == rank
+        model, cache, runner = engine_parts(d)
+        toks = tokens_for(cfg, (40,), seed=rank)[0]
+        Oracle(cfg, w, toks, "float32").check(run_cut(runner, cache, "r", toks, (11, 2, 1)), rank)
 
 
 @pytest.mark.parametrize("seed", range(12))
