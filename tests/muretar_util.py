@@ -89,7 +89,7 @@ MUR_ONE = model(61, 32, 1e-4, [              # single heads; layer 0 uses the we
 ])
 MUR_TC = model(96, 64, 1e-5, [               # sizes that the tensor-core kernels of long portions take
     layer(par(left(4, 1, 64, 32, 0.15, 2e5, 64, 3.0), right(4, 2, 32, 32, 4)), moe(8, 2, 3, 32, 64)),
-    layer(att(4, 2, 32, 64, 0.2, 0.4), moe(8, 4, 2, 64)),
+    layer(att(6, 3, 32, 64, 0.2, 0.4), moe(8, 4, 2, 64)),
     layer(gla(2, 64, 32, 12.0), dense(64)),
     layer(att(2, 2, 64, 128, 0.15, 0.7), None),
     1,

@@ -183,7 +183,7 @@ def near_exact(got, ref, dtype, what):
     assert not (err > 3e-5 * (ref.abs() + ref.abs().max())).any(), (what, float((err / ref.abs().max()).max()))
 
 
-GLA_SIZES = [(3, 12, 20, 16.0), (1, 40, 16, 0.5), (5, 30, 6, 2.0), (2, 64, 32, 12.0), (2, 128, 128, 16.0), (1, 9, 7, 1.0), (2, 48, 64, 16.0),
+GLA_SIZES = [(3, 12, 20, 16.0), (1, 40, 16, 0.5), (5, 30, 6, 2.0), (2, 64, 32, 12.0), (2, 128, 128, 16.0), (1, 9, 7, 1.0), (3, 48, 64, 14.0),
              (3, 16, 16, 4.0), (1, 200, 40, 3.0), (2, 96, 300, 8.0), (1, 256, 16, 1.0), (4, 80, 48, 0.8)]
 
 
@@ -342,7 +342,7 @@ def near(got, ref, dtype, what=None):
     assert not (err > tol * (ref.abs() + ref.abs().mean() + 1e-3)).any(), (what, float(err.max()))
 
 
-DIFF_SIZES = [(4, 2, 9, 16), (6, 3, 20, 12), (1, 1, 33, 17), (2, 1, 4, 8), (4, 2, 32, 64), (2, 2, 64, 128), (4, 1, 64, 64), (3, 3, 32, 128),
+DIFF_SIZES = [(4, 2, 9, 16), (6, 3, 20, 12), (1, 1, 33, 17), (2, 1, 4, 8), (6, 3, 32, 64), (2, 2, 64, 128), (4, 1, 64, 64), (3, 3, 32, 128),
               (6, 2, 64, 128), (16, 2, 16, 40), (40, 1, 8, 24), (2, 1, 128, 256)]
 
 
